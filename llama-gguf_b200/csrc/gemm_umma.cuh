@@ -15,9 +15,9 @@
 //     16-byte chunks into the K-major SWIZZLE_128B shared-memory tile (chunk c of row r at chunk c ^ (r & 7));
 //   * the activations (fp16 in HBM, rounded once by their producer) are copied into a second tile the same way;
 //   * fence.proxy.async, then ONE elected thread issues 4 x tcgen05.mma.cta_group::1.kind::f16 (M = 128 weight rows,
-//     N = TN tokens, K = 16 each; SASS UTCHMMA) on the two shared-memory descriptors; the f32 accumulator lives in TMEM
+//     N = TN tokens, K = 16 each) on the two shared-memory descriptors; the f32 accumulator lives in TMEM
 //     (TN columns x 128 lanes); tcgen05.commit -> mbarrier tells the CTA that the tiles may be overwritten;
-//   * epilogue: warp w reads TMEM lanes 32w..32w+31 with tcgen05.ld.32x32b.x32 (SASS LDTM), thread = weight row, 32
+//   * epilogue: warp w reads TMEM lanes 32w..32w+31 with tcgen05.ld.32x32b.x32, thread = weight row, 32
 //     tokens per load, and stores Y so that a warp writes 32 consecutive floats of one token's row.
 // fp16 operands, f32 accumulation: measured 3e-4 of the largest output against a double-precision dequant-then-dot
 // (tools/umma_lab.cu); the exact token-by-token path stays the default where bit-level greedy parity matters.

@@ -8,7 +8,7 @@
 // weights of a 32-row pass at 370 GB/s.  One persistent CTA per SM walks a list of (128 weight rows, TN tokens, K range)
 // items; its warps have fixed roles and meet only through mbarriers — there is no CTA-wide barrier in the loop:
 //
-//   warp 4      PRODUCER   one thread: per 256-element block of K one cp.async.bulk.tensor.2d (SASS UTMALDG) of the RAW
+//   warp 4      PRODUCER   one thread: per 256-element block of K one cp.async.bulk.tensor.2d of the RAW
 //                          GGUF bytes of 128 weight rows (tensor map over the untouched GGUF layout, box = 128 rows x one
 //                          block) into the raw ring, and per 64-element K step one box of TN activation rows x 128 bytes
 //                          through a SWIZZLE_128B tensor map over X into the B ring.  It runs ahead across item
@@ -18,9 +18,9 @@
 //                          as ONE f32 FMA on 1024 + q, rounded to fp16) and writes the row's eight 16-byte chunks into a
 //                          K-major SWIZZLE_128B stage of the A ring; fence.proxy.async + one mbarrier arrive per warp.
 //   warp 5      MMA        one thread: waits for the A and B stage of a step, issues 4 x tcgen05.mma.cta_group::1.kind::f16
-//                          (M = 128 rows, N = TN tokens, K = 16; SASS UTCHMMA), tcgen05.commit releases both stages; the
+//                          (M = 128 rows, N = TN tokens, K = 16), tcgen05.commit releases both stages; the
 //                          f32 accumulator of an item is one of TWO TMEM buffers, committed to the epilogue at item end.
-//   warps 0..3  EPILOGUE   tcgen05.ld (SASS LDTM) of the finished accumulator (warp w = TMEM lanes 32w..), bias / residual
+//   warps 0..3  EPILOGUE   tcgen05.ld of the finished accumulator (warp w = TMEM lanes 32w..), bias / residual
 //                          accumulate / split-K partial store, then hands the buffer back: the epilogue of item i overlaps
 //                          the main loop of item i + 1.
 //

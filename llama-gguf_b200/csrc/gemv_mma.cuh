@@ -9,7 +9,7 @@
 //
 // Second generation (profiles/v1_mega_ncu_full.md: the fp16 HMMA version spent 4.1 thread-instructions per
 // weight, half of them outside the dot products, and the token was issue-bound):
-//  * the dot products are INTEGER tensor-pipe MMAs (mma.sync.m16n8k32 u8 x s8 -> s32, SASS IMMA.16832):
+//  * the dot products are INTEGER tensor-pipe MMAs (mma.sync.m16n8k32 u8 x s8 -> s32):
 //    a 32-bit word of nibbles becomes four A-operand quants with ONE LOP3 (w & 0x0F0F0F0F; the high nibbles are
 //    w & 0xF0F0F0F0 = 16 q, the 1/16 goes into the scale), i.e. 0.25 instructions per weight for the unpack
 //    instead of 0.5 + the fp16 bias handling;
@@ -24,7 +24,7 @@
 //    converted with PRMT into the mantissa of 2^23 (no I2F);
 //  * a unit is 32 rows x 256 elements: per-unit overhead (producer, B-operand loads, loop) is paid once per
 //    8192 weights, and a finished tile is 32 consecutive outputs in one warp (one x-scale group of the next GEMV);
-//  * weights go HBM -> shared memory with 16-byte cp.async (SASS LDGSTS) into PER-WARP rings of 2-4 stages; a warp
+//  * weights go HBM -> shared memory with 16-byte cp.async into PER-WARP rings of 2-4 stages; a warp
 //    produces and consumes its own ring (no cross-warp hand-off) and the first stages are issued BEFORE the
 //    dependency wait (weights never depend on the previous kernel / phase of the token);
 //  * stream-K: all (tile, chunk) units of a launch are dealt evenly, in contiguous runs, to the warps of a
@@ -230,7 +230,7 @@ __device__ __forceinline__ void lds_piece8(uint32_t a, uint32_t& o0, uint32_t& o
     }
 }
 
-// Integer tensor-pipe MMAs (SASS IMMA.16832): D[16x8] += A[16x32] * B[32x8], s32 accumulators.
+// Integer tensor-pipe MMAs: D[16x8] += A[16x32] * B[32x8], s32 accumulators.
 // Fragments (lane = 4n + t): a0 = A[n][4t..4t+3], a1 = A[n+8][4t..], a2 = A[n][16+4t..], a3 = A[n+8][16+4t..];
 // b0 = B[4t..4t+3][n], b1 = B[16+4t..][n]; d0 = D[n][2t], d1 = D[n][2t+1], d2 = D[n+8][2t], d3 = D[n+8][2t+1].
 __device__ __forceinline__ void imma_u8s8(int (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {

@@ -7,7 +7,7 @@
 // here they are fetched by a warp that is not part of any phase:
 //
 //   * producer = one elected lane of warp 8.  It walks the same phase program as the consumers, but only the GEMV
-//     phases, and issues ONE `cp.async.bulk.tensor.2d` (TMA, SASS UTMALDG) per ring entry: a box of 32 weight rows x
+//     phases, and issues ONE `cp.async.bulk.tensor.2d` (TMA) per ring entry: a box of 32 weight rows x
 //     4 super-blocks (Q4_K: 32 x 576 B) straight from the untouched GGUF row layout, described by a tensor map per
 //     weight matrix ([n_rows][row_bytes], encoded once at model load).  Rows / columns past the end of a matrix are
 //     zero-filled by the TMA unit (a zero block has d = 0: it contributes nothing), so ragged shapes need no code.

@@ -21,7 +21,7 @@
 //     epilogue (bias, residual, SwiGLU, staged int8 form of the output) and moves on.  Four tile slots, generation-checked.
 //   * the loader warp owns the phase boundary: it waits for the CTA's consumers on an mbarrier, arrives at the grid
 //     barrier (one red.release.gpu per CTA), polls it, and pulls the phase's input into shared memory with ONE bulk copy
-//     (cp.async.bulk, SASS UBLKCP) that completes on the mbarrier the consumers wait on; the next phase's descriptor
+//     (cp.async.bulk) that completes on the mbarrier the consumers wait on; the next phase's descriptor
 //     rides on the same mbarrier.  Consumers go from their last entry of phase p straight to the set-up of phase p + 1.
 //   * attention (attn2_phase): K/V rows of earlier positions are requested BEFORE the boundary is waited for (they do
 //     not depend on this token), q / k / v of the new position arrive through the loader's bulk copies and are rotated
@@ -102,7 +102,7 @@ __device__ __forceinline__ void pdesc2_load(PDesc2& d, const MegaPhase* P) {
 }
 
 // One issuing thread is latency-bound: a try_wait that succeeds at once, expect_tx, the operand moves to uniform registers and the
-// UTMALDG issue take ~400 clocks per entry (measured: producer stamps of b200_debug_mega_phase), i.e. 23 B/clk for a 9 KB entry --
+// TMA issue take ~400 clocks per entry (measured: producer stamps of b200_debug_mega_phase), i.e. 23 B/clk for a 9 KB entry --
 // the HBM rate per SM with no slack, and the reason round 1's gate/up phase never went below 19 us.  So the ring is fed by
 // kS2Prods producer warps; producer `pidx` issues the entries whose global sequence number is pidx modulo kS2Prods (the slot of
 // an entry is its sequence number modulo n_slots, whoever issues it).

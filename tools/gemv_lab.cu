@@ -616,7 +616,7 @@ __global__ void __launch_bounds__(512, 1) stream_bulk_kernel(const StreamParams 
     if (acc == 0x12345678u) p.sink[0] = acc;
 }
 
-// cp.async (LDGSTS) 16 B per lane, commit groups per stage
+// cp.async 16 B per lane, commit groups per stage
 __global__ void __launch_bounds__(512, 1) stream_cpasync_kernel(const StreamParams p) {
     extern __shared__ __align__(128) uint8_t smem[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;

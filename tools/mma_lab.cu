@@ -1,5 +1,5 @@
 // mma_lab.cu — latency / throughput of the legacy warp-level MMA and dot-product instructions on sm_100a, the
-// numbers the dequant-GEMV design depends on: IMMA.16832 (u8 x s8), HMMA.16816 (f16 -> f32), IDP.4A (dp4a).
+// numbers the dequant-GEMV design depends on: m16n8k32 u8 x s8, m16n8k16 f16 -> f32, dp4a.
 // One CTA per SM, W warps per CTA; every warp runs `chains` independent dependent-chains of `iters` instructions.
 #include <cuda_runtime.h>
 #include <cstdio>
