@@ -278,8 +278,9 @@ B200_API const char* b200_batch_last_error(b200_batch* batch);   /* message of t
  *          (W_uk[n]^T q_plain), scores and the weighted sum run over the cached rows as one shared K/V head of size kv_rank + rot_dim
  *          / kv_rank, and W_uv[n] is applied to the summed latent.  score = (q_plain . k_plain + q_rot . k_rot) * scale; sliding window
  *          of mask_size positions (0 = all earlier positions); rotation in the half-split layout (channel i with i + dims / 2) with the
- *          frequencies of b200_rotary_desc; optional sigmoid gate per value channel from the mixer's input ('.g'); kv_from >= 0: the
- *          layer has no W_dkv and reads the cache rows of that earlier layer (same kv_rank, rot_dim and rotation) with its own W_uk,
+ *          frequencies of b200_rotary_desc, or, with rot_pairs = 1, in the interleaved layout (channel 2i with 2i + 1); q_rank = 0: there is
+ *          no query latent, q = W_q h ('.q'); optional sigmoid gate from the mixer's input ('.g') per value channel or one per head;
+ *          kv_from >= 0: the layer has no W_dkv and reads the cache rows of that earlier layer (same kv_rank, rot_dim and rotation) with its own W_uk,
  *          W_uv, queries and mask.
  *   B200_MIX_STATE_SPACE    gated linear recurrence with a scalar decay per head (b200_state_space_desc): W_in h = [z | x | B | C | dt]
  *          with inner = heads * vdim, B and C of groups * state; causal depthwise convolution ('.conv' [channels, taps], bias
@@ -311,6 +312,11 @@ B200_API const char* b200_batch_last_error(b200_batch* batch);   /* message of t
  * moe.route = B200_ROUTE_SIGMOID_TOP: scores sigmoid(logit), the `top` largest taken with their scores as weights (times route_scale
  * when it is not 0), not renormalised; moe.act = B200_ACT_SILU_GLU: gated experts W_down (silu(W_gate .) * W_up .) ('.e<j>.gate');
  * moe.weight_input = 1: the weight multiplies the expert's input, sum_e expert_e(w_e h), instead of its output.
+ * moe.act = B200_ACT_CLAMPED_GLU: experts (and the always-on expert, with shared_limit) in the form of B200_FF_CLAMPED_GLU with `limit`
+ * and `slope`; moe.router_bias = 1: '.router.b' is added to the logits; moe.shared_gate = 1: the always-on expert's output is multiplied by
+ * sigmoid(W_sg h), one number per token ('.shared.sg', [1, width]).
+ * B200_FF_XIELU: W_down act(W_up h) of width ff with the two numbers (p, q) = '.act': act(z) = softplus(p) z^2 + z / 2 for z > 0,
+ * (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 for z <= 0.
  * parallel_ff = 1 (with post_norm = 0, streams = 0): a layer has one norm and its feed-forward reads the mixer's input,
  * h = norm1(x), x += mixer(h) + ff(h); the layer's input projection then also holds the feed-forward's ([gate | up] or the router).
  * Layer form (program): post_norm = 0: x += sublayer(norm(x)); post_norm = 1: x <- norm(residual_alpha * x + sublayer(x)), the
@@ -320,6 +326,13 @@ B200_API const char* b200_batch_last_error(b200_batch* batch);   /* message of t
  * norm(sum_s hc<q>.in[s] x_s) and its output y updates all copies at once, x_t <- sum_s hc<q>.mix[s][t] x_s + residual_mult *
  * hc<q>.out[t] * y; the head reads the sum of the copies.  A layer without 'l<i>.hc<q>.*' tensors takes in = out = 1, mix = identity
  * (with one stream: x += residual_mult * y).
+ * norm_scalar = 1: 'norm1', 'norm2', 'final.norm' and 'embed.norm' hold ONE number for all coordinates.  embed_norm = 1: the embedding is
+ * normed ('embed.norm') before the first layer.  loop_in = 1: ahead of every pass of the repeated range x <- 'loop.in' [x; x0] ([width,
+ * 2 width], x0 = the embedding as the first layer reads it), then the pass's step vector is added.
+ * in_conv = taps >= 1: what a sublayer reads, h = norm(x), becomes h + conv(h), a causal convolution over time on every channel
+ * ('l<i>.canon1' for the mixer, 'l<i>.canon2' for the feed-forward, [width, taps], conv(h)_t = sum_j w[:, j] h_(t - taps + 1 + j), zeros
+ * before the sequence's start); a slot's state block keeps the last taps inputs per sublayer and layer run.  in_conv and loop_in belong to
+ * the norm-first form with one residual stream and two norms per layer.
  * Embedding: row * embed_scale (+ sinusoidal position vector, pos_sinusoid); logits = head . norm(x) * logit_scale.
  * compute: 0 = bf16 weights and GEMM operands with f32 accumulation (residual stream, norms, softmax, gates and every recurrent
  * state stay f32), 1 = everything in f32 (FMA, no reduced-precision matrix mode). */
@@ -332,10 +345,10 @@ enum { B200_COMBINE_WEIGHTED = 0, B200_COMBINE_NORMED_MEAN = 1 };
 enum { B200_QKNORM_NONE = 0, B200_QKNORM_HEAD_WEIGHT = 1, B200_QKNORM_WHOLE_WEIGHT = 2, B200_QKNORM_HEAD_UNIT = 3 };
 enum { B200_GATE_NONE = 0, B200_GATE_CHANNEL = 1, B200_GATE_HEAD = 2 };
 enum { B200_VMIX_NONE = 0, B200_VMIX_SOURCE = 1, B200_VMIX_BLEND = 2 };
-enum { B200_FF_RELU2 = 0, B200_FF_GATED_GELU = 1, B200_FF_MOE = 2, B200_FF_CLAMPED_GLU = 3 };
+enum { B200_FF_RELU2 = 0, B200_FF_GATED_GELU = 1, B200_FF_MOE = 2, B200_FF_CLAMPED_GLU = 3, B200_FF_XIELU = 4 };
 enum { B200_COMPUTE_BF16 = 0, B200_COMPUTE_F32 = 1 };
 enum { B200_NORM_RMS = 0, B200_NORM_LAYER = 1 };
-enum { B200_ACT_RELU2 = 0, B200_ACT_GELU = 1, B200_ACT_SILU_GLU = 2 };
+enum { B200_ACT_RELU2 = 0, B200_ACT_GELU = 1, B200_ACT_SILU_GLU = 2, B200_ACT_CLAMPED_GLU = 3 };
 enum { B200_ROUTE_TOP_SOFTMAX = 0, B200_ROUTE_SOFTMAX_TOP = 1, B200_ROUTE_SIGMOID_TOP = 2 };
 enum { B200_TYPE_BF16 = 30 };   /* ggml's id; accepted by layer-program contexts only */
 typedef struct b200_window_attn_desc {
@@ -375,6 +388,9 @@ typedef struct b200_moe_desc {
     int32_t route;                   /* B200_ROUTE_* */
     float route_scale;               /* B200_ROUTE_SOFTMAX_TOP: factor on the chosen probabilities */
     int32_t weight_input;            /* 1 = an expert's weight multiplies its input instead of its output */
+    float limit, shared_limit, slope;   /* B200_ACT_CLAMPED_GLU: clamps of the experts and of the always-on expert, slope of the gate */
+    int32_t router_bias;             /* 1 = '.router.b' ([experts]) is added to the logits */
+    int32_t shared_gate;             /* 1 = the always-on expert is multiplied by sigmoid('.shared.sg' h) */
 } b200_moe_desc;
 /* Rotary frequencies: f_i = base^(-2i / dims), i < dims / 2.  yarn_factor > 0 stretches long wavelengths: with
  * d(t) = dims ln(yarn_original / (2 pi t)) / (2 ln base), lo = max(floor(d(yarn_fast)), 0), hi = min(ceil(d(yarn_slow)), dims - 1) and
@@ -387,12 +403,13 @@ typedef struct b200_rotary_desc {
 } b200_rotary_desc;
 typedef struct b200_latent_attn_desc {
     int32_t heads, dim, rot_dim, vdim;   /* per head: dim plain + rot_dim rotated query / key channels, vdim value channels */
-    int32_t q_rank, kv_rank;
+    int32_t q_rank, kv_rank;             /* q_rank 0: no query latent, q = W_q h */
     int32_t mask_size;               /* sliding window; 0 = every earlier position */
     float scale;
     b200_rotary_desc rot;
     int32_t kv_from;                 /* -1: own W_dkv and cache rows; j: the rows of layer j */
-    int32_t out_gate;                /* B200_GATE_NONE or B200_GATE_CHANNEL ('.g': [heads * vdim, width]) */
+    int32_t out_gate;                /* B200_GATE_* ('.g': [heads * vdim, width] or [heads, width]) */
+    int32_t rot_pairs;               /* rotation layout: 0 = halves (i with i + dims / 2), 1 = neighbours (2i with 2i + 1) */
 } b200_latent_attn_desc;
 typedef struct b200_state_space_desc {
     int32_t heads, vdim, state, groups, conv, norm_groups;
@@ -434,6 +451,10 @@ typedef struct b200_program_desc {
     int32_t streams;                            /* 0: one residual stream in the forms above; >= 1: that many copies (see "streams") */
     float residual_mult;                        /* streams >= 1: factor on every sublayer's output */
     int32_t parallel_ff;                        /* 1 = one norm per layer, the feed-forward reads the mixer's input (see "parallel_ff") */
+    int32_t norm_scalar;                        /* 1 = a norm's weight is one number */
+    int32_t embed_norm;                         /* 1 = the embedding is normed with 'embed.norm' */
+    int32_t loop_in;                            /* 1 = 'loop.in' maps [x; x0] ahead of every pass of the repeated range */
+    int32_t in_conv;                            /* taps of the convolution on every sublayer's input; 0 = none */
 } b200_program_desc;
 B200_API int b200_ctx_create_layers(const b200_program_desc* prog, const b200_layer_desc* layers, int device, b200_ctx** out);
 /* One batch of token runs: run i continues sequence slot seqs[i] with lens[i] tokens (concatenated in `tokens`).  want_rows are

@@ -118,7 +118,8 @@ class SoftmaxAttnDesc(C.Structure):
 class MoeDesc(C.Structure):
     """b200_moe_desc"""
     _fields_ = [("experts", C.c_int32), ("top", C.c_int32), ("expert_ff", C.c_int32), ("shared_ff", C.c_int32), ("act", C.c_int32),
-                ("route", C.c_int32), ("route_scale", C.c_float), ("weight_input", C.c_int32)]
+                ("route", C.c_int32), ("route_scale", C.c_float), ("weight_input", C.c_int32), ("limit", C.c_float), ("shared_limit", C.c_float),
+                ("slope", C.c_float), ("router_bias", C.c_int32), ("shared_gate", C.c_int32)]
 
 
 class RotaryDesc(C.Structure):
@@ -131,7 +132,7 @@ class LatentAttnDesc(C.Structure):
     """b200_latent_attn_desc"""
     _fields_ = [("heads", C.c_int32), ("dim", C.c_int32), ("rot_dim", C.c_int32), ("vdim", C.c_int32), ("q_rank", C.c_int32),
                 ("kv_rank", C.c_int32), ("mask_size", C.c_int32), ("scale", C.c_float), ("rot", RotaryDesc), ("kv_from", C.c_int32),
-                ("out_gate", C.c_int32)]
+                ("out_gate", C.c_int32), ("rot_pairs", C.c_int32)]
 
 
 class StateSpaceDesc(C.Structure):
@@ -165,12 +166,13 @@ class ProgramDesc(C.Structure):
                 ("max_batch", C.c_int32), ("norm_eps", C.c_float), ("embed_scale", C.c_float), ("logit_scale", C.c_float),
                 ("pos_sinusoid", C.c_int32), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
                 ("compute", C.c_int32), ("post_norm", C.c_int32), ("residual_alpha", C.c_float), ("norm_weight_offset", C.c_float),
-                ("norm_kind", C.c_int32), ("streams", C.c_int32), ("residual_mult", C.c_float), ("parallel_ff", C.c_int32)]
+                ("norm_kind", C.c_int32), ("streams", C.c_int32), ("residual_mult", C.c_float), ("parallel_ff", C.c_int32),
+                ("norm_scalar", C.c_int32), ("embed_norm", C.c_int32), ("loop_in", C.c_int32), ("in_conv", C.c_int32)]
 
 
 MIX_WINDOW_MEMORY, MIX_GATED_DELTA, MIX_SOFTMAX_ATTN, MIX_LATENT_ATTN, MIX_STATE_SPACE, MIX_ATTN_RECURRENT = 1, 2, 3, 4, 5, 6
 NORM_RMS, NORM_LAYER = 0, 1
-ACT_RELU2, ACT_GELU, ACT_SILU_GLU = 0, 1, 2
+ACT_RELU2, ACT_GELU, ACT_SILU_GLU, ACT_CLAMPED_GLU = 0, 1, 2, 3
 ROUTE_TOP_SOFTMAX, ROUTE_SOFTMAX_TOP, ROUTE_SIGMOID_TOP = 0, 1, 2
 MASK_WINDOW, MASK_CHUNK, MASK_CAUSAL = 0, 1, 2
 SINK_NONE, SINK_LEARNED, SINK_ZERO = 0, 1, 2
@@ -179,7 +181,7 @@ COMBINE_WEIGHTED, COMBINE_NORMED_MEAN = 0, 1
 QKNORM_NONE, QKNORM_HEAD_WEIGHT, QKNORM_WHOLE_WEIGHT, QKNORM_HEAD_UNIT = 0, 1, 2, 3
 GATE_NONE, GATE_CHANNEL, GATE_HEAD = 0, 1, 2
 VMIX_NONE, VMIX_SOURCE, VMIX_BLEND = 0, 1, 2
-FF_RELU2, FF_GATED_GELU, FF_MOE, FF_CLAMPED_GLU = 0, 1, 2, 3
+FF_RELU2, FF_GATED_GELU, FF_MOE, FF_CLAMPED_GLU, FF_XIELU = 0, 1, 2, 3, 4
 COMPUTE_BF16, COMPUTE_F32 = 0, 1
 BF16 = 30   # ggml's id; layer-program contexts only
 

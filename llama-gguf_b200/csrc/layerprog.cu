@@ -132,14 +132,18 @@ __global__ void lp_rmsnorm_kernel(float* __restrict__ x, const float* __restrict
 
 // ------------------------------------------------------------------------------------------------ GEMM (CUDA cores)
 // Y[r][n] = epi(alpha * sum_k X[r][k] * W[n][k] + bias[n]); products of the stored operand values in f32, f32 accumulation
-// (bias: f32 per output column, or null).
-enum { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2, EPI_GELU = 3, EPI_COUNT = 4 };
+// (bias: f32 per output column, or null).  act: the two numbers of the xIELU epilogue, (softplus(p), 1/2 + softplus(q)).
+enum { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2, EPI_GELU = 3, EPI_XIELU = 4, EPI_COUNT = 5 };
+constexpr bool epi_is_act(int epi) { return epi >= EPI_RELU2; }
+// act.x z^2 + z / 2 above zero, act.y (exp(z) - 1 - z) + z / 2 below
+__device__ __forceinline__ float xielu_f(float z, float2 act) { return fmaf(0.5f, z, z > 0.0f ? act.x * z * z : act.y * (expm1f(z) - z)); }
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
 template <typename T, int EPI>
-__device__ __forceinline__ void epi_store(void* Y, size_t idx, float v) {
+__device__ __forceinline__ void epi_store(void* Y, size_t idx, float v, float2 act) {
     if (EPI == EPI_STORE) reinterpret_cast<float*>(Y)[idx] = v;
     else if (EPI == EPI_ADD) reinterpret_cast<float*>(Y)[idx] += v;
     else if (EPI == EPI_GELU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(gelu_erf_f(v));
+    else if (EPI == EPI_XIELU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(xielu_f(v, act));
     else {
         const float z = fmaxf(v, 0.0f);
         reinterpret_cast<T*>(Y)[idx] = from_f<T>(z * z);
@@ -149,7 +153,7 @@ __device__ __forceinline__ void epi_store(void* Y, size_t idx, float v) {
 // the output row `off` elements on (f32 for the store / add epilogues, the compute type for the activations)
 template <typename T, int EPI>
 __device__ __forceinline__ void* seg_rows(void* Y, size_t off) {
-    return (EPI == EPI_RELU2 || EPI == EPI_GELU) ? (void*)(reinterpret_cast<T*>(Y) + off) : (void*)(reinterpret_cast<float*>(Y) + off);
+    return epi_is_act(EPI) ? (void*)(reinterpret_cast<T*>(Y) + off) : (void*)(reinterpret_cast<float*>(Y) + off);
 }
 // Products batched over grid.z without row segments (the heads of a mixer): group z reads X and writes Y `xz` / `yz` elements on
 struct ZStride {
@@ -159,7 +163,7 @@ constexpr int GB = 64, GK = 16;
 template <typename T, int EPI>
 __global__ void __launch_bounds__(256) lp_gemm_kernel(const T* __restrict__ X, int ldx, const T* __restrict__ W, int ldw, void* __restrict__ Y,
                                                       int ldy, int R, int N, int K, float alpha, const int* __restrict__ seg, size_t w_zstride, ZStride zs,
-                                                      const float* __restrict__ bias) {
+                                                      const float* __restrict__ bias, float2 act) {
     __shared__ float As[GK][GB + 4];
     __shared__ float Bs[GK][GB + 4];
     if (!seg && gridDim.z > 1) {
@@ -208,7 +212,7 @@ __global__ void __launch_bounds__(256) lp_gemm_kernel(const T* __restrict__ X, i
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) epi_store<T, EPI>(Y, (size_t)r * ldy + n, alpha * acc[i][j] + (bias ? bias[n] : 0.0f));
+            if (n < N) epi_store<T, EPI>(Y, (size_t)r * ldy + n, alpha * acc[i][j] + (bias ? bias[n] : 0.0f), act);
         }
     }
 }
@@ -255,7 +259,8 @@ __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, uint32
 template <int TN, int EPI>
 __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict__ X, int ldx, const bf16* __restrict__ W, int ldw,
                                                          void* __restrict__ Y, int ldy, int R, int N, int K, float alpha, int* err,
-                                                         const int* __restrict__ seg, size_t w_zstride, ZStride zs, const float* __restrict__ bias) {
+                                                         const int* __restrict__ seg, size_t w_zstride, ZStride zs, const float* __restrict__ bias,
+                                                         float2 act) {
     extern __shared__ __align__(1024) uint8_t tc_smem[];
     if (!seg && gridDim.z > 1) {
         W += blockIdx.z * w_zstride;
@@ -378,7 +383,7 @@ __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict_
 #pragma unroll
                 for (int c = 0; c < 32; c++) {
                     const int t = t0 + c0 + c;
-                    if (t < R) epi_store<bf16, EPI>(Y, (size_t)t * ldy + n, alpha * __uint_as_float(v[c]) + bn);
+                    if (t < R) epi_store<bf16, EPI>(Y, (size_t)t * ldy + n, alpha * __uint_as_float(v[c]) + bn, act);
                 }
             }
         }
@@ -412,11 +417,12 @@ template <> struct Vec8<float> {
     }
 };
 #include "lp_rows_tail.cuh"
+#include "lp_input_conv.cuh"
 
 template <typename T, int EPI>
 __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, int ldx, const T* __restrict__ W, int ldw, void* __restrict__ Y,
                                                       int ldy, int R, int N, int K, float alpha, int vec_ok, int stage, RowsTail tail, int nh,
-                                                      ZStride zs, const float* __restrict__ bias) {
+                                                      ZStride zs, const float* __restrict__ bias, float2 act) {
     // nh > 0: the N outputs are heads of nh columns; head z = n / nh reads X `zs.x` elements on and writes column z * zs.y + n % nh
     extern __shared__ __align__(16) uint8_t gv_smem[];
     const T* X0 = X;
@@ -470,7 +476,7 @@ __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, i
         for (int i = 0; i < GV_ROWS; i++) {
             if (i < nr) {
                 const float s = wsum(acc[i]);
-                if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + ycol, alpha * s + (bias ? bias[n] : 0.0f));
+                if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + ycol, alpha * s + (bias ? bias[n] : 0.0f), act);
             }
         }
     }
@@ -481,10 +487,12 @@ __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, i
 // The same for a normed input: the block first norms the (few) rows of the f32 residual stream into shared memory -- rms over the
 // row, times the norm weight, rounded to the compute type exactly as lp_rmsnorm_kernel does -- and then multiplies from there.
 // Every block repeats the norm (the rows are a few KB out of L2); a launch and a round trip through global memory go away.
+// ic.taps > 0 (decoding: one row per run): the normed row h becomes h + conv(h) before the rounding; every block reads the run's earlier
+// inputs, block 0 writes this position's (input_conv_row: no other block reads that ring entry).
 template <typename T, int EPI>
 __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restrict__ X, const int* __restrict__ gather, const float* __restrict__ nw,
                                                            float eps, const T* __restrict__ W, void* __restrict__ Y, int ldy, int R, int N, int K,
-                                                           float alpha, int center, T* __restrict__ hn_out) {
+                                                           float alpha, int center, T* __restrict__ hn_out, float2 act, InConv ic, StepMeta sm) {
     extern __shared__ __align__(16) uint8_t gn_smem[];
     T* xs = reinterpret_cast<T*>(gn_smem);            // [R][K]
     __shared__ float red[8];
@@ -521,8 +529,10 @@ __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restri
         }
         __syncthreads();
         const float inv = inv_s;
+        const InConvRow cr = input_conv_row(ic, sm, r, blockIdx.x == 0);
         for (int k = threadIdx.x; k < K; k += 256) {
-            const T v = from_f<T>((xr[k] - mean) * inv * nw[k]);
+            const float h = (xr[k] - mean) * inv * nw[k];
+            const T v = from_f<T>(ic.taps > 0 ? input_conv_step(ic, cr, K, k, h) : h);
             xs[(size_t)r * K + k] = v;
             if (hn_out && blockIdx.x == 0) hn_out[(size_t)r * K + k] = v;   // (a later kernel of the layer reads the normed rows too)
         }
@@ -551,7 +561,7 @@ __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restri
         for (int i = 0; i < GV_ROWS; i++) {
             if (i < nr) {
                 const float sum = wsum(acc[i]);
-                if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + n, alpha * sum);
+                if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + n, alpha * sum, act);
             }
         }
     }
@@ -1358,6 +1368,11 @@ __global__ void lp_transpose_heads_kernel(const T* __restrict__ in, T* __restric
     out[(size_t)h * a * b + (size_t)ib * a + ia] = in[i];
 }
 
+// x[r] += v
+__global__ void lp_add_vec_kernel(float* __restrict__ x, const float* __restrict__ v, int width) {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) x[(size_t)blockIdx.x * width + c] += v[c];
+}
+
 __global__ void lp_add_scalar_kernel(float* __restrict__ v, int n, float a) {
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i < n) v[i] += a;
@@ -1413,6 +1428,11 @@ struct LayerPlan {
     // parallel_ff: first column of the feed-forward's part ([gate | up], [up] or the router) in the layer's input projection
     int ff_off = -1;
     int up_router_rows = 0;      // rows of the router at the head of w_up (0 when the router sits in the layer's input projection)
+    // input convolutions of the two sublayers (ring_off: inside the run's state block), the xIELU numbers, the biases of the router's rows
+    InConv ic[2];
+    float2 act2 = float2{0.0f, 0.0f};
+    const float* router_bias = nullptr;
+    int lat_splits = 0;          // latent attention: the largest row count x splits of the decoding kernels (0: they do not take these sizes)
     // multi-stream layer form: [in | out | mix] of the two sublayers (null: identity)
     const float *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
 };
@@ -1449,6 +1469,10 @@ struct LpModel {
     float* xs = nullptr;                // [rows][streams][width]: the residual copies of the multi-stream layer form
     void* cq = nullptr;                 // [rows][max_qrank] compute type: the normed query latent
     int max_qrank = 0;
+    void* xcat = nullptr;               // [rows][2 width] compute type: [x; x0] ahead of a pass of the repeated range (program.loop_in)
+    float *lat_o = nullptr, *lat_ml = nullptr;   // decoding latent attention: the splits' sums and their (maximum, sum)
+    size_t lat_o_floats = 0, lat_ml_floats = 0;
+    float* moe_shw = nullptr;           // [rows]: gate of the always-on expert
     int *moe_sel = nullptr, *moe_pos = nullptr, *moe_seg = nullptr;   // chosen experts per row; row of (token, choice) in expert order; {first, rows} per expert
     void* moe_xp = nullptr;             // the tokens' rows gathered in expert order, compute type
     float* moe_yp = nullptr;            // the experts' outputs in the same order
@@ -1481,6 +1505,8 @@ struct LpModel {
     uint64_t scratch_epoch = 1;
     bool use_graph = true;
     int tc_min_rows = 17;
+    int conv_fuse_rows = 1;      // B200_LP_CONV_FUSE_ROWS: decode steps of so many rows norm and convolve inside the projection
+    bool use_lat_split = true;   // B200_LP_LAT_SPLIT=0: decoding latent attention in the many-row kernels
     int* tc_err = nullptr;
     int* h_tc_err = nullptr;
     unsigned* tail_counter = nullptr;   // arrival counter of rows_tail (zero between kernels)
@@ -1543,7 +1569,7 @@ bool is_matrix_name(const std::string& n) {
     // vectors) is kept in f32
     if (n == "embed" || n == "head") return true;
     static const char* suf[] = {".q", ".k", ".v", ".g", ".o", ".i", ".f", ".a", ".b", ".up", ".down", ".gate", ".router",
-                                ".dq", ".uq", ".dkv", ".uk", ".uv", ".in", ".z", ".x"};
+                                ".dq", ".uq", ".dkv", ".uk", ".uv", ".in", ".z", ".x", ".sg"};
     for (const char* s : suf) {
         const size_t L = strlen(s);
         if (n.size() > L && n.compare(n.size() - L, L, s) == 0) return true;
@@ -1576,7 +1602,7 @@ void launch(LpModel* m, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t sm
 // The tensor-core GEMM takes bf16 operands whose rows are 16-byte aligned (K and the row pitches multiples of 8).
 template <int TN>
 bool tc_launch(LpModel* m, const bf16* x, int ldx, const bf16* w, int ldw, int N, int K, void* Y, int ldy, int R, float alpha, int epi, const int* seg,
-               int groups, size_t wz, ZStride zs, const float* bias) {
+               int groups, size_t wz, ZStride zs, const float* bias, float2 act) {
     const size_t smem = (size_t)TC_STAGES * (TC_M + TN) * 128 + 1024;
     static bool once[EPI_COUNT][64] = {};
     int dev = 0;
@@ -1594,24 +1620,25 @@ bool tc_launch(LpModel* m, const bf16* x, int ldx, const bf16* w, int ldw, int N
 #define LP_TC(E)                                                                                                                       \
     do {                                                                                                                               \
         if (!prep(lp_gemm_tc_kernel<TN, E>, E)) return false;                                                                          \
-        launch(m, lp_gemm_tc_kernel<TN, E>, grid, block, smem, x, ldx, w, ldw, Y, ldy, R, N, K, alpha, m->tc_err, seg, wz, zs, bias);  \
+        launch(m, lp_gemm_tc_kernel<TN, E>, grid, block, smem, x, ldx, w, ldw, Y, ldy, R, N, K, alpha, m->tc_err, seg, wz, zs, bias, act);  \
     } while (0)
     if (epi == EPI_STORE) LP_TC(EPI_STORE);
     else if (epi == EPI_ADD) LP_TC(EPI_ADD);
     else if (epi == EPI_GELU) LP_TC(EPI_GELU);
+    else if (epi == EPI_XIELU) LP_TC(EPI_XIELU);
     else LP_TC(EPI_RELU2);
 #undef LP_TC
     return true;
 }
 bool tc_gemm(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, int K, void* Y, int ldy, int R, float alpha, int epi, const int* seg,
-             int groups, size_t wz, ZStride zs, const float* bias) {
+             int groups, size_t wz, ZStride zs, const float* bias, float2 act) {
     if (m->f32 || !m->use_tc || R < m->tc_min_rows) return false;
     if (K % 8 || ldx % 8 || ldw % 8 || wz % 8 || zs.x % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return false;
     const bf16* x = (const bf16*)X;
     const bf16* w = (const bf16*)W;
-    if (R <= 64) return tc_launch<64>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias);
-    if (R <= 128) return tc_launch<128>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias);   // (wider token tiles move fewer operand bytes per FLOP: measured 2.5x on a 2048 x 8192 x 2048 product even at 128 CTAs)
-    return tc_launch<256>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias);
+    if (R <= 64) return tc_launch<64>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias, act);
+    if (R <= 128) return tc_launch<128>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias, act);   // (wider token tiles move fewer operand bytes per FLOP: measured 2.5x on a 2048 x 8192 x 2048 product even at 128 CTAs)
+    return tc_launch<256>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias, act);
 }
 
 // Y = epi(alpha X W^T): rows of the step against a [N][K] matrix in the compute type.  Without `seg`, groups > 1 batches the product
@@ -1619,7 +1646,8 @@ bool tc_gemm(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, 
 // [z zs.y, z zs.y + N) of Y.
 template <typename T>
 void gemm_t(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, int K, void* Y, int ldy, int R, float alpha, int epi, const int* seg = nullptr,
-            int groups = 1, size_t wz = 0, const RowsTail* tail = nullptr, ZStride zs = ZStride{0, 0}, const float* bias = nullptr) {
+            int groups = 1, size_t wz = 0, const RowsTail* tail = nullptr, ZStride zs = ZStride{0, 0}, const float* bias = nullptr,
+            float2 act = float2{0.0f, 0.0f}) {
     const T* x = (const T*)X;
     const T* w = (const T*)W;
     if (R <= 2 * GV_ROWS && !seg) {
@@ -1635,28 +1663,30 @@ void gemm_t(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, i
         const size_t smem = stage ? xbytes : 0;
         const RowsTail tl = tail ? *tail : RowsTail{};
         const int nh = heads ? N : 0;
-#define LP_GV(E) launch(m, lp_gemv_kernel<T, E>, grid, block, smem, x, ldx, w, ldw, Y, ldy, R, Nall, K, alpha, vec_ok, stage, tl, nh, zs, bias)
+#define LP_GV(E) launch(m, lp_gemv_kernel<T, E>, grid, block, smem, x, ldx, w, ldw, Y, ldy, R, Nall, K, alpha, vec_ok, stage, tl, nh, zs, bias, act)
         if (epi == EPI_STORE) LP_GV(EPI_STORE);
         else if (epi == EPI_ADD) LP_GV(EPI_ADD);
         else if (epi == EPI_GELU) LP_GV(EPI_GELU);
+        else if (epi == EPI_XIELU) LP_GV(EPI_XIELU);
         else LP_GV(EPI_RELU2);
 #undef LP_GV
         return;
     }
-    if (tc_gemm(m, X, ldx, W, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias)) return;
+    if (tc_gemm(m, X, ldx, W, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias, act)) return;
     dim3 grid((N + GB - 1) / GB, (R + GB - 1) / GB, groups), block(256);
-#define LP_GM(E) launch(m, lp_gemm_kernel<T, E>, grid, block, 0, x, ldx, w, ldw, Y, ldy, R, N, K, alpha, seg, wz, zs, bias)
+#define LP_GM(E) launch(m, lp_gemm_kernel<T, E>, grid, block, 0, x, ldx, w, ldw, Y, ldy, R, N, K, alpha, seg, wz, zs, bias, act)
     if (epi == EPI_STORE) LP_GM(EPI_STORE);
     else if (epi == EPI_ADD) LP_GM(EPI_ADD);
     else if (epi == EPI_GELU) LP_GM(EPI_GELU);
+    else if (epi == EPI_XIELU) LP_GM(EPI_XIELU);
     else LP_GM(EPI_RELU2);
 #undef LP_GM
 }
 // tail: few rows only (the caller has checked R): the last block goes on with rows_tail
 void gemm(LpModel* m, const void* X, int ldx, const void* W, int N, int K, void* Y, int ldy, int R, float alpha, int epi, const RowsTail* tail = nullptr,
-          const float* bias = nullptr) {
-    if (m->f32) gemm_t<float>(m, X, ldx, W, K, N, K, Y, ldy, R, alpha, epi, nullptr, 1, 0, tail, ZStride{0, 0}, bias);
-    else gemm_t<bf16>(m, X, ldx, W, K, N, K, Y, ldy, R, alpha, epi, nullptr, 1, 0, tail, ZStride{0, 0}, bias);
+          const float* bias = nullptr, float2 act = float2{0.0f, 0.0f}) {
+    if (m->f32) gemm_t<float>(m, X, ldx, W, K, N, K, Y, ldy, R, alpha, epi, nullptr, 1, 0, tail, ZStride{0, 0}, bias, act);
+    else gemm_t<bf16>(m, X, ldx, W, K, N, K, Y, ldy, R, alpha, epi, nullptr, 1, 0, tail, ZStride{0, 0}, bias, act);
 }
 // `groups` products in one launch (grid.z): group g multiplies rows [seg[2g], seg[2g] + seg[2g + 1]) of X -- the counts live on the
 // device, R is their upper bound -- with the matrix at Wm + g * zs elements, whose rows are ldw apart (contiguous matrices: ldw = K,
@@ -1689,7 +1719,7 @@ void rmsnorm(LpModel* m, float* x, const float* add, const float* w, void* out, 
 // written back into the stream).
 template <typename T>
 bool gemv_norm_t(LpModel* m, const float* x, const int* gather, const float* nw, const void* W, int N, int K, void* Y, int ldy, int R, float alpha,
-                 int epi, void* hn_out) {
+                 int epi, void* hn_out, float2 act, const InConv& ic, const StepMeta& sm) {
     constexpr int VN = Vec8<T>::N;
     const size_t smem = (size_t)R * K * sizeof(T);
     if (R > 2 * GV_ROWS || K % VN || ((uintptr_t)W & 15) || smem > 96 * 1024) return false;
@@ -1709,24 +1739,30 @@ bool gemv_norm_t(LpModel* m, const float* x, const int* gather, const float* nw,
     const T* w = (const T*)W;
     if (epi == EPI_STORE) {
         if (!prep(lp_gemv_norm_kernel<T, EPI_STORE>, 0)) return false;
-        launch(m, lp_gemv_norm_kernel<T, EPI_STORE>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out);
+        launch(m, lp_gemv_norm_kernel<T, EPI_STORE>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm);
     } else if (epi == EPI_RELU2) {
         if (!prep(lp_gemv_norm_kernel<T, EPI_RELU2>, 2)) return false;
-        launch(m, lp_gemv_norm_kernel<T, EPI_RELU2>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out);
+        launch(m, lp_gemv_norm_kernel<T, EPI_RELU2>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm);
+    } else if (epi == EPI_XIELU) {
+        if (!prep(lp_gemv_norm_kernel<T, EPI_XIELU>, 4)) return false;
+        launch(m, lp_gemv_norm_kernel<T, EPI_XIELU>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm);
     } else return false;
     return true;
 }
 // keep: the normed rows are also wanted in `scratch` afterwards (the fused kernel then writes them out as well)
 void norm_gemm(LpModel* m, float* x, const float* add, const int* gather, const float* nw, void* scratch, const void* W, int N, void* Y, int ldy,
-               int R, float alpha, int epi, bool keep = false) {
+               int R, float alpha, int epi, bool keep = false, float2 act = float2{0.0f, 0.0f}) {
     const int K = m->p.width;
     if (!add && m->use_fuse) {
         void* hn_out = keep ? scratch : nullptr;
-        if (m->f32 ? gemv_norm_t<float>(m, x, gather, nw, W, N, K, Y, ldy, R, alpha, epi, hn_out) : gemv_norm_t<bf16>(m, x, gather, nw, W, N, K, Y, ldy, R, alpha, epi, hn_out))
+        const InConv ic{};
+        const StepMeta sm{};
+        if (m->f32 ? gemv_norm_t<float>(m, x, gather, nw, W, N, K, Y, ldy, R, alpha, epi, hn_out, act, ic, sm)
+                   : gemv_norm_t<bf16>(m, x, gather, nw, W, N, K, Y, ldy, R, alpha, epi, hn_out, act, ic, sm))
             return;
     }
     rmsnorm(m, x, add, nw, scratch, gather, R);
-    gemm(m, scratch, K, W, N, K, Y, ldy, R, alpha, epi);
+    gemm(m, scratch, K, W, N, K, Y, ldy, R, alpha, epi, nullptr, nullptr, act);
 }
 
 int pick_dmax(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
@@ -1748,6 +1784,11 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
     if (p.streams < 0 || p.streams > ST_MAX) return bad("streams must be 0 .. " + std::to_string(ST_MAX));
     if (p.streams > 0 && (p.post_norm || looped)) return bad("the multi-stream form takes neither the norm after the sum nor a repeated range");
     if (p.parallel_ff && (p.post_norm || p.streams > 0)) return bad("parallel_ff belongs to the norm-first form with one residual stream");
+    if (p.in_conv < 0 || p.in_conv > 64) return bad("in_conv must be 0 .. 64 taps");
+    if (p.in_conv > 0 && (p.post_norm || p.streams > 0 || p.parallel_ff || p.norm_kind != B200_NORM_RMS))
+        return bad("in_conv belongs to the norm-first form with one residual stream, two norms per layer and RMS norms");
+    if (p.loop_in && (!looped || p.post_norm || p.streams > 0)) return bad("loop_in needs a repeated range in the norm-first form with one residual stream");
+    if (p.embed_norm && (p.post_norm || p.norm_kind != B200_NORM_RMS)) return bad("embed_norm belongs to the norm-first forms with RMS norms");
     for (int i = 0; i < p.n_layers; i++) {
         const b200_layer_desc& L = layers[i];
         const std::string at = "layer " + std::to_string(i) + ": ";
@@ -1800,13 +1841,13 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
             }
         } else if (L.mixer == B200_MIX_LATENT_ATTN) {
             const b200_latent_attn_desc& a = L.latent;
-            if (a.heads <= 0 || a.dim <= 0 || a.rot_dim < 0 || a.vdim <= 0 || a.q_rank <= 0 || a.kv_rank <= 0) return bad(at + "bad latent-attention sizes");
+            if (a.heads <= 0 || a.dim <= 0 || a.rot_dim < 0 || a.vdim <= 0 || a.q_rank < 0 || a.kv_rank <= 0) return bad(at + "bad latent-attention sizes");
             if (a.kv_rank > 32 * ATT_ACC) return bad(at + "latent size above " + std::to_string(32 * ATT_ACC));
             if (a.mask_size < 0) return bad(at + "negative window");
             if (a.rot.dims < 0 || a.rot.dims > a.rot_dim || (a.rot.dims & 1) || (a.rot.dims > 0 && !(a.rot.base > 0.0f))) return bad(at + "bad rotary sizes");
             if (a.rot.yarn_factor < 0.0f || (a.rot.yarn_factor > 0.0f && !(a.rot.yarn_original > 0.0f && a.rot.yarn_fast > 0.0f && a.rot.yarn_slow > 0.0f)))
                 return bad(at + "bad rotary scaling");
-            if (a.out_gate != B200_GATE_NONE && a.out_gate != B200_GATE_CHANNEL) return bad(at + "latent attention takes no gate or one per value channel");
+            if (a.out_gate < B200_GATE_NONE || a.out_gate > B200_GATE_HEAD) return bad(at + "unknown output gate");
             if (a.kv_from >= 0) {
                 if (a.kv_from >= i || layers[a.kv_from].mixer != B200_MIX_LATENT_ATTN || layers[a.kv_from].latent.kv_from >= 0)
                     return bad(at + "kv_from must name an earlier latent-attention layer with cache rows of its own");
@@ -1823,14 +1864,17 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
         if (L.ff_kind == B200_FF_MOE) {
             const b200_moe_desc& e = L.moe;
             if (e.experts <= 0 || e.top <= 0 || e.top > e.experts || e.expert_ff <= 0 || e.shared_ff < 0) return bad(at + "bad mixture-of-experts sizes");
-            if (e.act < B200_ACT_RELU2 || e.act > B200_ACT_SILU_GLU || e.route < B200_ROUTE_TOP_SOFTMAX || e.route > B200_ROUTE_SIGMOID_TOP)
+            if (e.act < B200_ACT_RELU2 || e.act > B200_ACT_CLAMPED_GLU || e.route < B200_ROUTE_TOP_SOFTMAX || e.route > B200_ROUTE_SIGMOID_TOP)
                 return bad(at + "unknown expert activation or routing rule");
-            if (e.act == B200_ACT_SILU_GLU && e.shared_ff > 0) return bad(at + "gated experts take no always-on expert");
+            if (e.act == B200_ACT_CLAMPED_GLU && (!(e.limit > 0.0f) || (e.shared_ff > 0 && !(e.shared_limit > 0.0f)))) return bad(at + "clamped experts need positive limits");
+            if (e.shared_gate && e.shared_ff <= 0) return bad(at + "a gate without an always-on expert");
+            if (p.parallel_ff && (e.router_bias || e.shared_gate)) return bad(at + "parallel_ff takes no router bias and no gated always-on expert");
             if (e.weight_input && p.streams > 0) return bad(at + "weights on the experts' inputs are not available in the multi-stream form");
         } else if (L.ff_kind == B200_FF_CLAMPED_GLU) {
             if (L.ff > 0 && !(L.ff_limit > 0.0f)) return bad(at + "the clamped feed-forward needs a positive limit");
-        } else if (L.ff_kind != B200_FF_RELU2 && L.ff_kind != B200_FF_GATED_GELU) return bad(at + "unknown feed-forward kind");
+        } else if (L.ff_kind != B200_FF_RELU2 && L.ff_kind != B200_FF_GATED_GELU && L.ff_kind != B200_FF_XIELU) return bad(at + "unknown feed-forward kind");
         if (L.ff < 0) return bad(at + "negative feed-forward width");
+        if (L.ff_kind == B200_FF_XIELU && p.parallel_ff) return bad(at + "parallel_ff takes no xIELU feed-forward");
     }
     LpModel* m = new LpModel();
     m->p = p;
@@ -1866,6 +1910,10 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
         if (e && *e) m->use_stream_tail = atoi(e) != 0;
         e = getenv("B200_LP_GRAPH");
         if (e && *e) m->use_graph = atoi(e) != 0;
+        e = getenv("B200_LP_CONV_FUSE_ROWS");
+        if (e && *e) m->conv_fuse_rows = atoi(e);
+        e = getenv("B200_LP_LAT_SPLIT");
+        if (e && *e) m->use_lat_split = atoi(e) != 0;
         e = getenv("B200_LP_TC_MIN_ROWS");
         if (e && *e) m->tc_min_rows = std::max(1, atoi(e));
     }
@@ -1988,6 +2036,32 @@ int need_mat(LpModel* m, const std::string& name, uint64_t rows, uint64_t cols, 
 }
 }  // namespace
 
+namespace {
+// program.norm_scalar: the one number of a norm spread over the width, so that every kernel sees a weight per coordinate
+int spread_norm(LpModel* m, const std::string& name, uint64_t n, std::string* err) {
+    auto it = m->tensors.find(name);
+    if (it == m->tensors.end()) return B200_OK;
+    Tensor& t = it->second;
+    if (t.rows * t.cols != 1) return lp_fail(err, B200_ERR_SHAPE_MISMATCH, name + ": expected one number, got " + std::to_string(t.rows * t.cols));
+    float* d = nullptr;
+    LCU_ALLOC(cudaMalloc((void**)&d, up16(n * 4)));
+    lp_fill_kernel<<<(unsigned)((n + 255) / 256), 256>>>(d, (const float*)t.d, (int)n);
+    LCU(cudaDeviceSynchronize());
+    cudaFree(t.d);
+    t.d = d;
+    t.cols = n;
+    t.bytes = n * 4;
+    return B200_OK;
+}
+double softplus_host(double z) { return std::max(z, 0.0) + std::log1p(std::exp(-std::fabs(z))); }
+
+// Splits of the decoding attention's keys for R rows: about two blocks per SM
+int latent_splits(int R, int heads) {
+    const int blocks = R * ((heads + LS_HEADS - 1) / LS_HEADS);
+    return std::max(1, std::min(64, 2 * 148 / blocks));
+}
+}  // namespace
+
 int lp_finalize(LpModel* m, std::string* err) {
     if (m->finalized) return B200_OK;
     LCU(cudaSetDevice(m->device));
@@ -2000,7 +2074,16 @@ int lp_finalize(LpModel* m, std::string* err) {
     m->weight_bytes -= find(m, "embed")->bytes - W * elt(m);   // one row per token
     if ((rc = need_mat(m, "head", p.vocab, W, &dummy, err))) return rc;
     const float* fv;
+    if (p.norm_scalar) {
+        std::vector<std::string> nm = {"final.norm", "embed.norm"};
+        for (int li = 0; li < p.n_layers; li++)
+            for (const char* s2 : {".norm1", ".norm2"}) nm.push_back("l" + std::to_string(li) + s2);
+        for (const std::string& n : nm)
+            if ((rc = spread_norm(m, n, W, err))) return rc;
+    }
     if ((rc = need_vec(m, "final.norm", W, &fv, err))) return rc;
+    if (p.embed_norm && (rc = need_vec(m, "embed.norm", W, &fv, err))) return rc;
+    if (p.loop_in && (rc = need_mat(m, "loop.in", W, 2 * W, &dummy, err))) return rc;
     if (p.loop_stop > p.loop_start && (rc = need_vec(m, "loop.step", (uint64_t)p.loop_times * W, &fv, err))) return rc;
     for (int li = 0; li < p.n_layers; li++) {
         LayerPlan& L = m->plan[li];
@@ -2193,18 +2276,19 @@ int lp_finalize(LpModel* m, std::string* err) {
             const std::string x = pre + "mix.";
             const bool own = a.kv_from < 0;
             const uint64_t H = a.heads, D = (uint64_t)a.kv_rank + a.rot_dim, per = (uint64_t)a.dim + a.rot_dim;
-            std::vector<std::string> names = {x + "dq"};
-            std::vector<uint64_t> rows = {(uint64_t)a.q_rank};
+            const bool direct = a.q_rank == 0;      // no query latent: the input projection gives the queries themselves
+            std::vector<std::string> names = {x + (direct ? "q" : "dq")};
+            std::vector<uint64_t> rows = {direct ? H * per : (uint64_t)a.q_rank};
             if (own) { names.push_back(x + "dkv"); rows.push_back(D); }
-            if (a.out_gate) { names.push_back(x + "g"); rows.push_back(H * a.vdim); }
+            if (a.out_gate) { names.push_back(x + "g"); rows.push_back(a.out_gate == B200_GATE_HEAD ? H : H * a.vdim); }
             if ((rc = fuse_rows(m, names, rows, W, &L.w_in, &L.n_in, &off, err))) return rc;
             LatentGeom& g = L.lg;
             g.H = a.heads; g.dim = a.dim; g.rot_dim = a.rot_dim; g.vdim = a.vdim; g.q_rank = a.q_rank; g.kv_rank = a.kv_rank;
-            g.rot_n = a.rot.dims; g.eps = p.norm_eps; g.cap = p.max_seq_len;
+            g.pairs = a.rot_pairs; g.gate = a.out_gate; g.rot_n = a.rot.dims; g.eps = p.norm_eps; g.cap = p.max_seq_len;
             g.q_off = off[0]; g.kv_off = own ? off[1] : -1; g.g_off = a.out_gate ? off[own ? 2 : 1] : 0;
-            if ((rc = need_vec(m, x + "dq.norm", a.q_rank, &L.dq_norm, err))) return rc;
+            if (!direct && (rc = need_vec(m, x + "dq.norm", a.q_rank, &L.dq_norm, err))) return rc;
             if (own && (rc = need_vec(m, x + "dkv.norm", a.kv_rank, &L.dkv_norm, err))) return rc;
-            if ((rc = need_mat(m, x + "uq", H * per, a.q_rank, &L.w_uq, err))) return rc;
+            if (!direct && (rc = need_mat(m, x + "uq", H * per, a.q_rank, &L.w_uq, err))) return rc;
             if ((rc = need_mat(m, x + "uv", H * a.vdim, a.kv_rank, &L.w_uv, err))) return rc;
             if ((rc = need_mat(m, x + "o", W, H * a.vdim, &L.wo, err))) return rc;
             {   // W_uk [H dim][kv_rank] -> per head [kv_rank][dim]: the matrix that carries a head's plain query into the latent
@@ -2241,6 +2325,14 @@ int lp_finalize(LpModel* m, std::string* err) {
             m->max_q = std::max(m->max_q, (int)(H * D));
             m->max_o = std::max(m->max_o, (int)(H * std::max(per, (uint64_t)a.vdim)));
             m->max_qrank = std::max(m->max_qrank, a.q_rank);
+            // decoding kernels: 16-byte loads of cached rows and weights, the rows in shared memory, two key tiles too
+            const int vn = m->f32 ? 4 : 8;
+            const size_t part = (size_t)2 * GV_ROWS * (std::max(a.dim, a.kv_rank) + std::max(64, a.rot.dims)) * 4;
+            if (D % 4 == 0 && a.kv_rank % vn == 0 && a.dim % vn == 0 && latent_split_smem((int)D) <= 200 * 1024 && part <= 96 * 1024) {
+                for (int r = 1; r <= 2 * GV_ROWS; r++) L.lat_splits = std::max(L.lat_splits, r * latent_splits(r, a.heads));
+                m->lat_o_floats = std::max(m->lat_o_floats, (size_t)L.lat_splits * a.heads * a.kv_rank);
+                m->lat_ml_floats = std::max(m->lat_ml_floats, (size_t)L.lat_splits * a.heads * 2);
+            }
         } else if (L.d.mixer == B200_MIX_STATE_SPACE) {
             const b200_state_space_desc& g = L.d.ssd;
             const std::string x = pre + "mix.";
@@ -2297,6 +2389,15 @@ int lp_finalize(LpModel* m, std::string* err) {
             m->max_conv = std::max(m->max_conv, d.C);
         }
         m->max_in = std::max(m->max_in, L.n_in);
+        if (p.in_conv > 0) {   // the rings of the two sublayers' inputs behind the mixer's own state
+            const bool ff = L.d.ff_kind == B200_FF_MOE || L.d.ff > 0;
+            for (int q = 0; q < (ff ? 2 : 1); q++) {
+                L.ic[q].taps = p.in_conv;
+                if ((rc = need_vec(m, pre + "canon" + std::to_string(q + 1), W * p.in_conv, &L.ic[q].w, err))) return rc;
+                L.ic[q].ring_off = L.rec_bytes;
+                if (p.in_conv > 1) L.rec_bytes += up16((size_t)p.in_conv * W * 4);
+            }
+        }
         if (p.streams > 0) {   // the stream weights of the two sublayers; a layer without them mixes nothing
             for (int q = 0; q < 2; q++) {
                 const std::string hc = pre + "hc" + std::to_string(q + 1) + ".";
@@ -2330,13 +2431,25 @@ int lp_finalize(LpModel* m, std::string* err) {
         if (L.d.ff_kind == B200_FF_MOE) {
             const b200_moe_desc& e = L.d.moe;
             if (!par && (rc = need_vec(m, pre + "norm2", W, &L.norm2, err))) return rc;
-            const bool glu = e.act == B200_ACT_SILU_GLU;
+            const bool glu = act_gated(e.act);
             const int per = glu ? 2 * e.expert_ff : e.expert_ff;   // rows of one expert's up matrix ([gate | up] when gated)
             if (par && (rc = join_input({pre + "mlp.router"}, {(uint64_t)e.experts}))) return rc;
             std::vector<std::string> names, down;
             std::vector<uint64_t> rows;
             if (!par) { names.push_back(pre + "mlp.router"); rows.push_back((uint64_t)e.experts); }
-            L.up_router_rows = par ? 0 : e.experts;
+            if (e.shared_gate) { names.push_back(pre + "mlp.shared.sg"); rows.push_back(1); }   // one more row of the router
+            L.up_router_rows = par ? 0 : e.experts + (e.shared_gate ? 1 : 0);
+            if (e.router_bias) {
+                const float* rb;
+                if ((rc = need_vec(m, pre + "mlp.router.b", e.experts, &rb, err))) return rc;
+                Tensor t;
+                t.rows = 1; t.cols = L.up_router_rows; t.bytes = t.cols * 4;
+                LCU_ALLOC(cudaMalloc(&t.d, up16(t.bytes)));
+                LCU(cudaMemset(t.d, 0, t.bytes));
+                LCU(cudaMemcpy(t.d, rb, (size_t)e.experts * 4, cudaMemcpyDeviceToDevice));
+                m->tensors[pre + "mlp.router.b_cat"] = t;
+                L.router_bias = (const float*)t.d;
+            }
             for (int i = 0; i < e.experts; i++) {
                 if (glu) { names.push_back(pre + "mlp.e" + std::to_string(i) + ".gate"); rows.push_back(e.expert_ff); }
                 names.push_back(pre + "mlp.e" + std::to_string(i) + ".up");
@@ -2344,6 +2457,7 @@ int lp_finalize(LpModel* m, std::string* err) {
                 down.push_back(pre + "mlp.e" + std::to_string(i) + ".down");
             }
             if (e.shared_ff > 0) {
+                if (glu) { names.push_back(pre + "mlp.shared.gate"); rows.push_back(e.shared_ff); }
                 names.push_back(pre + "mlp.shared.up");
                 rows.push_back(e.shared_ff);
                 down.push_back(pre + "mlp.shared.down");
@@ -2395,6 +2509,13 @@ int lp_finalize(LpModel* m, std::string* err) {
                 L.n_up = L.d.ff;
             }
             if ((rc = need_mat(m, pre + "mlp.down", W, L.d.ff, &L.w_down, err))) return rc;
+            if (L.d.ff_kind == B200_FF_XIELU) {
+                const float* pq;
+                float h[2];
+                if ((rc = need_vec(m, pre + "mlp.act", 2, &pq, err))) return rc;
+                LCU(cudaMemcpy(h, pq, 8, cudaMemcpyDeviceToHost));
+                L.act2 = float2{(float)softplus_host(h[0]), (float)(0.5 + softplus_host(h[1]))};
+            }
             L.k_down = L.d.ff;
             m->max_act = std::max(m->max_act, L.d.ff);
         } else if (p.post_norm && find(m, pre + "norm2")) {   // a layer without feed-forward whose file still holds the second norm
@@ -2409,8 +2530,26 @@ int lp_finalize(LpModel* m, std::string* err) {
         if (need > 200 * 1024) return lp_fail(err, B200_ERR_UNSUPPORTED, "softmax mixer: q, k and v of one token exceed 200 KB of shared memory");
         if (need > 32 * 1024) LCU(cudaFuncSetAttribute(lp_attn_prep2_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)need));
     }
+    if (m->lat_o_floats > 0) {
+        LCU_ALLOC(cudaMalloc((void**)&m->lat_o, up16(m->lat_o_floats * 4)));
+        LCU_ALLOC(cudaMalloc((void**)&m->lat_ml, up16(m->lat_ml_floats * 4)));
+        const int sb = 200 * 1024, pb = 96 * 1024;
+        LCU(cudaFuncSetAttribute(lp_latent_split_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
+        LCU(cudaFuncSetAttribute(lp_latent_split_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
+        LCU(cudaFuncSetAttribute(lp_latent_split_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
+        LCU(cudaFuncSetAttribute(lp_latent_absorb_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, pb));
+        LCU(cudaFuncSetAttribute(lp_latent_absorb_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, pb));
+        LCU(cudaFuncSetAttribute(lp_latent_merge_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, pb));
+        LCU(cudaFuncSetAttribute(lp_latent_merge_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, pb));
+    }
+    if (p.in_conv > 0 && (size_t)p.width * elt(m) > 40 * 1024) {
+        if ((size_t)p.width * elt(m) > 200 * 1024) return lp_fail(err, B200_ERR_UNSUPPORTED, "input convolution: a row exceeds 200 KB of shared memory");
+        LCU(cudaFuncSetAttribute(lp_norm_conv_step_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        LCU(cudaFuncSetAttribute(lp_norm_conv_step_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    }
     if (p.norm_weight_offset != 0.0f) {   // norm weights stored around zero: (offset + w) once, in f32
         std::vector<std::string> nm = {"final.norm"};
+        if (p.embed_norm) nm.push_back("embed.norm");
         for (int li = 0; li < p.n_layers; li++)
             for (const char* s2 : {".norm1", ".norm2"}) nm.push_back("l" + std::to_string(li) + s2);
         for (const std::string& n : nm) {
@@ -2481,7 +2620,8 @@ void lp_destroy(LpModel* m) {
     for (SlotMem& s : m->pool) { cudaFree(s.kv); cudaFree(s.rec); }
     for (void* ptr : {(void*)m->inv_freq, (void*)m->d_meta, (void*)m->x, (void*)m->P, (void*)m->qbuf, (void*)m->O, (void*)m->conv, (void*)m->logits,
                       m->hn, m->act_a, m->hw, (void*)m->pick, (void*)m->taps, (void*)m->glin_carry, (void*)m->y, (void*)m->vsrc, (void*)m->moe_w, (void*)m->moe_selw,
-                      (void*)m->moe_sel, (void*)m->moe_pos, (void*)m->moe_seg, m->moe_xp, (void*)m->moe_yp, (void*)m->xs, m->cq, (void*)m->vrot})
+                      (void*)m->moe_sel, (void*)m->moe_pos, (void*)m->moe_seg, m->moe_xp, (void*)m->moe_yp, (void*)m->xs, m->cq, (void*)m->vrot, m->xcat,
+                      (void*)m->lat_o, (void*)m->lat_ml, (void*)m->moe_shw})
         cudaFree(ptr);
     if (m->h_meta) cudaFreeHost(m->h_meta);
     if (m->h_logits) cudaFreeHost(m->h_logits);
@@ -2551,8 +2691,10 @@ int ensure_scratch(LpModel* m, int R, int n_runs, int n_want, std::string* err) 
         if (m->max_vrot > 0 && (rc = grow(&m->vrot, (size_t)cap * m->max_vrot * 4, err))) return rc;
         if (m->p.streams > 0 && (rc = grow(&m->xs, (size_t)cap * m->p.streams * W * 4, err))) return rc;
         if (m->max_qrank > 0 && (rc = grow(&m->cq, (size_t)cap * m->max_qrank * es, err))) return rc;
+        if (m->p.loop_in && (rc = grow(&m->xcat, (size_t)cap * 2 * W * es, err))) return rc;
         if (m->max_vsrc > 0 && (rc = grow(&m->vsrc, (size_t)cap * m->max_vsrc * 4, err))) return rc;
         if (m->max_experts > 0) {
+            if ((rc = grow(&m->moe_shw, (size_t)cap * 4, err))) return rc;
             if ((rc = grow(&m->moe_w, (size_t)cap * m->max_experts * 4, err))) return rc;
             if ((rc = grow(&m->moe_selw, (size_t)cap * m->max_top * 4, err))) return rc;
             if ((rc = grow(&m->moe_sel, (size_t)cap * m->max_top * 4, err))) return rc;
@@ -2643,6 +2785,11 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
     // embedding
     if (m->f32) launch(m, lp_embed_kernel<float>, dim3(R), dim3(128), 0, sm, (const float*)find(m, "embed")->d, m->inv_freq, m->x, W, p.embed_scale, p.pos_sinusoid);
     else launch(m, lp_embed_kernel<bf16>, dim3(R), dim3(128), 0, sm, (const bf16*)find(m, "embed")->d, m->inv_freq, m->x, W, p.embed_scale, p.pos_sinusoid);
+    if (p.embed_norm || p.loop_in) {   // the embedding's norm; with loop_in its copy x0 for the passes of the repeated range
+        const float* g = p.embed_norm ? (const float*)find(m, "embed.norm")->d : nullptr;
+        if (m->f32) launch(m, lp_embed_norm_kernel<float>, dim3(R), dim3(256), 0, m->x, g, W, p.norm_eps, p.embed_norm, (float*)m->xcat);
+        else launch(m, lp_embed_norm_kernel<bf16>, dim3(R), dim3(256), 0, m->x, g, W, p.norm_eps, p.embed_norm, (bf16*)m->xcat);
+    }
     // The two layer forms.  Norm first: a sublayer reads norm(x) and its output projection adds into x.  Norm after the sum
     // (post_norm): a sublayer reads x itself -- m->hn holds x in the compute type -- its output projection goes to m->y, and
     // lp_postnorm_kernel makes x <- norm(alpha x + y) and the next copy.
@@ -2707,12 +2854,49 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         if (m->f32) launch(m, lp_postnorm_kernel<float>, dim3(R), dim3(256), 0, m->x, y, w, (float*)m->hn, W, p.residual_alpha, p.norm_eps);
         else launch(m, lp_postnorm_kernel<bf16>, dim3(R), dim3(256), 0, m->x, y, w, (bf16*)m->hn, W, p.residual_alpha, p.norm_eps);
     };
+    // What sublayer `sub` reads in a program with input convolutions, h + conv(h) with h = norm(x), in the compute type -> m->hn.  One
+    // token per run: one block per row, which also moves the ring on and, given `rt`, routes; longer runs: the ring after the readers.
+    const bool ring_step = max_len == 1 && m->use_fuse;
+    auto conv_in = [&](const InConv& ic0, const float* nw, const StepRoute& rt) {
+        InConv ic = ic0;
+        ic.ring_off += m->run_rec_off[cur_run];
+        if (ring_step) {
+            const size_t smem = rt.router ? (size_t)W * elt(m) : 0;
+            if (m->f32) launch(m, lp_norm_conv_step_kernel<float>, dim3(R), dim3(512), smem, sm, ic, (const float*)m->x, nw, W, p.norm_eps, (float*)m->hn, rt);
+            else launch(m, lp_norm_conv_step_kernel<bf16>, dim3(R), dim3(512), smem, sm, ic, (const float*)m->x, nw, W, p.norm_eps, (bf16*)m->hn, rt);
+            return;
+        }
+        const dim3 grid((R + NC_ROWS - 1) / NC_ROWS), block(256);
+        const size_t smem = (size_t)(NC_ROWS + ic.taps - 1) * 4;
+#define LP_NC(T, V, TP) launch(m, lp_norm_conv_rows_kernel<T, V, TP>, grid, block, smem, sm, ic, (const float*)m->x, nw, W, p.norm_eps, (T*)m->hn, R)
+#define LP_NC_T(T)                                                                                                      \
+        if (W % 4) LP_NC(T, 1, 0);                                                                                      \
+        else if (ic.taps == 2) LP_NC(T, 4, 2);                                                                          \
+        else if (ic.taps == 3) LP_NC(T, 4, 3);                                                                          \
+        else if (ic.taps == 4) LP_NC(T, 4, 4);                                                                          \
+        else LP_NC(T, 4, 0)
+        if (m->f32) { LP_NC_T(float); } else { LP_NC_T(bf16); }
+#undef LP_NC_T
+#undef LP_NC
+        if (ic.taps > 1) launch(m, lp_norm_conv_tail_kernel, dim3(n_runs, ic.taps - 1), dim3(256), 0, sm, ic, (const float*)m->x, nw, W, p.norm_eps);
+    };
     auto project_in = [&](const float* add, const float* nw, const void* Wm, int N, void* Y, int ldy, int epi) {
-        if (streams) {
+        const float2 act = cur->act2;
+        if (p.in_conv > 0) {
+            if (ring_step && R <= m->conv_fuse_rows) {   // the norm and the convolution inside the projection
+                InConv ic = cur->ic[sub];
+                ic.ring_off += m->run_rec_off[cur_run];
+                if (m->f32 ? gemv_norm_t<float>(m, m->x, nullptr, nw, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, act, ic, sm)
+                           : gemv_norm_t<bf16>(m, m->x, nullptr, nw, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, act, ic, sm))
+                    return;
+            }
+            conv_in(cur->ic[sub], nw, StepRoute{});
+            gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, nullptr, act);
+        } else if (streams) {
             boundary(cur->hc_in[sub], nw, nullptr);
-            gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi);
-        } else if (post) gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi);
-        else norm_gemm(m, m->x, add, nullptr, nw, m->hn, Wm, N, Y, ldy, R, 1.0f, epi, p.parallel_ff != 0);   // (parallel_ff: the experts read m->hn later)
+            gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, nullptr, act);
+        } else if (post) gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, nullptr, act);
+        else norm_gemm(m, m->x, add, nullptr, nw, m->hn, Wm, N, Y, ldy, R, 1.0f, epi, p.parallel_ff != 0, act);   // (parallel_ff: the experts read m->hn later)
     };
     // Few rows (decoding) in the norm-after-sum form: the kernel that writes m->y also does what follows it -- its last block norms the
     // rows and, when `moe` follows, computes the router's logits and choices (rows_tail) -- instead of two or three more launches.
@@ -2747,14 +2931,26 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
     for (size_t run = 0; run < m->runs.size(); run++) {
         LayerPlan& L = m->plan[m->runs[run]];
         const float* add = m->run_pass[run] >= 0 ? loop_step + (size_t)m->run_pass[run] * W : nullptr;
+        if (add && p.loop_in) {   // ahead of a pass: x <- loop.in [x; x0] + the pass's vector
+            const unsigned nb = (unsigned)(((size_t)R * W + 255) / 256);
+            if (m->f32) launch(m, lp_cast_rows_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->x, W, (float*)m->xcat, 2 * W, R);
+            else launch(m, lp_cast_rows_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->x, W, (bf16*)m->xcat, 2 * W, R);
+            gemm(m, m->xcat, 2 * W, find(m, "loop.in")->d, W, 2 * W, m->x, W, R, 1.0f, EPI_STORE, nullptr, add);
+            add = nullptr;
+        }
+        if (add && p.in_conv > 0) {   // (the input convolution reads the stream as it is)
+            launch(m, lp_add_vec_kernel, dim3(R), dim3(256), 0, m->x, add, W);
+            add = nullptr;
+        }
         // the few-row expert kernels (16-byte loads: sizes multiples of 8 / 4, the rows in shared memory)
         const bool moe_sel_ok = L.d.ff_kind == B200_FF_MOE && m->use_fuse && R <= 2 * GV_ROWS && W % (m->f32 ? 4 : 8) == 0 &&
                                 L.d.moe.expert_ff % (m->f32 ? 4 : 8) == 0 && L.d.moe.shared_ff % (m->f32 ? 4 : 8) == 0 && (size_t)R * W * elt(m) <= 40 * 1024;
-        const LayerPlan* moe_next = ((few || sfew) && moe_sel_ok) ? &L : nullptr;      // the mixer's output kernel also routes
+        // (the fused tails know neither a router bias nor the always-on expert's gate)
+        const LayerPlan* moe_next = ((few || sfew) && moe_sel_ok && !L.d.moe.router_bias && !L.d.moe.shared_gate) ? &L : nullptr;      // the mixer's output kernel also routes
         cur = &L;
         sub = 0;
         cur_run = run;
-        cur_moe_sel = moe_sel_ok;
+        cur_moe_sel = moe_sel_ok && !L.d.moe.router_bias && !L.d.moe.shared_gate;
         project_in(add, L.norm1, L.w_in, L.n_in, m->P, L.n_in, EPI_STORE);
         if (L.d.mixer == B200_MIX_SOFTMAX_ATTN || L.d.mixer == B200_MIX_ATTN_RECURRENT) {
             const bool dual = L.d.mixer == B200_MIX_ATTN_RECURRENT, weighted = dual && L.d.combine == B200_COMBINE_WEIGHTED;
@@ -2859,22 +3055,45 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             lg.cache_off = m->run_kv_off[L.kv_layer == m->runs[run] ? run : (size_t)L.kv_layer];
             const size_t csm = (size_t)lg.rot_n * 4;
             const int per = a.dim + a.rot_dim, D = a.kv_rank + a.rot_dim, nv = a.heads * a.vdim;
-            if (m->f32) launch(m, lp_latent_prep_kernel<float>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (float*)m->cq);
-            else launch(m, lp_latent_prep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (bf16*)m->cq);
-            gemm(m, m->cq, a.q_rank, L.w_uq, a.heads * per, a.q_rank, m->O, a.heads * per, R, 1.0f, EPI_STORE);
-            if (m->f32) launch(m, lp_latent_qprep_kernel<float>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->O, L.rot_freq, (float*)m->act_a, m->qbuf);
-            else launch(m, lp_latent_qprep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->O, L.rot_freq, (bf16*)m->act_a, m->qbuf);
-            gemm_heads(m, m->act_a, a.heads * a.dim, a.dim, L.w_ukT, a.heads, a.kv_rank, a.dim, m->qbuf, a.heads * D, D, R);
+            const bool direct = a.q_rank == 0, own = a.kv_from < 0;
+            // one token per run, few rows: absorb / split attention / merge (lp_latent_attn.cuh)
+            const bool split = m->use_fuse && m->use_lat_split && max_len == 1 && R <= 2 * GV_ROWS && L.lat_splits > 0;
+            if (!(split && direct)) {
+                if (m->f32) launch(m, lp_latent_prep_kernel<float>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (float*)m->cq, (float*)m->act_a, m->qbuf);
+                else launch(m, lp_latent_prep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (bf16*)m->cq, (bf16*)m->act_a, m->qbuf);
+            }
+            if (!direct) gemm(m, m->cq, a.q_rank, L.w_uq, a.heads * per, a.q_rank, m->O, a.heads * per, R, 1.0f, EPI_STORE);
             AttnGeom ag = L.ag;
             ag.kv_off = lg.cache_off;
             ag.out_ld = a.heads * a.kv_rank;
             ag.out_scale = 1.0f;
             ag.fused_prep = 0;
-            if (!attn_tile(m, sm, ag, L.n_in, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
-            gemm_heads(m, m->act_a, a.heads * a.kv_rank, a.kv_rank, L.w_uv, a.heads, a.vdim, a.kv_rank, m->O, nv, a.vdim, R);
-            const unsigned nb = (unsigned)(((size_t)R * nv + 255) / 256);
-            if (m->f32) launch(m, lp_latent_gate_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->O, (const float*)m->P, L.n_in, lg.g_off, a.out_gate, nv, R, (float*)m->act_a);
-            else launch(m, lp_latent_gate_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->O, (const float*)m->P, L.n_in, lg.g_off, a.out_gate, nv, R, (bf16*)m->act_a);
+            if (split) {
+                const float* Q = direct ? m->P + lg.q_off : m->O;
+                const int ldq = direct ? L.n_in : a.heads * per, vn = m->f32 ? 4 : 8, splits = latent_splits(R, a.heads);
+                const int uk_cols = 8 * (32 / latent_lanes(a.dim, vn)), uk_ch = (a.kv_rank + uk_cols - 1) / uk_cols;
+                const int uv_cols = 8 * (32 / latent_lanes(a.kv_rank, vn)), uv_ch = (a.vdim + uv_cols - 1) / uv_cols;
+                const dim3 agrid(a.heads * uk_ch + (direct && own ? R : 0)), sgrid(splits, R, (a.heads + LS_HEADS - 1) / LS_HEADS), ugrid(a.heads * uv_ch);
+                const size_t asm_ = (size_t)(R * a.dim + lg.rot_n) * 4, usm = (size_t)R * (a.kv_rank + splits) * 4;
+                if (m->f32) launch(m, lp_latent_absorb_kernel<float>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const float*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
+                else launch(m, lp_latent_absorb_kernel<bf16>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const bf16*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
+#define LP_LS(V) launch(m, lp_latent_split_kernel<V>, sgrid, dim3(32 * LS_HEADS), latent_split_smem(D), sm, ag, (const float*)m->qbuf, m->lat_o, m->lat_ml)
+                if (a.kv_rank <= 128) LP_LS(4); else if (a.kv_rank <= 256) LP_LS(8); else LP_LS(16);
+#undef LP_LS
+                if (m->f32) launch(m, lp_latent_merge_kernel<float>, ugrid, dim3(256), usm, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (const float*)L.w_uv, (const float*)m->P, L.n_in, (float*)m->act_a, R, uv_ch);
+                else launch(m, lp_latent_merge_kernel<bf16>, ugrid, dim3(256), usm, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (const bf16*)L.w_uv, (const float*)m->P, L.n_in, (bf16*)m->act_a, R, uv_ch);
+            } else {
+                if (!direct) {
+                    if (m->f32) launch(m, lp_latent_qprep_kernel<float>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->O, L.rot_freq, (float*)m->act_a, m->qbuf);
+                    else launch(m, lp_latent_qprep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->O, L.rot_freq, (bf16*)m->act_a, m->qbuf);
+                }
+                gemm_heads(m, m->act_a, a.heads * a.dim, a.dim, L.w_ukT, a.heads, a.kv_rank, a.dim, m->qbuf, a.heads * D, D, R);
+                if (!attn_tile(m, sm, ag, L.n_in, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
+                gemm_heads(m, m->act_a, a.heads * a.kv_rank, a.kv_rank, L.w_uv, a.heads, a.vdim, a.kv_rank, m->O, nv, a.vdim, R);
+                const unsigned nb = (unsigned)(((size_t)R * nv + 255) / 256);
+                if (m->f32) launch(m, lp_latent_gate_kernel<float>, dim3(nb), dim3(256), 0, lg, (const float*)m->O, (const float*)m->P, L.n_in, R, (float*)m->act_a);
+                else launch(m, lp_latent_gate_kernel<bf16>, dim3(nb), dim3(256), 0, lg, (const float*)m->O, (const float*)m->P, L.n_in, R, (bf16*)m->act_a);
+            }
             project_out(m->act_a, nv, L.wo, L.norm1, moe_next);
         } else if (L.d.mixer == B200_MIX_STATE_SPACE) {
             const b200_state_space_desc& g = L.d.ssd;
@@ -2927,20 +3146,33 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             const b200_moe_desc& e = L.d.moe;
             const size_t es = elt(m);
             const int act_epi = e.act == B200_ACT_GELU ? EPI_GELU : EPI_RELU2;
-            const int per = e.act == B200_ACT_SILU_GLU ? 2 * e.expert_ff : e.expert_ff;      // rows of one expert's up matrix
-            const bool own_act = e.act == B200_ACT_SILU_GLU || e.weight_input != 0;            // the hidden units need a kernel of their own
+            const int per = act_gated(e.act) ? 2 * e.expert_ff : e.expert_ff;                // rows of one expert's up matrix
+            const bool own_act = act_gated(e.act) || e.weight_input != 0;                      // the hidden units need a kernel of their own
+            const ExpertAct ea{e.act, e.weight_input, e.limit, e.shared_limit, e.slope};
+            const int rrows = e.experts + (e.shared_gate ? 1 : 0);                             // logits of a row: the experts', then the always-on gate's
+            float* shw = e.shared_gate ? m->moe_shw : nullptr;
             sub = 1;
-            if (streams) boundary(L.hc_in[1], L.norm2, nullptr);
+            bool routed = par || moe_next != nullptr;
+            if (p.in_conv > 0) {
+                StepRoute rt{};
+                if (ring_step && R <= 2 * GV_ROWS) {       // few rows: the block that norms a row also routes it
+                    rt.router = L.w_up; rt.bias = L.router_bias; rt.rows = rrows; rt.E = e.experts; rt.top = e.top; rt.mode = e.route; rt.scale = e.route_scale;
+                    rt.logits = m->P; rt.wts = m->moe_w; rt.sel = m->moe_sel; rt.selw = m->moe_selw; rt.shw = shw;
+                    routed = true;
+                }
+                conv_in(L.ic[1], L.norm2, rt);
+            } else if (streams) boundary(L.hc_in[1], L.norm2, nullptr);
             else if (!post && !par) rmsnorm(m, m->x, nullptr, L.norm2, m->hn, nullptr, R);
             if (par) {
-                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P + L.ff_off, L.n_in, e.experts, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale);
-            } else if (!moe_next) {
-                gemm(m, m->hn, W, L.w_up, e.experts, W, m->P, e.experts, R, 1.0f, EPI_STORE);
-                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P, e.experts, e.experts, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale);
+                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P + L.ff_off, L.n_in, e.experts, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale, (float*)nullptr);
+            } else if (!routed) {
+                gemm(m, m->hn, W, L.w_up, rrows, W, m->P, rrows, R, 1.0f, EPI_STORE, nullptr, L.router_bias);
+                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P, rrows, e.experts, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale, shw);
             }
             const size_t hbytes = (size_t)R * W * es;
             const uint8_t* up_experts = (const uint8_t*)L.w_up + (size_t)L.up_router_rows * W * es;
-            float* ydst = par ? m->x : m->y;          // parallel_ff: the experts' sum goes straight into the residual stream
+            const bool direct = !post && !streams;     // x += : the experts' sum goes straight into the residual stream
+            float* ydst = direct ? m->x : m->y;
             bool normed = false;
             if (moe_sel_ok) {
                 // few rows (decoding): kernels that walk each row's choices and read those experts' weights only
@@ -2950,11 +3182,11 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                 normed = few || sfew;
                 if (sfew) pre_done = true;
                 if (m->f32) {
-                    launch(m, lp_moe_up_sel_kernel<float>, ugrid, dim3(256), hbytes, (const float*)m->hn, (const float*)up_experts, (const int*)m->moe_sel, (const float*)m->moe_selw, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, (float*)m->act_a, e.act, e.weight_input);
-                    launch(m, lp_moe_down_sel_kernel<float>, dgrid, dim3(256), 0, (const float*)m->act_a, (const float*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, par ? 1 : 0);
+                    launch(m, lp_moe_up_sel_kernel<float>, ugrid, dim3(256), hbytes, (const float*)m->hn, (const float*)up_experts, (const int*)m->moe_sel, (const float*)m->moe_selw, (const float*)shw, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, (float*)m->act_a, ea);
+                    launch(m, lp_moe_down_sel_kernel<float>, dgrid, dim3(256), 0, (const float*)m->act_a, (const float*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, direct ? 1 : 0);
                 } else {
-                    launch(m, lp_moe_up_sel_kernel<bf16>, ugrid, dim3(256), hbytes, (const bf16*)m->hn, (const bf16*)up_experts, (const int*)m->moe_sel, (const float*)m->moe_selw, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, (bf16*)m->act_a, e.act, e.weight_input);
-                    launch(m, lp_moe_down_sel_kernel<bf16>, dgrid, dim3(256), 0, (const bf16*)m->act_a, (const bf16*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, par ? 1 : 0);
+                    launch(m, lp_moe_up_sel_kernel<bf16>, ugrid, dim3(256), hbytes, (const bf16*)m->hn, (const bf16*)up_experts, (const int*)m->moe_sel, (const float*)m->moe_selw, (const float*)shw, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, (bf16*)m->act_a, ea);
+                    launch(m, lp_moe_down_sel_kernel<bf16>, dgrid, dim3(256), 0, (const bf16*)m->act_a, (const bf16*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, direct ? 1 : 0);
                 }
             } else if (m->use_fuse && R > 2 * GV_ROWS) {
                 // many rows: the (token, choice) pairs in expert order, one product pair per expert over its block of rows (the row
@@ -2968,34 +3200,46 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                 if (own_act) {
                     // pre-activations in f32 (m->P: its router columns have been read), then the units with the pair's weight
                     gemm_grouped(m, m->moe_xp, W, up_experts, W, (size_t)per * W, e.experts, per, W, m->P, per, R, EPI_STORE, m->moe_seg);
-                    const unsigned nb = (unsigned)(((size_t)pairs * e.expert_ff + 255) / 256);
-                    if (m->f32) launch(m, lp_moe_pair_act_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->P, per, (const int*)m->moe_pos, (const float*)m->moe_selw, e.expert_ff, (float*)m->act_a, pairs, e.act, e.weight_input);
-                    else launch(m, lp_moe_pair_act_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->P, per, (const int*)m->moe_pos, (const float*)m->moe_selw, e.expert_ff, (bf16*)m->act_a, pairs, e.act, e.weight_input);
+                    const int V = e.expert_ff % 4 ? 1 : 4;
+                    const unsigned nb = (unsigned)(((size_t)pairs * (e.expert_ff / V) + 255) / 256);
+#define LP_PA(T, V) launch(m, lp_moe_pair_act_kernel<T, V>, dim3(nb), dim3(256), 0, (const float*)m->P, per, (const int*)m->moe_pos, (const float*)m->moe_selw, e.expert_ff, (T*)m->act_a, pairs, ea)
+                    if (m->f32) { if (V == 4) LP_PA(float, 4); else LP_PA(float, 1); }
+                    else { if (V == 4) LP_PA(bf16, 4); else LP_PA(bf16, 1); }
+#undef LP_PA
                 } else {
                     gemm_grouped(m, m->moe_xp, W, up_experts, W, (size_t)e.expert_ff * W, e.experts, e.expert_ff, W, m->act_a, e.expert_ff, R, act_epi, m->moe_seg);
                 }
                 gemm_grouped(m, m->act_a, e.expert_ff, down, L.k_down, (size_t)e.expert_ff, e.experts, W, e.expert_ff, m->moe_yp, W, R, EPI_STORE, m->moe_seg);
                 if (e.shared_ff > 0) {
-                    gemm(m, m->hn, W, up_experts + (size_t)e.experts * per * W * es, e.shared_ff, W, act_sh, e.shared_ff, R, 1.0f, act_epi);
-                    gemm_ld(m, act_sh, e.shared_ff, down + (size_t)e.experts * e.expert_ff * es, L.k_down, W, e.shared_ff, ydst, W, R, par ? EPI_ADD : EPI_STORE);
+                    const uint8_t* up_sh = up_experts + (size_t)e.experts * per * W * es;
+                    if (act_gated(e.act) || shw) {         // (m->P: the pairs' pre-activations have been read)
+                        const int per_sh = act_gated(e.act) ? 2 * e.shared_ff : e.shared_ff;
+                        gemm(m, m->hn, W, up_sh, per_sh, W, m->P, per_sh, R, 1.0f, EPI_STORE);
+                        const int V = e.shared_ff % 4 || ((uintptr_t)act_sh & 15) ? 1 : 4;
+                        const unsigned nb = (unsigned)(((size_t)R * (e.shared_ff / V) + 255) / 256);
+#define LP_SA(T, V) launch(m, lp_moe_shared_act_kernel<T, V>, dim3(nb), dim3(256), 0, (const float*)m->P, per_sh, (const float*)shw, e.shared_ff, (T*)act_sh, R, ea)
+                        if (m->f32) { if (V == 4) LP_SA(float, 4); else LP_SA(float, 1); }
+                        else { if (V == 4) LP_SA(bf16, 4); else LP_SA(bf16, 1); }
+#undef LP_SA
+                    } else gemm(m, m->hn, W, up_sh, e.shared_ff, W, act_sh, e.shared_ff, R, 1.0f, act_epi);
+                    gemm_ld(m, act_sh, e.shared_ff, down + (size_t)e.experts * e.expert_ff * es, L.k_down, W, e.shared_ff, ydst, W, R, direct ? EPI_ADD : EPI_STORE);
                 }
                 launch(m, lp_moe_combine_kernel, dim3(R), dim3(256), 0, (const float*)m->moe_yp, (const int*)m->moe_pos, own_act ? (const float*)nullptr : (const float*)m->moe_selw, e.top, W,
-                       (par || e.shared_ff > 0) ? 1 : 0, ydst);
+                       (direct || e.shared_ff > 0) ? 1 : 0, ydst);
             } else {
                 // the plain form: every expert's up projection for every row, activations times their expert's weight (0 for experts
                 // that were not chosen), one product with the down matrices side by side
                 const int n_exp = L.n_up - L.up_router_rows;
                 gemm(m, m->hn, W, up_experts, n_exp, W, m->P, n_exp, R, 1.0f, EPI_STORE);
                 const unsigned nb = (unsigned)(((size_t)R * L.k_down + 255) / 256);
-                if (m->f32) launch(m, lp_moe_act_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, e.experts, e.expert_ff, L.k_down, (float*)m->act_a, R, e.act, e.weight_input);
-                else launch(m, lp_moe_act_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, e.experts, e.expert_ff, L.k_down, (bf16*)m->act_a, R, e.act, e.weight_input);
-                gemm(m, m->act_a, L.k_down, L.w_down, W, L.k_down, ydst, W, R, 1.0f, par ? EPI_ADD : EPI_STORE);
+                if (m->f32) launch(m, lp_moe_act_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, (const float*)shw, e.experts, e.expert_ff, e.shared_ff, (float*)m->act_a, R, ea);
+                else launch(m, lp_moe_act_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, (const float*)shw, e.experts, e.expert_ff, e.shared_ff, (bf16*)m->act_a, R, ea);
+                gemm(m, m->act_a, L.k_down, L.w_down, W, L.k_down, ydst, W, R, 1.0f, direct ? EPI_ADD : EPI_STORE);
             }
-            if (normed || par) {
+            if (normed || direct) {
             } else if (streams) {
                 pend.y = m->y; pend.mix = L.hc_mix[1]; pend.out = L.hc_out[1];
-            } else if (post) cast_x(m->y, L.norm2);
-            else launch(m, lp_add_rows_kernel, dim3((unsigned)(((size_t)R * W + 255) / 256)), dim3(256), 0, m->x, (const float*)m->y, (size_t)R * W);
+            } else cast_x(m->y, L.norm2);
         } else if (L.d.ff > 0 && (L.d.ff_kind == B200_FF_GATED_GELU || L.d.ff_kind == B200_FF_CLAMPED_GLU)) {
             // [gate | up] in one product (with parallel_ff: columns ff_off .. of the layer's input projection), the gated units, W_down
             sub = 1;
@@ -3028,7 +3272,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             project_out(m->act_a, L.d.ff, L.w_down, L.norm2, nullptr);
         } else if (L.d.ff > 0) {
             sub = 1;
-            project_in(nullptr, L.norm2, L.w_up, L.d.ff, m->act_a, L.d.ff, EPI_RELU2);
+            project_in(nullptr, L.norm2, L.w_up, L.d.ff, m->act_a, L.d.ff, L.d.ff_kind == B200_FF_XIELU ? EPI_XIELU : EPI_RELU2);
             project_out(m->act_a, L.d.ff, L.w_down, L.norm2, nullptr);
         } else if (post && L.norm2) {
             cast_x(nullptr, L.norm2);

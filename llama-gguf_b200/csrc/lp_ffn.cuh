@@ -64,10 +64,11 @@ __global__ void lp_relu2_kernel(const float* __restrict__ P, int ldp, OutT* __re
 
 // Router: one warp per row of the f32 logits P[r][0 .. E) (route_row, lp_rows_tail.cuh)
 __global__ void lp_moe_route_kernel(const float* __restrict__ P, int ldp, int E, int top, float* __restrict__ wts, int* __restrict__ sel,
-                                    float* __restrict__ selw, int R, int mode, float scale) {
+                                    float* __restrict__ selw, int R, int mode, float scale, float* __restrict__ shw) {
     const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (r >= R) return;
     route_row(P + (size_t)r * ldp, E, top, wts + (size_t)r * E, sel + (size_t)r * top, selw + (size_t)r * top, lane, mode, scale);
+    if (shw && lane == 0) shw[r] = sigmoid_f(P[(size_t)r * ldp + E]);      // the always-on expert's gate: the logit behind the experts'
 }
 
 // an expert's activation: relu(z)^2 (B200_ACT_RELU2) or the exact GELU (B200_ACT_GELU)
@@ -77,56 +78,95 @@ __device__ __forceinline__ float expert_act(float z, int act) {
     return z * z;
 }
 
-// A gated expert (B200_ACT_SILU_GLU) has two pre-activations per hidden unit, silu(g) * u; its up matrix is [gate | up] rows.
-__device__ __forceinline__ int expert_rows(int eff, int act) { return act == B200_ACT_SILU_GLU ? 2 * eff : eff; }
+// What an expert's hidden units are made of.  The gated kinds (B200_ACT_SILU_GLU, B200_ACT_CLAMPED_GLU) have two pre-activations per unit,
+// their up matrix is [gate | up] rows.
+struct ExpertAct {
+    int kind, win;               // B200_ACT_*; 1: the expert's weight goes onto its input
+    float limit, shared_limit, slope;
+};
+__host__ __device__ inline bool act_gated(int kind) { return kind == B200_ACT_SILU_GLU || kind == B200_ACT_CLAMPED_GLU; }
+__device__ __forceinline__ int expert_rows(int eff, int kind) { return act_gated(kind) ? 2 * eff : eff; }
+// min(z, limit) sigmoid(slope .) (clamp(zu, +-limit) + 1)
+__device__ __forceinline__ float clamped_glu_f(float z, float zu, float limit, float slope) {
+    const float g = fminf(z, limit), u = fminf(fmaxf(zu, -limit), limit);
+    return g * sigmoid_f(slope * g) * (u + 1.0f);
+}
 // hidden unit of an expert from its pre-activation(s) and the expert's weight w: on the output, act(.) w, or on the input (win),
 // where W (w h) = w (W h) puts it on the pre-activations
-__device__ __forceinline__ float expert_unit(float z, float zu, float w, int act, int win) {
-    if (win) { z *= w; zu *= w; }
-    const float v = act == B200_ACT_SILU_GLU ? z * sigmoid_f(z) * zu : expert_act(z, act);
-    return win ? v : v * w;
+__device__ __forceinline__ float expert_unit(float z, float zu, float w, const ExpertAct& a, float limit) {
+    if (a.win) { z *= w; zu *= w; }
+    const float v = a.kind == B200_ACT_CLAMPED_GLU ? clamped_glu_f(z, zu, limit, a.slope) : a.kind == B200_ACT_SILU_GLU ? z * sigmoid_f(z) * zu : expert_act(z, a.kind);
+    return a.win ? v : v * w;
+}
+// the always-on expert: the same form, its weight (1 without a gate) always on the output
+__device__ __forceinline__ float shared_unit(float z, float zu, float w, ExpertAct a) {
+    a.win = 0;
+    return expert_unit(z, zu, w, a, a.shared_limit);
 }
 
 // out[r][c] = hidden unit c of the row: expert e = c / eff with its weight (0 = not chosen: the unit is 0), the always-on expert's
-// units behind them with weight 1.  P holds every expert's pre-activations side by side (expert_rows per expert).
+// units behind them with weight shw[r] (null: 1).  P holds every expert's pre-activations side by side (expert_rows per expert).
 template <typename OutT>
-__global__ void lp_moe_act_kernel(const float* __restrict__ P, int ldp, int off, const float* __restrict__ wts, int E, int eff, int total,
-                                  OutT* __restrict__ out, int R, int act, int win) {
+__global__ void lp_moe_act_kernel(const float* __restrict__ P, int ldp, int off, const float* __restrict__ wts, const float* __restrict__ shw, int E, int eff,
+                                  int sff, OutT* __restrict__ out, int R, ExpertAct a) {
+    const int total = E * eff + sff;
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (size_t)R * total) return;
     const int r = (int)(i / total), c = (int)(i - (size_t)r * total);
-    const int e = c / eff, per = expert_rows(eff, act);
-    const float wgt = e < E ? wts[(size_t)r * E + e] : 1.0f;
+    const int per = expert_rows(eff, a.kind);
+    const bool glu = act_gated(a.kind);
+    const float* p = P + (size_t)r * ldp + off;
     float v = 0.0f;
-    if (wgt != 0.0f) {
-        const float* p = P + (size_t)r * ldp + off;
-        if (e < E) v = expert_unit(p[e * per + (c - e * eff)], act == B200_ACT_SILU_GLU ? p[e * per + eff + (c - e * eff)] : 0.0f, wgt, act, win);
-        else v = expert_act(p[E * per + (c - E * eff)], act);
+    if (c < E * eff) {
+        const int e = c / eff, n = c - e * eff;
+        const float w = wts[(size_t)r * E + e];
+        if (w != 0.0f) v = expert_unit(p[e * per + n], glu ? p[e * per + eff + n] : 0.0f, w, a, a.limit);
+    } else {
+        const int n = c - E * eff;
+        v = shared_unit(p[E * per + n], glu ? p[E * per + sff + n] : 0.0f, shw ? shw[r] : 1.0f, a);
     }
     out[i] = from_f<OutT>(v);
 }
 
 // The same for (token, choice) pairs in expert order: pair i = (row i / top, choice i % top) sits at row pos[i] of P (its expert's
-// pre-activations, expert_rows wide) and of out (eff wide); its weight is selw[i].
-template <typename OutT>
+// pre-activations, expert_rows wide) and of out (eff wide); its weight is selw[i].  V units per thread (4: eff a multiple of 4).
+template <typename OutT, int V>
 __global__ void lp_moe_pair_act_kernel(const float* __restrict__ P, int ldp, const int* __restrict__ pos, const float* __restrict__ selw, int eff,
-                                       OutT* __restrict__ out, int n_pairs, int act, int win) {
+                                       OutT* __restrict__ out, int n_pairs, ExpertAct a) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= (size_t)n_pairs * eff) return;
-    const int pr = (int)(i / eff), n = (int)(i - (size_t)pr * eff);
+    if (i >= (size_t)n_pairs * (eff / V)) return;
+    const int pr = (int)(i / (eff / V)), n = (int)(i - (size_t)pr * (eff / V)) * V;
     const float* p = P + (size_t)pos[pr] * ldp;
-    out[(size_t)pos[pr] * eff + n] = from_f<OutT>(expert_unit(p[n], act == B200_ACT_SILU_GLU ? p[eff + n] : 0.0f, selw[pr], act, win));
+    const FloatV<V> z = load_v<V>(p + n), zu = act_gated(a.kind) ? load_v<V>(p + eff + n) : z;
+    FloatV<V> o;
+#pragma unroll
+    for (int e = 0; e < V; e++) o.v[e] = expert_unit(z.v[e], zu.v[e], selw[pr], a, a.limit);
+    store_v<V>(out + (size_t)pos[pr] * eff + n, o);
+}
+// and for the always-on expert over all rows: P [R][expert_rows(sff)] -> out [R][sff]
+template <typename OutT, int V>
+__global__ void lp_moe_shared_act_kernel(const float* __restrict__ P, int ldp, const float* __restrict__ shw, int sff, OutT* __restrict__ out, int R, ExpertAct a) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (size_t)R * (sff / V)) return;
+    const int r = (int)(i / (sff / V)), n = (int)(i - (size_t)r * (sff / V)) * V;
+    const float* p = P + (size_t)r * ldp;
+    const FloatV<V> z = load_v<V>(p + n), zu = act_gated(a.kind) ? load_v<V>(p + sff + n) : z;
+    const float w = shw ? shw[r] : 1.0f;
+    FloatV<V> o;
+#pragma unroll
+    for (int e = 0; e < V; e++) o.v[e] = shared_unit(z.v[e], zu.v[e], w, a);
+    store_v<V>(out + (size_t)r * sff + n, o);
 }
 
 // Few rows (decoding): only the chosen experts' weights are read.  up_exp holds [e0 up | e1 up | ... | always-on up] rows of `width`
 // columns (a gated expert: [gate | up], expert_rows each); segment k < top of a row's activations belongs to expert sel[r][k],
 // segment `top` to the always-on expert.
-//   act[r][k eff + n] = unit(up_e[n] . h_r, selw[r][k])        act[r][top eff + n] = act(up_shared[n] . h_r)      (expert_unit)
+//   act[r][k eff + n] = unit(up_e[n] . h_r, selw[r][k])        act[r][top eff + n] = unit(up_shared[n] . h_r, shw[r] or 1)
 // One warp per (row, segment, n); h rows are staged in shared memory once per block.
 template <typename T>
 __global__ void __launch_bounds__(256) lp_moe_up_sel_kernel(const T* __restrict__ H, const T* __restrict__ up_exp, const int* __restrict__ sel,
-                                                            const float* __restrict__ selw, int E, int top, int eff, int sff, int width, int R,
-                                                            T* __restrict__ act, int act_kind, int win) {
+                                                            const float* __restrict__ selw, const float* __restrict__ shw, int E, int top, int eff, int sff,
+                                                            int width, int R, T* __restrict__ act, ExpertAct a) {
     extern __shared__ __align__(16) uint8_t mu_smem[];
     T* hs = reinterpret_cast<T*>(mu_smem);
     constexpr int VN = Vec8<T>::N;
@@ -134,17 +174,16 @@ __global__ void __launch_bounds__(256) lp_moe_up_sel_kernel(const T* __restrict_
         *reinterpret_cast<uint4*>(hs + (size_t)i * VN) = *reinterpret_cast<const uint4*>(H + (size_t)i * VN);
     __syncthreads();
     const int lane = threadIdx.x & 31;
-    const int per_row = top * eff + sff;
+    const int per_row = top * eff + sff, per = expert_rows(eff, a.kind);
     const int total = R * per_row;
+    const bool glu = act_gated(a.kind);
     for (int o = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5); o < total; o += gridDim.x * (blockDim.x >> 5)) {
         const int r = o / per_row, c = o - r * per_row;
         const int k = c < top * eff ? c / eff : top;
         const int n = c - k * eff;
         const int e = k < top ? sel[(size_t)r * top + k] : E;
-        const int per = expert_rows(eff, act_kind);
-        const bool glu = act_kind == B200_ACT_SILU_GLU && k < top;
         const T* wr = up_exp + ((size_t)e * per + n) * width;
-        const T* wu = wr + (size_t)eff * width;          // (gated experts: the up row of the same unit)
+        const T* wu = wr + (size_t)(k < top ? eff : sff) * width;          // (gated experts: the up row of the same unit)
         const T* hr = hs + (size_t)r * width;
         float acc = 0.0f, accu = 0.0f;
         for (int i = lane * VN; i < width; i += 32 * VN) {
@@ -161,7 +200,8 @@ __global__ void __launch_bounds__(256) lp_moe_up_sel_kernel(const T* __restrict_
         }
         acc = wsum(acc);
         accu = wsum(accu);
-        if (lane == 0) act[o] = from_f<T>(k < top ? expert_unit(acc, accu, selw[(size_t)r * top + k], act_kind, win) : expert_act(acc, act_kind));
+        if (lane == 0)
+            act[o] = from_f<T>(k < top ? expert_unit(acc, accu, selw[(size_t)r * top + k], a, a.limit) : shared_unit(acc, accu, shw ? shw[r] : 1.0f, a));
     }
 }
 
@@ -260,9 +300,4 @@ __global__ void lp_moe_combine_kernel(const float* __restrict__ Yp, const int* _
         for (int k = 0; k < top; k++) sum = fmaf(selw ? selw[(size_t)r * top + k] : 1.0f, Yp[(size_t)pos[(size_t)r * top + k] * width + c], sum);
         y[(size_t)r * width + c] = acc + sum;
     }
-}
-
-__global__ void lp_add_rows_kernel(float* __restrict__ x, const float* __restrict__ y, size_t n) {
-    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) x[i] += y[i];
 }

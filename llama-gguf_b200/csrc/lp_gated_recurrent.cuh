@@ -298,10 +298,6 @@ __global__ void __launch_bounds__(256) lp_dual_norm_add_kernel(float* __restrict
 // ------------------------------------------------------------------------------------------------ clamped gated feed-forward
 // out[r][n] = g sigmoid(slope g) (u + 1), g = min(P[r][n], limit), u = clamp(P[r][ff + n], -limit, limit): P holds [gate | up].
 // A thread takes VEC neighbouring units (VEC = 4: 16-byte loads; ff, the row pitch and the column offset multiples of 4).
-__device__ __forceinline__ float clamped_glu_f(float zg, float zu, float limit, float slope) {
-    const float g = fminf(zg, limit), u = fminf(fmaxf(zu, -limit), limit);
-    return g * sigmoid_f(slope * g) * (u + 1.0f);
-}
 template <typename OutT, int VEC>
 __global__ void lp_clamped_glu_kernel(const float* __restrict__ P, int ldp, OutT* __restrict__ out, int ff, int R, float limit, float slope) {
     const int per = ff / VEC;

@@ -3,14 +3,16 @@
 // of layerprog.cu read it as ONE K/V head whose keys are the whole row and whose values are the row's first kv_rank entries
 // (AttnGeom.v_in_k).  For that, head n's query is carried into the latent: qbuf[r][n] = [W_uk[n]^T q_plain | rotated q part], and the
 // summed latent comes back through W_uv[n] afterwards (two products batched over the heads).  Included by layerprog.cu inside its
-// anonymous namespace.  Norms, angles and the rotation are f32 (the angle, its sine and cosine in double).
+// anonymous namespace, behind lp_input_conv.cuh (block_sum_sq).  Norms, angles and the rotation are f32 (the angle, its sine and cosine in double).
 #pragma once
 
 struct LatentGeom {
     int H, dim, rot_dim, vdim, q_rank, kv_rank;
-    int rot_n;               // rotated channels (even, <= rot_dim); channel i pairs with i + rot_n / 2
+    int rot_n;               // rotated channels (even, <= rot_dim); channel i pairs with i + rot_n / 2, or 2i with 2i + 1 (pairs)
+    int pairs;
     float rot_mult;          // factor on cos and sin
-    int q_off, kv_off, g_off;   // columns of the fused input projection P: [W_dq h | W_dkv h | W_g h]; kv_off < 0: no W_dkv (borrowed rows)
+    int q_off, kv_off, g_off;   // columns of the fused input projection P: [W_dq h or W_q h | W_dkv h | W_g h]; kv_off < 0: no W_dkv (borrowed rows)
+    int gate;                // B200_GATE_*
     size_t cache_off;        // byte offset of the rows inside a slot's cache block
     int cap;
     float eps;
@@ -28,25 +30,54 @@ __device__ __forceinline__ void latent_angles(const LatentGeom& g, const double*
 __device__ __forceinline__ float latent_rot(const LatentGeom& g, const float* v, int i, const float* cs, const float* sn) {
     const int half = g.rot_n / 2;
     if (i >= g.rot_n) return v[i];
+    if (g.pairs) return (i & 1) ? v[i] * cs[i >> 1] + v[i - 1] * sn[i >> 1] : v[i] * cs[i >> 1] - v[i + 1] * sn[i >> 1];
     return i < half ? v[i] * cs[i] - v[i + half] * sn[i] : v[i] * cs[i - half] + v[i - half] * sn[i - half];
 }
 
-// One block per row, after the fused input projection.  c_q = rmsnorm(P[q_off ..]) * qw -> cq (compute type, the operand of W_uq).
-// With a W_dkv of its own: c = rmsnorm(P[kv_off .. + kv_rank]) * kvw and the rotated last rot_dim columns -> the cache row of the
-// row's position.
+// sigmoid of the gate column of value channel c (head c / vdim) of a row of P
+__device__ __forceinline__ float latent_gate(const LatentGeom& g, const float* __restrict__ p, int c) {
+    return g.gate == B200_GATE_NONE ? 1.0f : sigmoid_f(p[g.g_off + (g.gate == B200_GATE_HEAD ? c / g.vdim : c)]);
+}
+
+// The cache row of a row's position: c = rmsnorm(P[kv_off .. + kv_rank]) * kvw and the rotated last rot_dim columns.  sk: the squared sum of
+// the first part; cs / sn: latent_angles of the position.
+__device__ __forceinline__ void latent_cache_row(const LatentGeom& g, const StepMeta& sm, int r, const float* __restrict__ p, float sk,
+                                                 const float* __restrict__ kvw, const float* cs, const float* sn) {
+    const float ik = 1.0f / sqrtf(sk / (float)g.kv_rank + g.eps);
+    float* row = reinterpret_cast<float*>(sm.run_kv[sm.row_run[r]] + g.cache_off) + (size_t)sm.row_pos[r] * (g.kv_rank + g.rot_dim);
+    for (int c = threadIdx.x; c < g.kv_rank; c += blockDim.x) row[c] = p[g.kv_off + c] * ik * kvw[c];
+    const float* kr = p + g.kv_off + g.kv_rank;
+    for (int i = threadIdx.x; i < g.rot_dim; i += blockDim.x) row[g.kv_rank + i] = latent_rot(g, kr, i, cs, sn);
+}
+
+// A row's query q (per head [dim | rot_dim], f32): the plain part of every head in the compute type -> qn [H dim] (the operand of the
+// product with W_uk^T), the rotated part -> qrow[n (kv_rank + rot_dim) + kv_rank ..].
+template <typename T>
+__device__ __forceinline__ void latent_query_row(const LatentGeom& g, const float* __restrict__ q, const float* cs, const float* sn, T* __restrict__ qn,
+                                                 float* __restrict__ qrow) {
+    const int per = g.dim + g.rot_dim, D = g.kv_rank + g.rot_dim;
+    for (int i = threadIdx.x; i < g.H * per; i += blockDim.x) {
+        const int n = i / per, c = i - n * per;
+        if (c < g.dim) qn[n * g.dim + c] = from_f<T>(q[i]);
+        else qrow[(size_t)n * D + g.kv_rank + (c - g.dim)] = latent_rot(g, q + n * per + g.dim, c - g.dim, cs, sn);
+    }
+}
+
+// One block per row, after the fused input projection.  With a query latent: c_q = rmsnorm(P[q_off ..]) * qw -> cq (compute type, the
+// operand of W_uq); without one (q_rank = 0) P holds the query itself, which goes to qn / qbuf (latent_query_row).  With a W_dkv of its
+// own the row's cache row is written.
 template <typename T>
 __global__ void __launch_bounds__(256) lp_latent_prep_kernel(StepMeta sm, LatentGeom g, const float* __restrict__ P, int ldp,
                                                              const float* __restrict__ qw, const float* __restrict__ kvw,
-                                                             const double* __restrict__ freq, T* __restrict__ cq) {
+                                                             const double* __restrict__ freq, T* __restrict__ cq, T* __restrict__ qn, float* __restrict__ qbuf) {
     extern __shared__ float lp_cs[];     // [rot_n / 2] cos, then sin
     __shared__ float red[2][8];
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    const int run = sm.row_run[r], pos = sm.row_pos[r];
     const float* p = P + (size_t)r * ldp;
     float* cs = lp_cs;
     float* sn = lp_cs + g.rot_n / 2;
-    const bool own = g.kv_off >= 0;
-    if (own) latent_angles(g, freq, pos, cs, sn);
+    const bool own = g.kv_off >= 0, direct = g.q_rank == 0;
+    if (own || direct) latent_angles(g, freq, sm.row_pos[r], cs, sn);
     float sq = 0.0f, sk = 0.0f;
     for (int c = threadIdx.x; c < g.q_rank; c += blockDim.x) sq = fmaf(p[g.q_off + c], p[g.q_off + c], sq);
     if (own)
@@ -57,43 +88,261 @@ __global__ void __launch_bounds__(256) lp_latent_prep_kernel(StepMeta sm, Latent
     __syncthreads();
     sq = 0.0f; sk = 0.0f;
     for (int i = 0; i < nw; i++) { sq += red[0][i]; sk += red[1][i]; }
-    const float iq = 1.0f / sqrtf(sq / (float)g.q_rank + g.eps);
-    for (int c = threadIdx.x; c < g.q_rank; c += blockDim.x) cq[(size_t)r * g.q_rank + c] = from_f<T>(p[g.q_off + c] * iq * qw[c]);
-    if (!own) return;
-    const float ik = 1.0f / sqrtf(sk / (float)g.kv_rank + g.eps);
-    float* row = reinterpret_cast<float*>(sm.run_kv[run] + g.cache_off) + (size_t)pos * (g.kv_rank + g.rot_dim);
-    for (int c = threadIdx.x; c < g.kv_rank; c += blockDim.x) row[c] = p[g.kv_off + c] * ik * kvw[c];
-    const float* kr = p + g.kv_off + g.kv_rank;
-    for (int i = threadIdx.x; i < g.rot_dim; i += blockDim.x) row[g.kv_rank + i] = latent_rot(g, kr, i, cs, sn);
+    if (direct) latent_query_row(g, p + g.q_off, cs, sn, qn + (size_t)r * g.H * g.dim, qbuf + (size_t)r * g.H * (g.kv_rank + g.rot_dim));
+    else {
+        const float iq = 1.0f / sqrtf(sq / (float)g.q_rank + g.eps);
+        for (int c = threadIdx.x; c < g.q_rank; c += blockDim.x) cq[(size_t)r * g.q_rank + c] = from_f<T>(p[g.q_off + c] * iq * qw[c]);
+    }
+    if (own) latent_cache_row(g, sm, r, p, sk, kvw, cs, sn);
 }
 
-// One block per row, after q = W_uq c_q (Q [R][H (dim + rot_dim)] f32): the plain part of every head in the compute type -> qn
-// [R][H dim] (the operand of the product with W_uk^T), the rotated part -> qbuf[r][n (kv_rank + rot_dim) + kv_rank ..].
+// One block per row, after q = W_uq c_q (Q [R][H (dim + rot_dim)] f32)
 template <typename T>
 __global__ void __launch_bounds__(256) lp_latent_qprep_kernel(StepMeta sm, LatentGeom g, const float* __restrict__ Q, const double* __restrict__ freq,
                                                               T* __restrict__ qn, float* __restrict__ qbuf) {
     extern __shared__ float lq_cs[];
-    const int r = blockIdx.x, pos = sm.row_pos[r];
+    const int r = blockIdx.x;
     float* cs = lq_cs;
     float* sn = lq_cs + g.rot_n / 2;
-    latent_angles(g, freq, pos, cs, sn);
+    latent_angles(g, freq, sm.row_pos[r], cs, sn);
     __syncthreads();
-    const int per = g.dim + g.rot_dim, D = g.kv_rank + g.rot_dim;
-    const float* q = Q + (size_t)r * g.H * per;
-    for (int i = threadIdx.x; i < g.H * per; i += blockDim.x) {
-        const int n = i / per, c = i - n * per;
-        if (c < g.dim) qn[(size_t)r * g.H * g.dim + n * g.dim + c] = from_f<T>(q[i]);
-        else qbuf[(size_t)r * g.H * D + (size_t)n * D + g.kv_rank + (c - g.dim)] = latent_rot(g, q + n * per + g.dim, c - g.dim, cs, sn);
-    }
+    latent_query_row(g, Q + (size_t)r * g.H * (g.dim + g.rot_dim), cs, sn, qn + (size_t)r * g.H * g.dim, qbuf + (size_t)r * g.H * (g.kv_rank + g.rot_dim));
 }
 
-// out[r][c] = V[r][c] * sigmoid(P[r][g_off + c]) in the compute type (gate = 0: a plain conversion): the operand of W_o
+// out[r][c] = V[r][c] * gate in the compute type: the operand of W_o
 template <typename T>
-__global__ void lp_latent_gate_kernel(const float* __restrict__ V, const float* __restrict__ P, int ldp, int g_off, int gate, int n, int R,
-                                      T* __restrict__ out) {
+__global__ void lp_latent_gate_kernel(LatentGeom g, const float* __restrict__ V, const float* __restrict__ P, int ldp, int R, T* __restrict__ out) {
+    const int n = g.H * g.vdim;
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (size_t)R * n) return;
     const int r = (int)(i / n), c = (int)(i - (size_t)r * n);
-    const float v = V[i];
-    out[i] = from_f<T>(gate ? v * sigmoid_f(P[(size_t)r * ldp + g_off + c]) : v);
+    out[i] = from_f<T>(V[i] * latent_gate(g, P + (size_t)r * ldp, c));
+}
+
+// ------------------------------------------------------------------------------------------------ few rows, one token per run (decoding)
+// Three kernels take a layer from its input projection to the operand of W_o: the query into the latent (with the rotations and the cache
+// row), the attention with the keys cut into splits and all heads of a row on the same staged rows, and the merge of the splits with W_uv
+// and the gate.  Everything between the two products is f32.
+
+// Lanes that share one output of a per-head product of length K: the smallest power of two with VN values each, at most a warp
+__host__ __device__ inline int latent_lanes(int K, int VN) {
+    int l = 1;
+    while (l < 32 && l * VN < K) l <<= 1;
+    return l;
+}
+// acc[i] = w . rows[i] over K values, summed over the `lanes` neighbouring lanes of the output (sub = place among them)
+template <typename T>
+__device__ __forceinline__ void latent_dot(const T* __restrict__ w, const float* rows, int ld, int nr, int K, int lanes, int sub, bool live, float* acc) {
+    constexpr int VN = Vec8<T>::N;
+#pragma unroll
+    for (int i = 0; i < GV_ROWS; i++) acc[i] = 0.0f;
+    if (live) {
+#pragma unroll 2
+        for (int k = sub * VN; k < K; k += lanes * VN) {
+            float wv[VN];
+            Vec8<T>::load(w + k, wv);
+#pragma unroll
+            for (int i = 0; i < GV_ROWS; i++) {
+                if (i < nr) {
+#pragma unroll
+                    for (int e = 0; e < VN; e++) acc[i] = fmaf(wv[e], rows[(size_t)i * ld + k + e], acc[i]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < GV_ROWS; i++)
+        if (i < nr)
+            for (int o = lanes >> 1; o > 0; o >>= 1) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], o);
+}
+
+// Blocks [0, H nch): head n, a chunk of latent columns of all rows: qbuf[r][n][j] = W_uk[n]^T[j] . q_plain (ukT [H][kv_rank][dim]); the
+// chunk 0 of a head also writes the head's rotated parts.  Blocks behind them (one per row, only with a W_dkv of the layer's own): the
+// row's cache row.  Q: f32 queries [R][ldq], per head [dim | rot_dim].
+template <typename T>
+__global__ void __launch_bounds__(256) lp_latent_absorb_kernel(StepMeta sm, LatentGeom g, const float* __restrict__ Q, int ldq, const float* __restrict__ P, int ldp,
+                                                               const T* __restrict__ ukT, const float* __restrict__ kvw, const double* __restrict__ freq,
+                                                               float* __restrict__ qbuf, int R, int nch) {
+    extern __shared__ float la_sm[];     // product blocks: [R][dim] plain queries; [rot_n] angles
+    __shared__ float red[33];
+    const int per = g.dim + g.rot_dim, D = g.kv_rank + g.rot_dim;
+    if ((int)blockIdx.x >= g.H * nch) {
+        const int r = blockIdx.x - g.H * nch;
+        const float* p = P + (size_t)r * ldp;
+        float* cs = la_sm;
+        float* sn = la_sm + g.rot_n / 2;
+        latent_angles(g, freq, sm.row_pos[r], cs, sn);
+        const float sk = block_sum_sq(p + g.kv_off, g.kv_rank, red);
+        latent_cache_row(g, sm, r, p, sk, kvw, cs, sn);
+        return;
+    }
+    constexpr int VN = Vec8<T>::N;
+    const int n = blockIdx.x / nch, ch = blockIdx.x - n * nch;
+    const int lanes = latent_lanes(g.dim, VN), cols = 8 * (32 / lanes);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane % lanes;
+    for (int i = threadIdx.x; i < R * g.dim; i += 256) {
+        const int r = i / g.dim, d = i - r * g.dim;
+        la_sm[i] = Q[(size_t)r * ldq + n * per + d];
+    }
+    __syncthreads();
+    const int j = ch * cols + warp * (32 / lanes) + lane / lanes;
+    for (int rb = 0; rb < R; rb += GV_ROWS) {
+        const int nr = min(GV_ROWS, R - rb);
+        float acc[GV_ROWS];
+        latent_dot<T>(ukT + ((size_t)n * g.kv_rank + j) * g.dim, la_sm + (size_t)rb * g.dim, g.dim, nr, g.dim, lanes, sub, j < g.kv_rank, acc);
+        if (sub == 0 && j < g.kv_rank) {
+#pragma unroll
+            for (int i = 0; i < GV_ROWS; i++)
+                if (i < nr) qbuf[((size_t)(rb + i) * g.H + n) * D + j] = acc[i];
+        }
+    }
+    if (ch == 0) {
+        float* cs = la_sm + (size_t)R * g.dim;
+        float* sn = cs + g.rot_n / 2;
+        for (int r = 0; r < R; r++) {
+            latent_angles(g, freq, sm.row_pos[r], cs, sn);
+            __syncthreads();
+            const float* q = Q + (size_t)r * ldq + n * per + g.dim;
+            for (int i = threadIdx.x; i < g.rot_dim; i += 256) qbuf[((size_t)r * g.H + n) * D + g.kv_rank + i] = latent_rot(g, q, i, cs, sn);
+            __syncthreads();
+        }
+    }
+}
+
+// Attention of one row over its cached rows, the keys cut into gridDim.x splits of whole 32-key tiles; a block stages its tiles in shared
+// memory (two in flight, 16-byte cp.async) and its LS_HEADS warps each take one head: a key per lane for the scores, online softmax, the
+// latent channels dealt over the lanes for the weighted sum.  part_o [R][H][splits][kv_rank] receives the unnormalised sums, part_ml
+// the running maximum and sum (an empty split: -inf, 0).
+constexpr int LS_HEADS = 8, LS_KEYS = 32;
+__host__ __device__ inline size_t latent_split_smem(int D) { return (size_t)(LS_HEADS * D + 2 * LS_KEYS * (D + 4)) * 4; }
+template <int VCH>
+__global__ void __launch_bounds__(32 * LS_HEADS) lp_latent_split_kernel(StepMeta sm, AttnGeom a, const float* __restrict__ qbuf, float* __restrict__ part_o,
+                                                                        float* __restrict__ part_ml) {
+    extern __shared__ __align__(16) float ls_sm[];
+    const int D = a.dim, pitch = D + 4;
+    float* qs = ls_sm;                         // [LS_HEADS][D]
+    float* ks = ls_sm + LS_HEADS * D;          // [2][LS_KEYS][pitch]
+    const int split = blockIdx.x, splits = gridDim.x, r = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h = blockIdx.z * LS_HEADS + warp;
+    const int i = sm.row_pos[r], lo = attn_lo(a, i);
+    const float* rows = reinterpret_cast<const float*>(sm.run_kv[sm.row_run[r]] + a.kv_off);
+    const int tiles = (i + 1 - lo + LS_KEYS - 1) / LS_KEYS, each = (tiles + splits - 1) / splits;
+    const int t_beg = min(tiles, split * each), t_end = min(tiles, t_beg + each);
+    const int vec = D / 4;
+    auto stage = [&](int t, int buf) {
+        const int j0 = lo + t * LS_KEYS;
+        for (int u = threadIdx.x; u < LS_KEYS * vec; u += 32 * LS_HEADS) {
+            const int key = u / vec, c = (u - key * vec) * 4, j = j0 + key;
+            cp_async16(smem_u32(ks + ((size_t)buf * LS_KEYS + key) * pitch + c), rows + (size_t)min(j, i) * D + c, j <= i ? 16u : 0u);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (t_beg < t_end) {
+        stage(t_beg, 0);
+        if (h < a.H)
+            for (int d = lane * 4; d < D; d += 128)
+                *reinterpret_cast<float4*>(qs + warp * D + d) = *reinterpret_cast<const float4*>(qbuf + ((size_t)r * a.H + h) * D + d);
+    }
+    float m = -INFINITY, l = 0.0f, acc[VCH];
+#pragma unroll
+    for (int c = 0; c < VCH; c++) acc[c] = 0.0f;
+    for (int t = t_beg; t < t_end; t++) {
+        const int buf = (t - t_beg) & 1;
+        if (t + 1 < t_end) {
+            stage(t + 1, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (h < a.H) {
+            const float* kt = ks + (size_t)buf * LS_KEYS * pitch;
+            const int j = lo + t * LS_KEYS + lane;
+            const float* kr = kt + (size_t)lane * pitch;
+            const float* q = qs + warp * D;
+            float s0 = 0.0f, s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
+#pragma unroll 8
+            for (int d = 0; d < D; d += 4) {
+                const float4 kv = *reinterpret_cast<const float4*>(kr + d), qv = *reinterpret_cast<const float4*>(q + d);
+                s0 = fmaf(qv.x, kv.x, s0);
+                s1 = fmaf(qv.y, kv.y, s1);
+                s2 = fmaf(qv.z, kv.z, s2);
+                s3 = fmaf(qv.w, kv.w, s3);
+            }
+            const float s = j <= i ? ((s0 + s1) + (s2 + s3)) * a.scale : -INFINITY;
+            const float mn = fmaxf(m, wmax(s));       // (a tile of the split holds a visible key: mn is finite)
+            const float p = expf(s - mn), corr = expf(m - mn);
+            l = l * corr + wsum(p);
+            m = mn;
+#pragma unroll
+            for (int c = 0; c < VCH; c++) acc[c] *= corr;
+#pragma unroll 8
+            for (int k = 0; k < LS_KEYS; k++) {
+                const float pk = __shfl_sync(0xffffffffu, p, k);
+#pragma unroll
+                for (int c = 0; c < VCH; c++) {
+                    const int chn = c * 32 + lane;
+                    if (chn < a.vdim) acc[c] = fmaf(pk, kt[(size_t)k * pitch + chn], acc[c]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (h >= a.H) return;
+    const size_t at = ((size_t)r * a.H + h) * splits + split;
+    if (lane == 0) {
+        part_ml[2 * at] = m;
+        part_ml[2 * at + 1] = l;
+    }
+    if (t_beg < t_end) {
+#pragma unroll
+        for (int c = 0; c < VCH; c++)
+            if (c * 32 + lane < a.vdim) part_o[at * a.vdim + c * 32 + lane] = acc[c];
+    }
+}
+
+// The splits' parts of a head's rows summed into the latent (shared memory, f32), then a chunk of the head's value columns: W_uv[n] times
+// the latent, times the gate, in the compute type: out[r][n vdim + c].
+template <typename T>
+__global__ void __launch_bounds__(256) lp_latent_merge_kernel(LatentGeom g, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
+                                                              const T* __restrict__ uv, const float* __restrict__ P, int ldp, T* __restrict__ out, int R, int nch) {
+    extern __shared__ float lm_sm[];
+    float* lat = lm_sm;                                  // [R][kv_rank]
+    float* wgt = lm_sm + (size_t)R * g.kv_rank;          // [R][splits]
+    constexpr int VN = Vec8<T>::N;
+    const int n = blockIdx.x / nch, ch = blockIdx.x - n * nch, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int r = warp; r < R; r += 8) {                  // a warp per row: the splits' weights, their sum taken off
+        const float* ml = part_ml + ((size_t)r * g.H + n) * splits * 2;
+        float M = -INFINITY, L = 0.0f;
+        for (int s = lane; s < splits; s += 32) M = fmaxf(M, ml[2 * s]);
+        M = wmax(M);
+        for (int s = lane; s < splits; s += 32) L = fmaf(ml[2 * s + 1], expf(ml[2 * s] - M), L);
+        L = wsum(L);
+        for (int s = lane; s < splits; s += 32) wgt[r * splits + s] = expf(ml[2 * s] - M) / L;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < R * g.kv_rank; i += 256) {
+        const int r = i / g.kv_rank, c = i - r * g.kv_rank;
+        const float* po = part_o + ((size_t)r * g.H + n) * splits * g.kv_rank + c;
+        const float* w = wgt + r * splits;
+        float acc = 0.0f;
+#pragma unroll 8
+        for (int s = 0; s < splits; s++)
+            if (w[s] > 0.0f) acc = fmaf(w[s], po[(size_t)s * g.kv_rank], acc);       // (an empty split has written nothing)
+        lat[i] = acc;
+    }
+    __syncthreads();
+    const int lanes = latent_lanes(g.kv_rank, VN), cols = 8 * (32 / lanes), sub = lane % lanes;
+    const int c = ch * cols + warp * (32 / lanes) + lane / lanes;
+    for (int rb = 0; rb < R; rb += GV_ROWS) {
+        const int nr = min(GV_ROWS, R - rb);
+        float acc[GV_ROWS];
+        latent_dot<T>(uv + ((size_t)n * g.vdim + c) * g.kv_rank, lat + (size_t)rb * g.kv_rank, g.kv_rank, nr, g.kv_rank, lanes, sub, c < g.vdim, acc);
+        if (sub == 0 && c < g.vdim) {
+#pragma unroll
+            for (int i = 0; i < GV_ROWS; i++)
+                if (i < nr) {
+                    const int r = rb + i, o = n * g.vdim + c;
+                    out[(size_t)r * g.H * g.vdim + o] = from_f<T>(acc[i] * latent_gate(g, P + (size_t)r * ldp, o));
+                }
+        }
+    }
 }

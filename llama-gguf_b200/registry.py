@@ -29,7 +29,12 @@ def _marosun(path, **kw):
     return marosun.load(path, **kw)
 
 
-LOADERS = {"Lazilorn": _lazilorn, "Mefurax": _mefurax, "Madudra": _madudra, "Marosun": _marosun}
+def _fizesun(path, **kw):
+    from . import fizesun
+    return fizesun.load(path, **kw)
+
+
+LOADERS = {"Lazilorn": _lazilorn, "Mefurax": _mefurax, "Madudra": _madudra, "Marosun": _marosun, "Fizesun": _fizesun}
 
 
 def architecture_of(path):
