@@ -1,9 +1,10 @@
-"""bench.py --design lazilorn | mefurax | madudra | marosun: prefill and decode throughput of a layer-program design at sizes that resemble a real model's
+"""bench.py --design lazilorn | mefurax | madudra | marosun | fizesun: prefill and decode throughput of a layer-program design at sizes that resemble a real model's
 layers (random weights), beside the library's closest existing model -- a llama-architecture transformer of the same width, depth
 and parameter count in Q8_0 blocks (the densest weight type its tensor-core prompt path takes); Mefurax also beside Lazilorn at
 the same width and depth (the other bf16 layer program, whose attention and GEMM kernels it shares); Madudra beside Lazilorn (the
 other hybrid of attention and recurrent scans) and Mefurax (the other mixture of experts) at the same width and depth; Marosun beside
-the same two (Lazilorn: attention beside a matrix memory; Mefurax: softmax mixers with rotation and experts).
+the same two (Lazilorn: attention beside a matrix memory; Mefurax: softmax mixers with rotation and experts); Fizesun beside Madudra (the other latent attention) and Mefurax (the other mixture with an
+always-on expert) at the same width and as many layer runs.
 
 Per size and model: prompt tokens/s for one prompt of --prefill-len tokens, decode tokens/s at batch 1 and at --batch sequences
 after prompts of --prompt-len tokens.  Every number is host wall clock around the library call (each call ends with a stream
@@ -115,6 +116,29 @@ def marosun_config(s, span=1024):
     return {"architecture": "Marosun", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "layers": layers}
 
 
+FIZESUN_SIZES = {
+    # name: width, layers (D = dense xIELU, M = mixture of clamped gated experts beside a gated shared one; every mixer latent attention), the
+    # repeated range (start, stop, times): as many layer runs as the other designs have layers, attention heads, dense ff, experts /
+    # chosen / expert ff / shared ff
+    "w1024": dict(width=1024, pattern="DMMDM", loop=(1, 2, 2), heads=8, ff=4096, experts=8, top=2, eff=1024, sff=1024, vocab=32000),
+    "w2048": dict(width=2048, pattern="DMMDMMM", loop=(1, 2, 2), heads=16, ff=8192, experts=8, top=2, eff=2048, sff=2048, vocab=32000),
+}
+
+
+def fizesun_config(s):
+    # heads and cached row as in madudra_config: 64 + 32 query / key and 128 value channels, 96 latent + 32 rotated floats per position
+    layers = []
+    for ch in s["pattern"]:
+        mlp = {"kind": "dense", "ff": s["ff"]} if ch == "D" else {"kind": "moe", "router": {"experts": s["experts"], "top": s["top"]},
+                                                                  "expert": {"ff": s["eff"], "limit": 7.0}, "shared": {"ff": s["sff"], "limit": 7.0}}
+        layers.append({"type": "latent_attention", "mlp": mlp,
+                       "mixer": {"heads": s["heads"], "dim": 64, "rot_dim": 32, "vdim": 128, "kv_rank": 96, "scale": 96 ** -0.5,
+                                 "rot": {"dims": 32, "base": 10000.0}}})
+    a, b, t = s["loop"]
+    return {"architecture": "Fizesun", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "canon": {"taps": 4},
+            "loop": {"start": a, "stop": b, "times": t}, "layers": layers}
+
+
 def lazilorn_feeder(cfg, seed, tensor_shapes=None):
     """upload(name, type, ne, data) for every tensor of cfg: bf16 bit patterns of N(0, 1/fan_in) matrices, f32 vectors."""
     import llama_gguf_b200 as B
@@ -131,11 +155,13 @@ def lazilorn_feeder(cfg, seed, tensor_shapes=None):
                      "out": lambda: np.ones(shape)}[last]()
                 upload(name, B.F32, list(reversed(shape)), np.ascontiguousarray(a, dtype=np.float32))
                 continue
-            if len(shape) == 2 and last != "conv" and name != "loop.step":
+            if len(shape) == 2 and last not in ("conv", "canon1", "canon2") and name != "loop.step":
                 a = rng.standard_normal(shape, dtype=np.float32) * np.float32(1.0 / np.sqrt(shape[-1]))
                 upload(name, B.BF16, list(reversed(shape)), bf16_bits(a).reshape(shape))
                 continue
-            if last == "conv":
+            if last in ("canon1", "canon2"):
+                a = 0.3 * rng.standard_normal(shape)
+            elif last == "conv":
                 a = 0.5 * rng.standard_normal(shape)
             elif name.endswith("f.b"):
                 a = rng.uniform(1.0, 4.0, shape)
@@ -152,8 +178,8 @@ def lazilorn_feeder(cfg, seed, tensor_shapes=None):
 
 
 def design_module(cfg):
-    from llama_gguf_b200 import lazilorn, madudra, marosun, mefurax
-    return {"Lazilorn": lazilorn, "Mefurax": mefurax, "Madudra": madudra, "Marosun": marosun}[cfg["architecture"]]
+    from llama_gguf_b200 import fizesun, lazilorn, madudra, marosun, mefurax
+    return {"Lazilorn": lazilorn, "Mefurax": mefurax, "Madudra": madudra, "Marosun": marosun, "Fizesun": fizesun}[cfg["architecture"]]
 
 
 def n_params(cfg):
@@ -247,6 +273,8 @@ def main(args):
         return main_madudra(args)
     if args.design == "marosun":
         return main_marosun(args)
+    if args.design == "fizesun":
+        return main_fizesun(args)
     sizes = [x for x in (args.sizes.split(",") if args.sizes else SIZES) if x]
     max_seq = max(args.prefill_len, args.prompt_len + args.warmup + args.steps + 8) + 8
     res = {}
@@ -336,4 +364,26 @@ def main_marosun(args):
     print(json.dumps({"bench": "design", "design": "marosun", "unit": "tok/s", "prefill_len": args.prefill_len, "prompt_len": args.prompt_len,
                       "batch": args.batch, "steps": args.steps, "warmup": args.warmup, "timing": "host wall clock around the library calls",
                       "dtype": "bf16 (marosun, lazilorn, mefurax at the same width and depth)", "data": "synthetic", "sizes": res}))
+    return 0
+
+
+def main_fizesun(args):
+    sizes = [x for x in (args.sizes.split(",") if args.sizes else FIZESUN_SIZES) if x]
+    max_seq = max(args.prefill_len, args.prompt_len + args.warmup + args.steps + 8) + 8
+    res = {}
+    for name in sizes:
+        s = FIZESUN_SIZES[name]
+        cfg = fizesun_config(s)
+        params = n_params(cfg)
+        active = params - s["pattern"].count("M") * (s["experts"] - s["top"]) * 3 * s["width"] * s["eff"]
+        r = {"params_without_embedding": params, "active_params_without_embedding": active, "layers": s["pattern"], "loop": list(s["loop"]),
+             "fizesun_bf16": bench_lazilorn(cfg, args, max_seq)}
+        print(name, json.dumps(r), file=sys.stderr, flush=True)
+        r["madudra_bf16"] = bench_lazilorn(madudra_config(MADUDRA_SIZES[name]), args, max_seq)
+        r["mefurax_bf16"] = bench_lazilorn(mefurax_config(MEFURAX_SIZES[name]), args, max_seq)
+        res[name] = r
+        print(name, json.dumps(r), file=sys.stderr, flush=True)
+    print(json.dumps({"bench": "design", "design": "fizesun", "unit": "tok/s", "prefill_len": args.prefill_len, "prompt_len": args.prompt_len,
+                      "batch": args.batch, "steps": args.steps, "warmup": args.warmup, "timing": "host wall clock around the library calls",
+                      "dtype": "bf16 (fizesun, madudra, mefurax at the same width and number of layer runs)", "data": "synthetic", "sizes": res}))
     return 0
