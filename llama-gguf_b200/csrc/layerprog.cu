@@ -379,7 +379,19 @@ __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict_
                   "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
                 : "r"(taddr));
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-            if (n < N) {
+            if (EPI == EPI_ADD && n < N) {   // all 32 sums are read before the first one is written
+                float old[32];
+#pragma unroll
+                for (int c = 0; c < 32; c++) {
+                    const int t = t0 + c0 + c;
+                    old[c] = t < R ? reinterpret_cast<const float*>(Y)[(size_t)t * ldy + n] : 0.0f;
+                }
+#pragma unroll
+                for (int c = 0; c < 32; c++) {
+                    const int t = t0 + c0 + c;
+                    if (t < R) reinterpret_cast<float*>(Y)[(size_t)t * ldy + n] = old[c] + (alpha * __uint_as_float(v[c]) + bn);
+                }
+            } else if (n < N) {
 #pragma unroll
                 for (int c = 0; c < 32; c++) {
                     const int t = t0 + c0 + c;
@@ -417,9 +429,43 @@ template <> struct Vec8<float> {
     }
 };
 #include "lp_rows_tail.cuh"
+
+// A warp asks for a weight row's cache lines ahead of the work that has to come first (staging, norms): the DRAM latency runs meanwhile.
+template <typename T> __device__ __forceinline__ void prefetch_row(const T* row, int K, int lane) {
+    const char* p = reinterpret_cast<const char*>(row);
+    for (size_t o = (size_t)lane * 128; o < (size_t)K * sizeof(T); o += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + o));
+}
+// acc[i] = this lane's part of w . X[i], i < NR (rows past the last are the last again: no branch between the loads, so that several
+// 16-byte weight loads are in flight)
+template <typename T, int NR> __device__ __forceinline__ void gemv_dot(const T* __restrict__ w, const T* X, size_t ldx, int nr, int K, int lane, float* acc) {
+    constexpr int VN = Vec8<T>::N;
+    const T* xr[NR];
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        acc[i] = 0.0f;
+        xr[i] = X + (size_t)min(i, nr - 1) * ldx;
+    }
+#pragma unroll(NR <= 2 ? 8 : 4)
+    for (int k = lane * VN; k < K; k += 32 * VN) {
+        float wv[VN], xv[VN];
+        Vec8<T>::load(w + k, wv);
+#pragma unroll
+        for (int i = 0; i < NR; i++) {
+            Vec8<T>::load(xr[i] + k, xv);
+#pragma unroll
+            for (int e = 0; e < VN; e++) acc[i] = fmaf(wv[e], xv[e], acc[i]);
+        }
+    }
+}
 #include "lp_input_conv.cuh"
 
-template <typename T, int EPI>
+// the row count a few-row kernel is instantiated for: 1, 2, 4 or 8 (GV_ROWS) rows per pass over the weights
+#define LP_NR_DISPATCH(R, CALL)                                                                                        \
+    do {                                                                                                               \
+        if ((R) <= 1) { CALL(1); } else if ((R) <= 2) { CALL(2); } else if ((R) <= 4) { CALL(4); } else { CALL(GV_ROWS); } \
+    } while (0)
+
+template <typename T, int EPI, int NR>
 __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, int ldx, const T* __restrict__ W, int ldw, void* __restrict__ Y,
                                                       int ldy, int R, int N, int K, float alpha, int vec_ok, int stage, RowsTail tail, int nh,
                                                       ZStride zs, const float* __restrict__ bias, float2 act) {
@@ -428,6 +474,10 @@ __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, i
     const T* X0 = X;
     const int lane = threadIdx.x & 31;
     constexpr int VN = Vec8<T>::N;
+    {
+        const int n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+        if (stage && n < N) prefetch_row(W + (size_t)n * ldw, K, lane);
+    }
     if (stage) {   // the activation rows once per block into shared memory (every warp of the block reads all of them)
         T* xs = reinterpret_cast<T*>(gv_smem);
         const int per_row = K / VN;
@@ -447,33 +497,23 @@ __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, i
         X = X0 + (size_t)z * zs.x;
         ycol = (size_t)z * zs.y + (size_t)(n - z * nh);
     }
-    for (int rb = 0; rb < R; rb += GV_ROWS) {
-        const int nr = min(GV_ROWS, R - rb);
-        float acc[GV_ROWS] = {};
+    for (int rb = 0; rb < R; rb += NR) {
+        const int nr = min(NR, R - rb);
+        float acc[NR];
         if (vec_ok) {
-#pragma unroll 4
-            for (int k = lane * VN; k < K; k += 32 * VN) {
-                float wv[VN], xv[VN];
-                Vec8<T>::load(wr + k, wv);
-#pragma unroll
-                for (int i = 0; i < GV_ROWS; i++) {
-                    if (i < nr) {
-                        Vec8<T>::load(X + (size_t)(rb + i) * ldx + k, xv);
-#pragma unroll
-                        for (int e = 0; e < VN; e++) acc[i] = fmaf(wv[e], xv[e], acc[i]);
-                    }
-                }
-            }
+            gemv_dot<T, NR>(wr, X + (size_t)rb * ldx, ldx, nr, K, lane, acc);
         } else {
+#pragma unroll
+            for (int i = 0; i < NR; i++) acc[i] = 0.0f;
             for (int k = lane; k < K; k += 32) {
                 const float wv = to_f(wr[k]);
 #pragma unroll
-                for (int i = 0; i < GV_ROWS; i++)
+                for (int i = 0; i < NR; i++)
                     if (i < nr) acc[i] = fmaf(wv, to_f(X[(size_t)(rb + i) * ldx + k]), acc[i]);
             }
         }
 #pragma unroll
-        for (int i = 0; i < GV_ROWS; i++) {
+        for (int i = 0; i < NR; i++) {
             if (i < nr) {
                 const float s = wsum(acc[i]);
                 if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + ycol, alpha * s + (bias ? bias[n] : 0.0f), act);
@@ -488,8 +528,8 @@ __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, i
 // row, times the norm weight, rounded to the compute type exactly as lp_rmsnorm_kernel does -- and then multiplies from there.
 // Every block repeats the norm (the rows are a few KB out of L2); a launch and a round trip through global memory go away.
 // ic.taps > 0 (decoding: one row per run): the normed row h becomes h + conv(h) before the rounding; every block reads the run's earlier
-// inputs, block 0 writes this position's (input_conv_row: no other block reads that ring entry).
-template <typename T, int EPI>
+// inputs, block 0 writes this position's (norm_conv_row; no other block reads that ring entry).
+template <typename T, int EPI, int NR>
 __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restrict__ X, const int* __restrict__ gather, const float* __restrict__ nw,
                                                            float eps, const T* __restrict__ W, void* __restrict__ Y, int ldy, int R, int N, int K,
                                                            float alpha, int center, T* __restrict__ hn_out, float2 act, InConv ic, StepMeta sm) {
@@ -498,7 +538,12 @@ __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restri
     __shared__ float red[8];
     __shared__ float inv_s, mean_s;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (blockIdx.x * 8 + warp < N) prefetch_row(W + (size_t)(blockIdx.x * 8 + warp) * K, K, lane);
     for (int r = 0; r < R; r++) {
+        if (ic.taps > 0) {   // (RMS norm, no gather: checked by the host)
+            norm_conv_row<T, 256>(ic, sm, r, X + (size_t)r * K, nw, K, eps, blockIdx.x == 0, xs + (size_t)r * K, nullptr);
+            continue;
+        }
         const float* xr = X + (size_t)(gather ? gather[r] : r) * K;
         float mean = 0.0f;
         if (center) {   // layer norm: the mean first
@@ -529,42 +574,27 @@ __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restri
         }
         __syncthreads();
         const float inv = inv_s;
-        const InConvRow cr = input_conv_row(ic, sm, r, blockIdx.x == 0);
         for (int k = threadIdx.x; k < K; k += 256) {
-            const float h = (xr[k] - mean) * inv * nw[k];
-            const T v = from_f<T>(ic.taps > 0 ? input_conv_step(ic, cr, K, k, h) : h);
+            const T v = from_f<T>((xr[k] - mean) * inv * nw[k]);
             xs[(size_t)r * K + k] = v;
             if (hn_out && blockIdx.x == 0) hn_out[(size_t)r * K + k] = v;   // (a later kernel of the layer reads the normed rows too)
         }
     }
     __syncthreads();
-    constexpr int VN = Vec8<T>::N;
-    for (int n = blockIdx.x * 8 + warp; n < N; n += gridDim.x * 8) {
-    const T* wr = W + (size_t)n * K;
-    for (int rb = 0; rb < R; rb += GV_ROWS) {
-        const int nr = min(GV_ROWS, R - rb);
-        float acc[GV_ROWS] = {};
-#pragma unroll 4
-        for (int k = lane * VN; k < K; k += 32 * VN) {   // (K is a multiple of VN: checked by the host)
-            float wv[VN], xv[VN];
-            Vec8<T>::load(wr + k, wv);
+    for (int n = blockIdx.x * 8 + warp; n < N; n += gridDim.x * 8) {   // (K is a multiple of VN: checked by the host)
+        const T* wr = W + (size_t)n * K;
+        for (int rb = 0; rb < R; rb += NR) {
+            const int nr = min(NR, R - rb);
+            float acc[NR];
+            gemv_dot<T, NR>(wr, xs + (size_t)rb * K, K, nr, K, lane, acc);
 #pragma unroll
-            for (int i = 0; i < GV_ROWS; i++) {
+            for (int i = 0; i < NR; i++) {
                 if (i < nr) {
-                    Vec8<T>::load(xs + (size_t)(rb + i) * K + k, xv);
-#pragma unroll
-                    for (int e = 0; e < VN; e++) acc[i] = fmaf(wv[e], xv[e], acc[i]);
+                    const float sum = wsum(acc[i]);
+                    if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + n, alpha * sum, act);
                 }
             }
         }
-#pragma unroll
-        for (int i = 0; i < GV_ROWS; i++) {
-            if (i < nr) {
-                const float sum = wsum(acc[i]);
-                if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + n, alpha * sum, act);
-            }
-        }
-    }
     }
 }
 
@@ -1472,6 +1502,10 @@ struct LpModel {
     void* xcat = nullptr;               // [rows][2 width] compute type: [x; x0] ahead of a pass of the repeated range (program.loop_in)
     float *lat_o = nullptr, *lat_ml = nullptr;   // decoding latent attention: the splits' sums and their (maximum, sum)
     size_t lat_o_floats = 0, lat_ml_floats = 0;
+    size_t* ring_offs = nullptr;        // [n_convs] rings of the input convolutions inside a state block
+    int n_convs = 0;
+    float* conv_pend = nullptr;         // [n_convs][runs][taps - 1][width]: last inputs of longer runs until the step's end
+    size_t conv_pend_bytes = 0;
     float* moe_shw = nullptr;           // [rows]: gate of the always-on expert
     int *moe_sel = nullptr, *moe_pos = nullptr, *moe_seg = nullptr;   // chosen experts per row; row of (token, choice) in expert order; {first, rows} per expert
     void* moe_xp = nullptr;             // the tokens' rows gathered in expert order, compute type
@@ -1663,12 +1697,24 @@ void gemm_t(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, i
         const size_t smem = stage ? xbytes : 0;
         const RowsTail tl = tail ? *tail : RowsTail{};
         const int nh = heads ? N : 0;
-#define LP_GV(E) launch(m, lp_gemv_kernel<T, E>, grid, block, smem, x, ldx, w, ldw, Y, ldy, R, Nall, K, alpha, vec_ok, stage, tl, nh, zs, bias, act)
+#define LP_GV(E) LP_NR_DISPATCH(R, LP_GV_##E)
+#define LP_GV_N(E, NR) launch(m, lp_gemv_kernel<T, E, NR>, grid, block, smem, x, ldx, w, ldw, Y, ldy, R, Nall, K, alpha, vec_ok, stage, tl, nh, zs, bias, act)
+#define LP_GV_EPI_STORE(NR) LP_GV_N(EPI_STORE, NR)
+#define LP_GV_EPI_ADD(NR) LP_GV_N(EPI_ADD, NR)
+#define LP_GV_EPI_GELU(NR) LP_GV_N(EPI_GELU, NR)
+#define LP_GV_EPI_XIELU(NR) LP_GV_N(EPI_XIELU, NR)
+#define LP_GV_EPI_RELU2(NR) LP_GV_N(EPI_RELU2, NR)
         if (epi == EPI_STORE) LP_GV(EPI_STORE);
         else if (epi == EPI_ADD) LP_GV(EPI_ADD);
         else if (epi == EPI_GELU) LP_GV(EPI_GELU);
         else if (epi == EPI_XIELU) LP_GV(EPI_XIELU);
         else LP_GV(EPI_RELU2);
+#undef LP_GV_EPI_STORE
+#undef LP_GV_EPI_ADD
+#undef LP_GV_EPI_GELU
+#undef LP_GV_EPI_XIELU
+#undef LP_GV_EPI_RELU2
+#undef LP_GV_N
 #undef LP_GV
         return;
     }
@@ -1723,30 +1769,34 @@ bool gemv_norm_t(LpModel* m, const float* x, const int* gather, const float* nw,
     constexpr int VN = Vec8<T>::N;
     const size_t smem = (size_t)R * K * sizeof(T);
     if (R > 2 * GV_ROWS || K % VN || ((uintptr_t)W & 15) || smem > 96 * 1024) return false;
-    static bool once[EPI_COUNT][64] = {};
+    if (epi != EPI_STORE && epi != EPI_RELU2 && epi != EPI_XIELU) return false;
+    static bool once[EPI_COUNT][GV_ROWS + 1][64] = {};
     int dev = 0;
     cudaGetDevice(&dev);
-    auto prep = [&](auto kern, int e) {
-        if (dev >= 0 && dev < 64 && once[e][dev]) return true;
+    auto prep = [&](auto kern, int e, int nr) {
+        if (dev >= 0 && dev < 64 && once[e][nr][dev]) return true;
         if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024) != cudaSuccess) {
             cudaGetLastError();
             return false;
         }
-        if (dev >= 0 && dev < 64) once[e][dev] = true;
+        if (dev >= 0 && dev < 64) once[e][nr][dev] = true;
         return true;
     };
     dim3 grid(std::min((N + 7) / 8, 4 * 148)), block(256);
     const T* w = (const T*)W;
-    if (epi == EPI_STORE) {
-        if (!prep(lp_gemv_norm_kernel<T, EPI_STORE>, 0)) return false;
-        launch(m, lp_gemv_norm_kernel<T, EPI_STORE>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm);
-    } else if (epi == EPI_RELU2) {
-        if (!prep(lp_gemv_norm_kernel<T, EPI_RELU2>, 2)) return false;
-        launch(m, lp_gemv_norm_kernel<T, EPI_RELU2>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm);
-    } else if (epi == EPI_XIELU) {
-        if (!prep(lp_gemv_norm_kernel<T, EPI_XIELU>, 4)) return false;
-        launch(m, lp_gemv_norm_kernel<T, EPI_XIELU>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm);
-    } else return false;
+#define LP_GN(E, NR)                                                                                                                       \
+    if (!prep(lp_gemv_norm_kernel<T, E, NR>, E, NR)) return false;                                                                         \
+    launch(m, lp_gemv_norm_kernel<T, E, NR>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm)
+#define LP_GN_STORE(NR) LP_GN(EPI_STORE, NR)
+#define LP_GN_RELU2(NR) LP_GN(EPI_RELU2, NR)
+#define LP_GN_XIELU(NR) LP_GN(EPI_XIELU, NR)
+    if (epi == EPI_STORE) LP_NR_DISPATCH(R, LP_GN_STORE);
+    else if (epi == EPI_RELU2) LP_NR_DISPATCH(R, LP_GN_RELU2);
+    else LP_NR_DISPATCH(R, LP_GN_XIELU);
+#undef LP_GN_STORE
+#undef LP_GN_RELU2
+#undef LP_GN_XIELU
+#undef LP_GN
     return true;
 }
 // keep: the normed rows are also wanted in `scratch` afterwards (the fused kernel then writes them out as well)
@@ -2327,9 +2377,9 @@ int lp_finalize(LpModel* m, std::string* err) {
             m->max_qrank = std::max(m->max_qrank, a.q_rank);
             // decoding kernels: 16-byte loads of cached rows and weights, the rows in shared memory, two key tiles too
             const int vn = m->f32 ? 4 : 8;
-            const size_t part = (size_t)2 * GV_ROWS * (std::max(a.dim, a.kv_rank) + std::max(64, a.rot.dims)) * 4;
-            if (D % 4 == 0 && a.kv_rank % vn == 0 && a.dim % vn == 0 && latent_split_smem((int)D) <= 200 * 1024 && part <= 96 * 1024) {
-                for (int r = 1; r <= 2 * GV_ROWS; r++) L.lat_splits = std::max(L.lat_splits, r * latent_splits(r, a.heads));
+            const size_t part = (size_t)LS_ROWS * (std::max(a.dim, a.kv_rank) + std::max(64, a.rot.dims)) * 4;
+            if (D % 4 == 0 && a.kv_rank % vn == 0 && a.dim % vn == 0 && latent_split_smem((int)D) <= 200 * 1024 && part <= 190 * 1024) {
+                for (int r = 1; r <= LS_ROWS; r++) L.lat_splits = std::max(L.lat_splits, r * latent_splits(r, a.heads));
                 m->lat_o_floats = std::max(m->lat_o_floats, (size_t)L.lat_splits * a.heads * a.kv_rank);
                 m->lat_ml_floats = std::max(m->lat_ml_floats, (size_t)L.lat_splits * a.heads * 2);
             }
@@ -2393,7 +2443,16 @@ int lp_finalize(LpModel* m, std::string* err) {
             const bool ff = L.d.ff_kind == B200_FF_MOE || L.d.ff > 0;
             for (int q = 0; q < (ff ? 2 : 1); q++) {
                 L.ic[q].taps = p.in_conv;
-                if ((rc = need_vec(m, pre + "canon" + std::to_string(q + 1), W * p.in_conv, &L.ic[q].w, err))) return rc;
+                const std::string nm = pre + "canon" + std::to_string(q + 1);
+                const float* cw;
+                if ((rc = need_vec(m, nm, W * p.in_conv, &cw, err))) return rc;
+                Tensor t = *find(m, nm);      // [width][taps] -> [taps][width]
+                LCU_ALLOC(cudaMalloc(&t.d, up16(t.bytes)));
+                lp_transpose_heads_kernel<float><<<(unsigned)((W * p.in_conv + 255) / 256), 256>>>(cw, (float*)t.d, 1, (int)W, p.in_conv);
+                LCU(cudaDeviceSynchronize());
+                cudaFree(m->tensors[nm].d);
+                m->tensors[nm] = t;
+                L.ic[q].w = (const float*)t.d;
                 L.ic[q].ring_off = L.rec_bytes;
                 if (p.in_conv > 1) L.rec_bytes += up16((size_t)p.in_conv * W * 4);
             }
@@ -2533,7 +2592,7 @@ int lp_finalize(LpModel* m, std::string* err) {
     if (m->lat_o_floats > 0) {
         LCU_ALLOC(cudaMalloc((void**)&m->lat_o, up16(m->lat_o_floats * 4)));
         LCU_ALLOC(cudaMalloc((void**)&m->lat_ml, up16(m->lat_ml_floats * 4)));
-        const int sb = 200 * 1024, pb = 96 * 1024;
+        const int sb = 200 * 1024, pb = 200 * 1024;
         LCU(cudaFuncSetAttribute(lp_latent_split_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
         LCU(cudaFuncSetAttribute(lp_latent_split_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
         LCU(cudaFuncSetAttribute(lp_latent_split_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
@@ -2571,6 +2630,15 @@ int lp_finalize(LpModel* m, std::string* err) {
         if (L.d.mixer == B200_MIX_SOFTMAX_ATTN || L.d.mixer == B200_MIX_ATTN_RECURRENT)
             m->kv_bytes_per_pos += (size_t)L.d.sattn.kv_heads * (L.d.sattn.dim + L.d.sattn.vdim) * 4;
         if (L.d.mixer == B200_MIX_LATENT_ATTN && L.d.latent.kv_from < 0) m->kv_bytes_per_pos += (size_t)(L.d.latent.kv_rank + L.d.latent.rot_dim) * 4;
+    }
+    if (p.in_conv > 1) {   // the rings of all layer runs: convolution i of the order in which a step meets them
+        std::vector<size_t> offs;
+        for (size_t r = 0; r < m->runs.size(); r++)
+            for (const InConv& ic : m->plan[m->runs[r]].ic)
+                if (ic.taps > 0) offs.push_back(m->run_rec_off[r] + ic.ring_off);
+        LCU_ALLOC(cudaMalloc((void**)&m->ring_offs, up16(offs.size() * sizeof(size_t))));
+        LCU(cudaMemcpy(m->ring_offs, offs.data(), offs.size() * sizeof(size_t), cudaMemcpyHostToDevice));
+        m->n_convs = (int)offs.size();
     }
     m->slot_kv_bytes = std::max<size_t>(kv, 256);
     m->slot_rec_bytes = std::max<size_t>(rec, 256);
@@ -2621,7 +2689,7 @@ void lp_destroy(LpModel* m) {
     for (void* ptr : {(void*)m->inv_freq, (void*)m->d_meta, (void*)m->x, (void*)m->P, (void*)m->qbuf, (void*)m->O, (void*)m->conv, (void*)m->logits,
                       m->hn, m->act_a, m->hw, (void*)m->pick, (void*)m->taps, (void*)m->glin_carry, (void*)m->y, (void*)m->vsrc, (void*)m->moe_w, (void*)m->moe_selw,
                       (void*)m->moe_sel, (void*)m->moe_pos, (void*)m->moe_seg, m->moe_xp, (void*)m->moe_yp, (void*)m->xs, m->cq, (void*)m->vrot, m->xcat,
-                      (void*)m->lat_o, (void*)m->lat_ml, (void*)m->moe_shw})
+                      (void*)m->lat_o, (void*)m->lat_ml, (void*)m->moe_shw, (void*)m->ring_offs, (void*)m->conv_pend})
         cudaFree(ptr);
     if (m->h_meta) cudaFreeHost(m->h_meta);
     if (m->h_logits) cudaFreeHost(m->h_logits);
@@ -2751,6 +2819,30 @@ bool attn_tile(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int ldp, int 
     return attn_tile_launch<128, 256>(m, sm, ag, ldp, n_runs, max_len);
 }
 
+// The same for latent attention (lp_latent_tile_kernel): cached rows a multiple of 16 wide up to 320, latents a multiple of 8 up to 256
+template <int DK, int DV>
+bool latent_tile_launch(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int n_runs, int max_len) {
+    static bool once[64] = {};
+    int dev = 0;
+    cudaGetDevice(&dev);
+    if (dev < 0 || dev >= 64 || !once[dev]) {
+        if (cudaFuncSetAttribute(lp_latent_tile_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_tile_smem<DK>()) != cudaSuccess) {
+            cudaGetLastError();
+            return false;
+        }
+        if (dev >= 0 && dev < 64) once[dev] = true;
+    }
+    launch(m, lp_latent_tile_kernel<DK, DV>, dim3((unsigned)(((size_t)max_len * ag.H + LT_ROWS - 1) / LT_ROWS), n_runs), dim3(256), latent_tile_smem<DK>(), sm, ag,
+           (const float*)m->qbuf, (bf16*)m->act_a);
+    return true;
+}
+bool latent_tile(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int n_runs, int max_len) {
+    if (m->f32 || !m->use_attn_tile || max_len < 16 || ag.dim % 16 || ag.vdim % 8) return false;
+    if (ag.dim <= 128 && ag.vdim <= 128) return latent_tile_launch<128, 128>(m, sm, ag, n_runs, max_len);
+    if (ag.dim <= 320 && ag.vdim <= 256) return latent_tile_launch<320, 256>(m, sm, ag, n_runs, max_len);
+    return false;
+}
+
 // Into how many segments the gated linear memory cuts the runs of a step (1 = whole runs): only long runs, and only while whole runs
 // would leave SMs idle (a block per 16 to 64 columns of a head's state and run); segments of at least 64 tokens.
 int glin_segments(const LpModel* m, int H, int dim, int vdim, int n_runs, int max_len) {
@@ -2855,8 +2947,9 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         else launch(m, lp_postnorm_kernel<bf16>, dim3(R), dim3(256), 0, m->x, y, w, (bf16*)m->hn, W, p.residual_alpha, p.norm_eps);
     };
     // What sublayer `sub` reads in a program with input convolutions, h + conv(h) with h = norm(x), in the compute type -> m->hn.  One
-    // token per run: one block per row, which also moves the ring on and, given `rt`, routes; longer runs: the ring after the readers.
+    // token per run: one block per row, which also moves the ring on and, given `rt`, routes; longer runs: the rings move at the step's end.
     const bool ring_step = max_len == 1 && m->use_fuse;
+    int conv_at = 0;
     auto conv_in = [&](const InConv& ic0, const float* nw, const StepRoute& rt) {
         InConv ic = ic0;
         ic.ring_off += m->run_rec_off[cur_run];
@@ -2866,6 +2959,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             else launch(m, lp_norm_conv_step_kernel<bf16>, dim3(R), dim3(512), smem, sm, ic, (const float*)m->x, nw, W, p.norm_eps, (bf16*)m->hn, rt);
             return;
         }
+        if (ic.taps > 1) ic.pend = m->conv_pend + (size_t)conv_at * n_runs * (ic.taps - 1) * W;
         const dim3 grid((R + NC_ROWS - 1) / NC_ROWS), block(256);
         const size_t smem = (size_t)(NC_ROWS + ic.taps - 1) * 4;
 #define LP_NC(T, V, TP) launch(m, lp_norm_conv_rows_kernel<T, V, TP>, grid, block, smem, sm, ic, (const float*)m->x, nw, W, p.norm_eps, (T*)m->hn, R)
@@ -2878,12 +2972,12 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         if (m->f32) { LP_NC_T(float); } else { LP_NC_T(bf16); }
 #undef LP_NC_T
 #undef LP_NC
-        if (ic.taps > 1) launch(m, lp_norm_conv_tail_kernel, dim3(n_runs, ic.taps - 1), dim3(256), 0, sm, ic, (const float*)m->x, nw, W, p.norm_eps);
+        conv_at++;
     };
     auto project_in = [&](const float* add, const float* nw, const void* Wm, int N, void* Y, int ldy, int epi) {
         const float2 act = cur->act2;
         if (p.in_conv > 0) {
-            if (ring_step && R <= m->conv_fuse_rows) {   // the norm and the convolution inside the projection
+            if (ring_step && R <= m->conv_fuse_rows && W <= 2048) {   // the norm and the convolution inside the projection
                 InConv ic = cur->ic[sub];
                 ic.ring_off += m->run_rec_off[cur_run];
                 if (m->f32 ? gemv_norm_t<float>(m, m->x, nullptr, nw, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, act, ic, sm)
@@ -2932,9 +3026,14 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         LayerPlan& L = m->plan[m->runs[run]];
         const float* add = m->run_pass[run] >= 0 ? loop_step + (size_t)m->run_pass[run] * W : nullptr;
         if (add && p.loop_in) {   // ahead of a pass: x <- loop.in [x; x0] + the pass's vector
-            const unsigned nb = (unsigned)(((size_t)R * W + 255) / 256);
-            if (m->f32) launch(m, lp_cast_rows_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->x, W, (float*)m->xcat, 2 * W, R);
-            else launch(m, lp_cast_rows_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->x, W, (bf16*)m->xcat, 2 * W, R);
+            const dim3 g4(R, (W / 4 + 255) / 256), g1(R, (W + 255) / 256);
+            if (m->f32) {
+                if (W % 4 == 0) launch(m, lp_cast_rows_kernel<float, 4>, g4, dim3(256), 0, (const float*)m->x, W, (float*)m->xcat, 2 * W);
+                else launch(m, lp_cast_rows_kernel<float, 1>, g1, dim3(256), 0, (const float*)m->x, W, (float*)m->xcat, 2 * W);
+            } else {
+                if (W % 4 == 0) launch(m, lp_cast_rows_kernel<bf16, 4>, g4, dim3(256), 0, (const float*)m->x, W, (bf16*)m->xcat, 2 * W);
+                else launch(m, lp_cast_rows_kernel<bf16, 1>, g1, dim3(256), 0, (const float*)m->x, W, (bf16*)m->xcat, 2 * W);
+            }
             gemm(m, m->xcat, 2 * W, find(m, "loop.in")->d, W, 2 * W, m->x, W, R, 1.0f, EPI_STORE, nullptr, add);
             add = nullptr;
         }
@@ -3057,7 +3156,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             const int per = a.dim + a.rot_dim, D = a.kv_rank + a.rot_dim, nv = a.heads * a.vdim;
             const bool direct = a.q_rank == 0, own = a.kv_from < 0;
             // one token per run, few rows: absorb / split attention / merge (lp_latent_attn.cuh)
-            const bool split = m->use_fuse && m->use_lat_split && max_len == 1 && R <= 2 * GV_ROWS && L.lat_splits > 0;
+            const bool split = m->use_fuse && m->use_lat_split && max_len == 1 && R <= LS_ROWS && L.lat_splits > 0;
             if (!(split && direct)) {
                 if (m->f32) launch(m, lp_latent_prep_kernel<float>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (float*)m->cq, (float*)m->act_a, m->qbuf);
                 else launch(m, lp_latent_prep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (bf16*)m->cq, (bf16*)m->act_a, m->qbuf);
@@ -3074,7 +3173,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                 const int uk_cols = 8 * (32 / latent_lanes(a.dim, vn)), uk_ch = (a.kv_rank + uk_cols - 1) / uk_cols;
                 const int uv_cols = 8 * (32 / latent_lanes(a.kv_rank, vn)), uv_ch = (a.vdim + uv_cols - 1) / uv_cols;
                 const dim3 agrid(a.heads * uk_ch + (direct && own ? R : 0)), sgrid(splits, R, (a.heads + LS_HEADS - 1) / LS_HEADS), ugrid(a.heads * uv_ch);
-                const size_t asm_ = (size_t)(R * a.dim + lg.rot_n) * 4, usm = (size_t)R * (a.kv_rank + splits) * 4;
+                const size_t asm_ = (size_t)(R * a.dim + lg.rot_n) * 4, usm = ((size_t)R * (a.kv_rank + splits) + 1024 + 4) * 4;
                 if (m->f32) launch(m, lp_latent_absorb_kernel<float>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const float*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
                 else launch(m, lp_latent_absorb_kernel<bf16>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const bf16*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
 #define LP_LS(V) launch(m, lp_latent_split_kernel<V>, sgrid, dim3(32 * LS_HEADS), latent_split_smem(D), sm, ag, (const float*)m->qbuf, m->lat_o, m->lat_ml)
@@ -3088,11 +3187,12 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                     else launch(m, lp_latent_qprep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->O, L.rot_freq, (bf16*)m->act_a, m->qbuf);
                 }
                 gemm_heads(m, m->act_a, a.heads * a.dim, a.dim, L.w_ukT, a.heads, a.kv_rank, a.dim, m->qbuf, a.heads * D, D, R);
-                if (!attn_tile(m, sm, ag, L.n_in, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
+                if (!latent_tile(m, sm, ag, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
                 gemm_heads(m, m->act_a, a.heads * a.kv_rank, a.kv_rank, L.w_uv, a.heads, a.vdim, a.kv_rank, m->O, nv, a.vdim, R);
-                const unsigned nb = (unsigned)(((size_t)R * nv + 255) / 256);
-                if (m->f32) launch(m, lp_latent_gate_kernel<float>, dim3(nb), dim3(256), 0, lg, (const float*)m->O, (const float*)m->P, L.n_in, R, (float*)m->act_a);
-                else launch(m, lp_latent_gate_kernel<bf16>, dim3(nb), dim3(256), 0, lg, (const float*)m->O, (const float*)m->P, L.n_in, R, (bf16*)m->act_a);
+#define LP_LG(T, N) launch(m, lp_latent_gate_kernel<T, N>, dim3(R), dim3(256), 0, lg, (const float*)m->O, (const float*)m->P, L.n_in, (T*)m->act_a)
+                if (m->f32) { if (a.vdim % 4) LP_LG(float, 1); else LP_LG(float, 4); }
+                else { if (a.vdim % 4) LP_LG(bf16, 1); else LP_LG(bf16, 4); }
+#undef LP_LG
             }
             project_out(m->act_a, nv, L.wo, L.norm1, moe_next);
         } else if (L.d.mixer == B200_MIX_STATE_SPACE) {
@@ -3155,7 +3255,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             bool routed = par || moe_next != nullptr;
             if (p.in_conv > 0) {
                 StepRoute rt{};
-                if (ring_step && R <= 2 * GV_ROWS) {       // few rows: the block that norms a row also routes it
+                if (ring_step && R <= LS_ROWS) {       // few rows: the block that norms a row also routes it
                     rt.router = L.w_up; rt.bias = L.router_bias; rt.rows = rrows; rt.E = e.experts; rt.top = e.top; rt.mode = e.route; rt.scale = e.route_scale;
                     rt.logits = m->P; rt.wts = m->moe_w; rt.sel = m->moe_sel; rt.selw = m->moe_selw; rt.shw = shw;
                     routed = true;
@@ -3281,6 +3381,8 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         if (taps_len > 0) cudaMemcpyAsync(m->taps + run * (size_t)taps_len * W, m->x, (size_t)taps_len * W * 4, cudaMemcpyDeviceToDevice, m->stream);
     }
     if (streams) boundary(nullptr, nullptr, m->x);   // the head reads the sum of the copies
+    if (p.in_conv > 1 && !ring_step)
+        launch(m, lp_ring_commit_kernel, dim3(m->n_convs, n_runs, p.in_conv - 1), dim3(256), 0, sm, (const size_t*)m->ring_offs, (const float*)m->conv_pend, p.in_conv, W);
     if (head) {
         norm_gemm(m, m->x, nullptr, sm.want, (const float*)find(m, "final.norm")->d, m->hw, find(m, "head")->d, p.vocab, m->logits, p.vocab, n_want,
                   p.logit_scale, EPI_STORE);
@@ -3395,6 +3497,15 @@ int lp_step(LpModel* m, int n_runs, const int* seqs, const int* pos0, const int*
             m->glin_carry_bytes = 0;
             if ((rc = grow(&m->glin_carry, need, err))) return rc;
             m->glin_carry_bytes = need;
+        }
+    }
+    if (p.in_conv > 1 && (max_len > 1 || !m->use_fuse)) {   // (decode graphs never touch this buffer)
+        const size_t need = (size_t)m->n_convs * n_runs * (p.in_conv - 1) * W * 4;
+        if (need > m->conv_pend_bytes) {
+            m->conv_pend_bytes = 0;
+            if ((rc = grow(&m->conv_pend, need, err))) return rc;
+            m->scratch_epoch++;
+            m->conv_pend_bytes = need;
         }
     }
     const int head = (n_want > 0 && pick_out) ? 2 : (n_want > 0 && logits_out) ? 1 : 0;

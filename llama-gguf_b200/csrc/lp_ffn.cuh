@@ -223,19 +223,17 @@ __global__ void __launch_bounds__(256) lp_moe_down_sel_kernel(const T* __restric
             const int r = o / width, c = o - r * width;
             const T* ar = act + (size_t)r * per_row;
             const T* dr = down_cat + (size_t)c * kd;
-            for (int k = 0; k <= top; k++) {
-                const int e = k < top ? sel[(size_t)r * top + k] : E;
-                const int len = k < top ? eff : sff;
-                const T* w = dr + (size_t)e * eff;
-                const T* a = ar + (size_t)k * eff;
+            // the row's segments as one list of 16-byte groups (expert sizes are multiples of VN): no loop per segment, so that the
+            // loads of several groups are in flight
 #pragma unroll 4
-                for (int i = (sw * 32 + lane) * VN; i < len; i += MD_SPLIT * 32 * VN) {
-                    float wv[VN], xv[VN];
-                    Vec8<T>::load(w + i, wv);
-                    Vec8<T>::load(a + i, xv);
+            for (int i = (sw * 32 + lane) * VN; i < per_row; i += MD_SPLIT * 32 * VN) {
+                const int k = min(i / eff, top);
+                const int e = k < top ? sel[(size_t)r * top + k] : E;
+                float wv[VN], xv[VN];
+                Vec8<T>::load(dr + (size_t)e * eff + (i - k * eff), wv);
+                Vec8<T>::load(ar + i, xv);
 #pragma unroll
-                    for (int j = 0; j < VN; j++) acc = fmaf(wv[j], xv[j], acc);
-                }
+                for (int j = 0; j < VN; j++) acc = fmaf(wv[j], xv[j], acc);
             }
         }
         acc = wsum(acc);

@@ -109,14 +109,16 @@ __global__ void __launch_bounds__(256) lp_latent_qprep_kernel(StepMeta sm, Laten
     latent_query_row(g, Q + (size_t)r * g.H * (g.dim + g.rot_dim), cs, sn, qn + (size_t)r * g.H * g.dim, qbuf + (size_t)r * g.H * (g.kv_rank + g.rot_dim));
 }
 
-// out[r][c] = V[r][c] * gate in the compute type: the operand of W_o
-template <typename T>
-__global__ void lp_latent_gate_kernel(LatentGeom g, const float* __restrict__ V, const float* __restrict__ P, int ldp, int R, T* __restrict__ out) {
-    const int n = g.H * g.vdim;
-    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= (size_t)R * n) return;
-    const int r = (int)(i / n), c = (int)(i - (size_t)r * n);
-    out[i] = from_f<T>(V[i] * latent_gate(g, P + (size_t)r * ldp, c));
+// out[r][c] = V[r][c] * gate in the compute type: the operand of W_o.  N channels per thread (4: vdim a multiple of 4)
+template <typename T, int N>
+__global__ void lp_latent_gate_kernel(LatentGeom g, const float* __restrict__ V, const float* __restrict__ P, int ldp, T* __restrict__ out) {
+    const int n = g.H * g.vdim, r = blockIdx.x;
+    for (int c = threadIdx.x * N; c < n; c += blockDim.x * N) {
+        FloatV<N> v = load_v<N>(V + (size_t)r * n + c);
+#pragma unroll
+        for (int e = 0; e < N; e++) v.v[e] *= latent_gate(g, P + (size_t)r * ldp, c + e);
+        store_v<N>(out + (size_t)r * n + c, v);
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ few rows, one token per run (decoding)
@@ -180,12 +182,16 @@ __global__ void __launch_bounds__(256) lp_latent_absorb_kernel(StepMeta sm, Late
     const int n = blockIdx.x / nch, ch = blockIdx.x - n * nch;
     const int lanes = latent_lanes(g.dim, VN), cols = 8 * (32 / lanes);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane % lanes;
+    const int j = ch * cols + warp * (32 / lanes) + lane / lanes;
+    {
+        const int j0 = ch * cols + warp * (32 / lanes);
+        if (j0 < g.kv_rank) prefetch_row(ukT + ((size_t)n * g.kv_rank + j0) * g.dim, min(32 / lanes, g.kv_rank - j0) * g.dim, lane);
+    }
     for (int i = threadIdx.x; i < R * g.dim; i += 256) {
         const int r = i / g.dim, d = i - r * g.dim;
         la_sm[i] = Q[(size_t)r * ldq + n * per + d];
     }
     __syncthreads();
-    const int j = ch * cols + warp * (32 / lanes) + lane / lanes;
     for (int rb = 0; rb < R; rb += GV_ROWS) {
         const int nr = min(GV_ROWS, R - rb);
         float acc[GV_ROWS];
@@ -213,7 +219,7 @@ __global__ void __launch_bounds__(256) lp_latent_absorb_kernel(StepMeta sm, Late
 // memory (two in flight, 16-byte cp.async) and its LS_HEADS warps each take one head: a key per lane for the scores, online softmax, the
 // latent channels dealt over the lanes for the weighted sum.  part_o [R][H][splits][kv_rank] receives the unnormalised sums, part_ml
 // the running maximum and sum (an empty split: -inf, 0).
-constexpr int LS_HEADS = 8, LS_KEYS = 32;
+constexpr int LS_HEADS = 8, LS_KEYS = 32, LS_ROWS = 64;   // (LS_ROWS: the most rows these kernels take)
 __host__ __device__ inline size_t latent_split_smem(int D) { return (size_t)(LS_HEADS * D + 2 * LS_KEYS * (D + 4)) * 4; }
 template <int VCH>
 __global__ void __launch_bounds__(32 * LS_HEADS) lp_latent_split_kernel(StepMeta sm, AttnGeom a, const float* __restrict__ qbuf, float* __restrict__ part_o,
@@ -309,6 +315,10 @@ __global__ void __launch_bounds__(256) lp_latent_merge_kernel(LatentGeom g, cons
     float* wgt = lm_sm + (size_t)R * g.kv_rank;          // [R][splits]
     constexpr int VN = Vec8<T>::N;
     const int n = blockIdx.x / nch, ch = blockIdx.x - n * nch, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    {
+        const int per_warp = 32 / latent_lanes(g.kv_rank, VN), c0 = (ch * 8 + warp) * per_warp;
+        if (c0 < g.vdim) prefetch_row(uv + ((size_t)n * g.vdim + c0) * g.kv_rank, min(per_warp, g.vdim - c0) * g.kv_rank, lane);
+    }
     for (int r = warp; r < R; r += 8) {                  // a warp per row: the splits' weights, their sum taken off
         const float* ml = part_ml + ((size_t)r * g.H + n) * splits * 2;
         float M = -INFINITY, L = 0.0f;
@@ -319,17 +329,31 @@ __global__ void __launch_bounds__(256) lp_latent_merge_kernel(LatentGeom g, cons
         for (int s = lane; s < splits; s += 32) wgt[r * splits + s] = expf(ml[2 * s] - M) / L;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < R * g.kv_rank; i += 256) {
-        const int r = i / g.kv_rank, c = i - r * g.kv_rank;
+    // a thread per (group of splits, row, 4 channels): as many groups as the block's threads allow
+    const int v4 = g.kv_rank / 4, items = R * v4, groups = max(1, 256 / items);
+    float* gsum = lm_sm + (((size_t)R * (g.kv_rank + splits) + 3) & ~(size_t)3);      // [groups][items][4] (groups > 1)
+    for (int it = threadIdx.x; it < items * groups; it += 256) {
+        const int q = it / items, i = it - q * items, r = i / v4, c = (i - r * v4) * 4;
         const float* po = part_o + ((size_t)r * g.H + n) * splits * g.kv_rank + c;
         const float* w = wgt + r * splits;
-        float acc = 0.0f;
-#pragma unroll 8
-        for (int s = 0; s < splits; s++)
-            if (w[s] > 0.0f) acc = fmaf(w[s], po[(size_t)s * g.kv_rank], acc);       // (an empty split has written nothing)
-        lat[i] = acc;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int s = q; s < splits; s += groups) {
+            const float ws = w[s];
+            const float4 o = ws > 0.0f ? *reinterpret_cast<const float4*>(po + (size_t)s * g.kv_rank) : make_float4(0.f, 0.f, 0.f, 0.f);   // (an empty split has written nothing)
+            acc.x = fmaf(ws, o.x, acc.x); acc.y = fmaf(ws, o.y, acc.y); acc.z = fmaf(ws, o.z, acc.z); acc.w = fmaf(ws, o.w, acc.w);
+        }
+        *reinterpret_cast<float4*>(groups > 1 ? gsum + (size_t)it * 4 : lat + (size_t)i * 4) = acc;
     }
     __syncthreads();
+    if (groups > 1) {
+        for (int i = threadIdx.x; i < items * 4; i += 256) {
+            float acc = 0.0f;
+            for (int q = 0; q < groups; q++) acc += gsum[(size_t)q * items * 4 + i];
+            lat[i] = acc;
+        }
+        __syncthreads();
+    }
     const int lanes = latent_lanes(g.kv_rank, VN), cols = 8 * (32 / lanes), sub = lane % lanes;
     const int c = ch * cols + warp * (32 / lanes) + lane / lanes;
     for (int rb = 0; rb < R; rb += GV_ROWS) {
@@ -343,6 +367,173 @@ __global__ void __launch_bounds__(256) lp_latent_merge_kernel(LatentGeom g, cons
                     const int r = rb + i, o = n * g.vdim + c;
                     out[(size_t)r * g.H * g.vdim + o] = from_f<T>(acc[i] * latent_gate(g, P + (size_t)r * ldp, o));
                 }
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ prompt rows (bf16)
+// All heads of a token meet the same cached rows, so the (token, head) pairs of a run are ONE list of query rows, [tokens * H][D] as qbuf
+// holds them: a block of 8 warps takes LT_ROWS neighbours of the list (16 per warp) against tiles of LT_KEYS cached rows.  A tile is
+// staged once, as bf16 [key][channel], and serves both products on the tensor pipe (mma.sync m16n8k16, f32 accumulators): ldmatrix gives
+// its keys for the scores, ldmatrix.trans its first vdim channels as the values.  Two tiles in shared memory: the next one is loaded
+// (DK <= 128: into registers, ahead of the products) while this one is used.  Mask, online softmax and normalisation in f32.  DK / DV:
+// upper bounds of the row and of the latent.  Blocks start with the last tokens, which see the most keys.
+constexpr int LT_ROWS = 128, LT_KEYS = 64;
+template <int DK> constexpr size_t latent_tile_smem() { return (size_t)(LT_ROWS + 2 * LT_KEYS) * (DK + 8) * 2; }
+__device__ __forceinline__ void ldsm4(uint32_t* r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t* r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+template <int DK, int DV>
+__global__ void __launch_bounds__(256) lp_latent_tile_kernel(StepMeta sm, AttnGeom a, const float* __restrict__ qbuf, bf16* __restrict__ out) {
+    constexpr int PITCH = DK + 8, NU = LT_KEYS * (DK / 4) / 256;
+    constexpr bool AHEAD = DK <= 128;
+    extern __shared__ __align__(16) uint8_t lt_sm[];
+    bf16* Qs = reinterpret_cast<bf16*>(lt_sm);          // [LT_ROWS][PITCH]
+    bf16* Ks = Qs + LT_ROWS * PITCH;                    // [2][LT_KEYS][PITCH]
+    const int run = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+    const int r0 = sm.run_start[run], len = sm.run_start[run + 1] - r0, p0 = sm.run_pos0[run];
+    const int rows = len * a.H, nb = (rows + LT_ROWS - 1) / LT_ROWS;
+    if ((int)blockIdx.x >= nb) return;
+    const int f0 = (nb - 1 - (int)blockIdx.x) * LT_ROWS, D = a.dim;
+    const float* cache = reinterpret_cast<const float*>(sm.run_kv[run] + a.kv_off);
+    const float* q = qbuf + ((size_t)r0 * a.H + f0) * D;
+    for (int u = threadIdx.x; u < LT_ROWS * (DK / 4); u += 256) {
+        const int f = u / (DK / 4), d = (u - f * (DK / 4)) * 4;
+        const float4 v = (f0 + f < rows && d < D) ? *reinterpret_cast<const float4*>(q + (size_t)f * D + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+        *reinterpret_cast<uint2*>(Qs + f * PITCH + d) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
+    }
+    const int last = p0 + min(f0 + LT_ROWS - 1, rows - 1) / a.H, lo = attn_lo(a, p0 + f0 / a.H);
+    const int tiles = (last - lo) / LT_KEYS + 1;
+    auto get = [&](int t, int u) {
+        const int i = threadIdx.x + u * 256, key = i / (DK / 4), d = (i - key * (DK / 4)) * 4, j = lo + t * LT_KEYS + key;
+        return (j <= last && d < D) ? *reinterpret_cast<const float4*>(cache + (size_t)j * D + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+    };
+    auto put = [&](int t, int u, const float4& v) {
+        const int i = threadIdx.x + u * 256, key = i / (DK / 4), d = (i - key * (DK / 4)) * 4;
+        *reinterpret_cast<uint2*>(Ks + ((t & 1) * LT_KEYS + key) * PITCH + d) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
+    };
+    auto stage = [&](int t) {
+#pragma unroll
+        for (int u0 = 0; u0 < NU; u0 += 4) {
+            float4 v[4];
+#pragma unroll
+            for (int u = 0; u < 4; u++) v[u] = get(t, u0 + u);
+#pragma unroll
+            for (int u = 0; u < 4; u++) put(t, u0 + u, v[u]);
+        }
+    };
+    stage(0);
+    // this thread's two rows of the warp's 16, their positions, and the warp's first and last position
+    const int fa = f0 + warp * 16 + gid, fb = fa + 8;
+    const int ia = p0 + min(fa, rows - 1) / a.H, ib = p0 + min(fb, rows - 1) / a.H;
+    const int w_first = p0 + min(f0 + warp * 16, rows - 1) / a.H, w_last = p0 + min(f0 + warp * 16 + 15, rows - 1) / a.H;
+    const uint32_t q_addr = smem_u32(Qs + (warp * 16 + (lane & 15)) * PITCH + (lane >> 4) * 8);
+    const uint32_t k_off = (uint32_t)(((lane & 7) + ((lane >> 4) << 3)) * PITCH + ((lane >> 3) & 1) * 8) * 2;
+    const uint32_t v_off = (uint32_t)(((lane & 7) + (((lane >> 3) & 1) << 3)) * PITCH + (lane >> 4) * 8) * 2;
+    const float sl = a.scale * 1.4426950408889634f;      // scores in powers of two
+    float o[DV / 8][4];
+#pragma unroll
+    for (int n = 0; n < DV / 8; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
+    __syncthreads();
+    for (int t = 0; t < tiles; t++) {
+        const int j0 = lo + t * LT_KEYS;
+        float4 nx[AHEAD ? NU : 1];
+        if (AHEAD && t + 1 < tiles) {
+#pragma unroll
+            for (int u = 0; u < NU; u++) nx[u % (AHEAD ? NU : 1)] = get(t + 1, u);
+        }
+        if (j0 <= w_last && j0 + LT_KEYS - 1 > w_first - a.window) {      // (some row of the warp sees some key of the tile)
+            const uint32_t kt = smem_u32(Ks + (t & 1) * LT_KEYS * PITCH);
+            float sc[LT_KEYS / 8][4];
+#pragma unroll
+            for (int n = 0; n < LT_KEYS / 8; n++) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.0f;
+#pragma unroll
+            for (int kb = 0; kb < DK / 16; kb++) {
+                if (kb * 16 < D) {
+                    uint32_t qa[4];
+                    ldsm4(qa, q_addr + kb * 32);
+#pragma unroll
+                    for (int n = 0; n < LT_KEYS / 16; n++) {
+                        uint32_t b[4];
+                        ldsm4(b, kt + k_off + (uint32_t)(n * 16 * PITCH + kb * 16) * 2);
+                        mma_bf16(sc[2 * n], qa, b[0], b[1]);
+                        mma_bf16(sc[2 * n + 1], qa, b[2], b[3]);
+                    }
+                }
+            }
+            const bool all = j0 + LT_KEYS - 1 <= w_first && j0 > w_last - a.window;     // nothing of the tile is masked
+            float x0 = -INFINITY, x1 = -INFINITY;
+#pragma unroll
+            for (int n = 0; n < LT_KEYS / 8; n++) {
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int j = j0 + n * 8 + 2 * tig + (e & 1), i = (e & 2) ? ib : ia;
+                    sc[n][e] = (all || (j <= i && i - j < a.window)) ? sc[n][e] * sl : -INFINITY;
+                }
+                x0 = fmaxf(x0, fmaxf(sc[n][0], sc[n][1]));
+                x1 = fmaxf(x1, fmaxf(sc[n][2], sc[n][3]));
+            }
+            x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1));
+            x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
+            x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1));
+            x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
+            const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
+            const float b0 = n0 == -INFINITY ? 0.0f : n0, b1 = n1 == -INFINITY ? 0.0f : n1;      // (a row without a visible key yet: all weights 0)
+            const float c0 = exp2f(m0 - b0), c1 = exp2f(m1 - b1);
+            m0 = n0;
+            m1 = n1;
+            float s0 = 0.0f, s1 = 0.0f;
+            uint32_t pa[LT_KEYS / 16][4];
+#pragma unroll
+            for (int n = 0; n < LT_KEYS / 8; n++) {
+                const float e0 = exp2f(sc[n][0] - b0), e1 = exp2f(sc[n][1] - b0), e2 = exp2f(sc[n][2] - b1), e3 = exp2f(sc[n][3] - b1);
+                s0 += e0 + e1;
+                s1 += e2 + e3;
+                pa[n >> 1][(n & 1) * 2] = pack_bf2(e0, e1);
+                pa[n >> 1][(n & 1) * 2 + 1] = pack_bf2(e2, e3);
+            }
+            l0 = l0 * c0 + s0;
+            l1 = l1 * c1 + s1;
+#pragma unroll
+            for (int n = 0; n < DV / 8; n++) {
+                o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1;
+            }
+#pragma unroll
+            for (int n = 0; n < DV / 16; n++) {
+                if (n * 16 < a.vdim) {
+#pragma unroll
+                    for (int k = 0; k < LT_KEYS / 16; k++) {
+                        uint32_t b[4];
+                        ldsm4_t(b, kt + v_off + (uint32_t)(k * 16 * PITCH + n * 16) * 2);
+                        mma_bf16(o[2 * n], pa[k], b[0], b[1]);
+                        mma_bf16(o[2 * n + 1], pa[k], b[2], b[3]);
+                    }
+                }
+            }
+        }
+        if (t + 1 < tiles) {
+            if (AHEAD) {
+#pragma unroll
+                for (int u = 0; u < NU; u++) put(t + 1, u, nx[u % (AHEAD ? NU : 1)]);
+            } else stage(t + 1);
+        }
+        __syncthreads();
+    }
+    l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
+    l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    const float v0 = 1.0f / l0, v1 = 1.0f / l1;
+#pragma unroll
+    for (int n = 0; n < DV / 8; n++) {
+        const int c = n * 8 + 2 * tig;
+        if (c < a.vdim) {        // (vdim is even: c + 1 < vdim)
+            if (fa < rows) *reinterpret_cast<uint32_t*>(out + ((size_t)r0 * a.H + fa) * a.vdim + c) = pack_bf2(o[n][0] * v0, o[n][1] * v0);
+            if (fb < rows) *reinterpret_cast<uint32_t*>(out + ((size_t)r0 * a.H + fb) * a.vdim + c) = pack_bf2(o[n][2] * v1, o[n][3] * v1);
         }
     }
 }
