@@ -524,6 +524,66 @@ __global__ void __launch_bounds__(256) lp_gemv_kernel(const T* __restrict__ X, i
     if (tail.on) rows_tail<T>(tail);
 }
 
+__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&v);
+}
+__device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// Three to sixteen rows in bf16 (small decode batches): the weights meet the rows on the tensor pipe (mma.sync m16n8k16, A = 16 weight rows,
+// B = 8 activation rows, NT of them), because the CUDA cores would spend a multiply and an unpack per weight and row.  A block takes 16
+// weight rows, its 8 warps take K in chunks of 32 in turn; a lane's 16-byte load holds 8 consecutive k of one row, for both operands
+// alike, so the order of k inside a chunk does not matter to the sum.  The warps' 16 x 8 NT parts meet in shared memory, warp order.
+// K a multiple of 32, rows 16-byte aligned.
+template <int EPI, int NT>
+__global__ void __launch_bounds__(256) lp_gemv_mma_kernel(const bf16* __restrict__ X, int ldx, const bf16* __restrict__ W, int ldw, void* __restrict__ Y, int ldy,
+                                                          int R, int N, int K, float alpha, RowsTail tail, const float* __restrict__ bias, float2 act) {
+    __shared__ float red[8][16 * 8 * NT];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+    const bf16* xr[NT];
+#pragma unroll
+    for (int t = 0; t < NT; t++) xr[t] = X + (size_t)min(t * 8 + gid, R - 1) * ldx + tig * 8;
+    for (int n0 = blockIdx.x * 16; n0 < N; n0 += gridDim.x * 16) {
+        const bf16* wa = W + (size_t)min(n0 + gid, N - 1) * ldw + tig * 8;
+        const bf16* wb = W + (size_t)min(n0 + gid + 8, N - 1) * ldw + tig * 8;
+        float c[NT][4];
+#pragma unroll
+        for (int t = 0; t < NT; t++) c[t][0] = c[t][1] = c[t][2] = c[t][3] = 0.0f;
+#pragma unroll 4
+        for (int k = warp * 32; k < K; k += 8 * 32) {
+            const uint4 lo = *reinterpret_cast<const uint4*>(wa + k), hi = *reinterpret_cast<const uint4*>(wb + k);
+            const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+#pragma unroll
+            for (int t = 0; t < NT; t++) {
+                const uint4 b = *reinterpret_cast<const uint4*>(xr[t] + k);
+                mma_bf16(c[t], a0, b.x, b.y);
+                mma_bf16(c[t], a1, b.z, b.w);
+            }
+        }
+        __syncthreads();   // the sums of the group before have been read
+#pragma unroll
+        for (int t = 0; t < NT; t++) {
+            float* d = red[warp] + (t * 8 + 2 * tig) * 16 + gid;      // [activation row][weight row]
+            d[0] = c[t][0];
+            d[16] = c[t][1];
+            d[8] = c[t][2];
+            d[24] = c[t][3];
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < 16 * R; i += 256) {
+            const int r = i >> 4, n = n0 + (i & 15);
+            float v = 0.0f;
+#pragma unroll
+            for (int w = 0; w < 8; w++) v += red[w][i];
+            if (n < N) epi_store<bf16, EPI>(Y, (size_t)r * ldy + n, alpha * v + (bias ? bias[n] : 0.0f), act);
+        }
+    }
+    if (tail.on) rows_tail<bf16>(tail);
+}
+
 // The same for a normed input: the block first norms the (few) rows of the f32 residual stream into shared memory -- rms over the
 // row, times the norm weight, rounded to the compute type exactly as lp_rmsnorm_kernel does -- and then multiplies from there.
 // Every block repeats the norm (the rows are a few KB out of L2); a launch and a round trip through global memory go away.
@@ -861,15 +921,6 @@ __global__ void __launch_bounds__(32 * ATT_WARPS) lp_window_attn_kernel(StepMeta
 // the accumulator layout of the score tile straight into the A operand of the value product.  DK / DV are upper bounds of the key
 // and value sizes (multiples of 16 / 8 at run time); the visible keys of a tile of queries are [0, min(keep_first, lo0)) and
 // [lo0, last query], lo0 = the window start of its first query, every element masked by the rule itself.
-__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&v);
-}
-__device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 constexpr int AT_Q = 64, AT_K = 64;
 template <int DK, int DV>
 __global__ void __launch_bounds__(128) lp_window_attn_tile_kernel(StepMeta sm, AttnGeom a, const float* __restrict__ qbuf,
@@ -1364,8 +1415,14 @@ __global__ void lp_argmax_kernel(const float* __restrict__ logits, int vocab, in
     const float* row = logits + (size_t)blockIdx.x * vocab;
     float best = -INFINITY;
     int bi = 0;
-    for (int i = threadIdx.x; i < vocab; i += blockDim.x)
-        if (row[i] >= best) { best = row[i]; bi = i; }
+    for (int i0 = threadIdx.x; i0 < vocab; i0 += 8 * blockDim.x) {      // eight loads in flight
+        float v[8];
+#pragma unroll
+        for (int u = 0; u < 8; u++) v[u] = i0 + u * (int)blockDim.x < vocab ? row[i0 + u * blockDim.x] : -INFINITY;
+#pragma unroll
+        for (int u = 0; u < 8; u++)
+            if (i0 + u * (int)blockDim.x < vocab && v[u] >= best) { best = v[u]; bi = i0 + u * blockDim.x; }
+    }
     __shared__ float sv[1024];
     __shared__ int si[1024];
     sv[threadIdx.x] = best;
@@ -1539,6 +1596,7 @@ struct LpModel {
     uint64_t scratch_epoch = 1;
     bool use_graph = true;
     int tc_min_rows = 17;
+    bool use_gemv_mma = true;    // B200_LP_GEMV_MMA=0: small decode batches multiply on the CUDA cores
     int conv_fuse_rows = 1;      // B200_LP_CONV_FUSE_ROWS: decode steps of so many rows norm and convolve inside the projection
     bool use_lat_split = true;   // B200_LP_LAT_SPLIT=0: decoding latent attention in the many-row kernels
     int* tc_err = nullptr;
@@ -1688,6 +1746,24 @@ void gemm_t(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, i
         constexpr int VN = Vec8<T>::N;
         const bool heads = groups > 1;
         const int vec_ok = (K % VN == 0 && ldx % VN == 0 && ldw % VN == 0 && zs.x % VN == 0 && ((uintptr_t)X % 16) == 0 && ((uintptr_t)W % 16) == 0) ? 1 : 0;
+        if constexpr (sizeof(T) == 2) {
+            if (R >= 3 && m->use_gemv_mma && !heads && vec_ok && K % 32 == 0) {
+                const RowsTail tl = tail ? *tail : RowsTail{};
+                const dim3 g((unsigned)std::min((N + 15) / 16, 8 * 148)), b(256);
+#define LP_GT(E)                                                                                                                            \
+    do {                                                                                                                                    \
+        if (R <= 8) launch(m, lp_gemv_mma_kernel<E, 1>, g, b, 0, x, ldx, w, ldw, Y, ldy, R, N, K, alpha, tl, bias, act);                    \
+        else launch(m, lp_gemv_mma_kernel<E, 2>, g, b, 0, x, ldx, w, ldw, Y, ldy, R, N, K, alpha, tl, bias, act);                           \
+    } while (0)
+                if (epi == EPI_STORE) LP_GT(EPI_STORE);
+                else if (epi == EPI_ADD) LP_GT(EPI_ADD);
+                else if (epi == EPI_GELU) LP_GT(EPI_GELU);
+                else if (epi == EPI_XIELU) LP_GT(EPI_XIELU);
+                else LP_GT(EPI_RELU2);
+#undef LP_GT
+                return;
+            }
+        }
         // a few blocks per SM, each walking its share of the output columns with the activation rows staged once
         const int Nall = N * groups;
         dim3 grid(std::min((Nall + 7) / 8, 4 * 148)), block(256);
@@ -1769,6 +1845,7 @@ bool gemv_norm_t(LpModel* m, const float* x, const int* gather, const float* nw,
     constexpr int VN = Vec8<T>::N;
     const size_t smem = (size_t)R * K * sizeof(T);
     if (R > 2 * GV_ROWS || K % VN || ((uintptr_t)W & 15) || smem > 96 * 1024) return false;
+    if (sizeof(T) == 2 && R >= 3 && m->use_gemv_mma && K % 32 == 0) return false;      // (lp_gemv_mma_kernel behind a norm of its own)
     if (epi != EPI_STORE && epi != EPI_RELU2 && epi != EPI_XIELU) return false;
     static bool once[EPI_COUNT][GV_ROWS + 1][64] = {};
     int dev = 0;
@@ -1960,6 +2037,8 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
         if (e && *e) m->use_stream_tail = atoi(e) != 0;
         e = getenv("B200_LP_GRAPH");
         if (e && *e) m->use_graph = atoi(e) != 0;
+        e = getenv("B200_LP_GEMV_MMA");
+        if (e && *e) m->use_gemv_mma = atoi(e) != 0;
         e = getenv("B200_LP_CONV_FUSE_ROWS");
         if (e && *e) m->conv_fuse_rows = atoi(e);
         e = getenv("B200_LP_LAT_SPLIT");
@@ -2377,7 +2456,7 @@ int lp_finalize(LpModel* m, std::string* err) {
             m->max_qrank = std::max(m->max_qrank, a.q_rank);
             // decoding kernels: 16-byte loads of cached rows and weights, the rows in shared memory, two key tiles too
             const int vn = m->f32 ? 4 : 8;
-            const size_t part = (size_t)LS_ROWS * (std::max(a.dim, a.kv_rank) + std::max(64, a.rot.dims)) * 4;
+            const size_t part = (size_t)2 * GV_ROWS * (std::max(a.dim, a.kv_rank) + std::max(64, a.rot.dims)) * 4;
             if (D % 4 == 0 && a.kv_rank % vn == 0 && a.dim % vn == 0 && latent_split_smem((int)D) <= 200 * 1024 && part <= 190 * 1024) {
                 for (int r = 1; r <= LS_ROWS; r++) L.lat_splits = std::max(L.lat_splits, r * latent_splits(r, a.heads));
                 m->lat_o_floats = std::max(m->lat_o_floats, (size_t)L.lat_splits * a.heads * a.kv_rank);
@@ -3157,7 +3236,9 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             const bool direct = a.q_rank == 0, own = a.kv_from < 0;
             // one token per run, few rows: absorb / split attention / merge (lp_latent_attn.cuh)
             const bool split = m->use_fuse && m->use_lat_split && max_len == 1 && R <= LS_ROWS && L.lat_splits > 0;
-            if (!(split && direct)) {
+            // few rows: the per-head products in kernels of their own too (absorb, merge); more: prep / GEMMs around the split attention
+            const bool few_lat = split && R <= 2 * GV_ROWS;
+            if (!(few_lat && direct)) {
                 if (m->f32) launch(m, lp_latent_prep_kernel<float>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (float*)m->cq, (float*)m->act_a, m->qbuf);
                 else launch(m, lp_latent_prep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->P, L.n_in, L.dq_norm, L.dkv_norm, L.rot_freq, (bf16*)m->cq, (bf16*)m->act_a, m->qbuf);
             }
@@ -3167,7 +3248,9 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             ag.out_ld = a.heads * a.kv_rank;
             ag.out_scale = 1.0f;
             ag.fused_prep = 0;
-            if (split) {
+#define LP_LS(V) launch(m, lp_latent_split_kernel<V>, sgrid, dim3(32 * LS_HEADS), latent_split_smem(D), sm, ag, (const float*)m->qbuf, m->lat_o, m->lat_ml)
+#define LP_LS_ANY() do { if (a.kv_rank <= 128) LP_LS(4); else if (a.kv_rank <= 256) LP_LS(8); else LP_LS(16); } while (0)
+            if (few_lat) {
                 const float* Q = direct ? m->P + lg.q_off : m->O;
                 const int ldq = direct ? L.n_in : a.heads * per, vn = m->f32 ? 4 : 8, splits = latent_splits(R, a.heads);
                 const int uk_cols = 8 * (32 / latent_lanes(a.dim, vn)), uk_ch = (a.kv_rank + uk_cols - 1) / uk_cols;
@@ -3176,9 +3259,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                 const size_t asm_ = (size_t)(R * a.dim + lg.rot_n) * 4, usm = ((size_t)R * (a.kv_rank + splits) + 1024 + 4) * 4;
                 if (m->f32) launch(m, lp_latent_absorb_kernel<float>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const float*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
                 else launch(m, lp_latent_absorb_kernel<bf16>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const bf16*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
-#define LP_LS(V) launch(m, lp_latent_split_kernel<V>, sgrid, dim3(32 * LS_HEADS), latent_split_smem(D), sm, ag, (const float*)m->qbuf, m->lat_o, m->lat_ml)
-                if (a.kv_rank <= 128) LP_LS(4); else if (a.kv_rank <= 256) LP_LS(8); else LP_LS(16);
-#undef LP_LS
+                LP_LS_ANY();
                 if (m->f32) launch(m, lp_latent_merge_kernel<float>, ugrid, dim3(256), usm, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (const float*)L.w_uv, (const float*)m->P, L.n_in, (float*)m->act_a, R, uv_ch);
                 else launch(m, lp_latent_merge_kernel<bf16>, ugrid, dim3(256), usm, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (const bf16*)L.w_uv, (const float*)m->P, L.n_in, (bf16*)m->act_a, R, uv_ch);
             } else {
@@ -3187,13 +3268,21 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                     else launch(m, lp_latent_qprep_kernel<bf16>, dim3(R), dim3(256), csm, sm, lg, (const float*)m->O, L.rot_freq, (bf16*)m->act_a, m->qbuf);
                 }
                 gemm_heads(m, m->act_a, a.heads * a.dim, a.dim, L.w_ukT, a.heads, a.kv_rank, a.dim, m->qbuf, a.heads * D, D, R);
-                if (!latent_tile(m, sm, ag, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
+                if (split) {
+                    const int splits = latent_splits(R, a.heads);
+                    const dim3 sgrid(splits, R, (a.heads + LS_HEADS - 1) / LS_HEADS);
+                    LP_LS_ANY();
+                    if (m->f32) launch(m, lp_latent_combine_kernel<float>, dim3(R, a.heads), dim3(128), 0, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (float*)m->act_a);
+                    else launch(m, lp_latent_combine_kernel<bf16>, dim3(R, a.heads), dim3(128), 0, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (bf16*)m->act_a);
+                } else if (!latent_tile(m, sm, ag, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
                 gemm_heads(m, m->act_a, a.heads * a.kv_rank, a.kv_rank, L.w_uv, a.heads, a.vdim, a.kv_rank, m->O, nv, a.vdim, R);
 #define LP_LG(T, N) launch(m, lp_latent_gate_kernel<T, N>, dim3(R), dim3(256), 0, lg, (const float*)m->O, (const float*)m->P, L.n_in, (T*)m->act_a)
                 if (m->f32) { if (a.vdim % 4) LP_LG(float, 1); else LP_LG(float, 4); }
                 else { if (a.vdim % 4) LP_LG(bf16, 1); else LP_LG(bf16, 4); }
 #undef LP_LG
             }
+#undef LP_LS_ANY
+#undef LP_LS
             project_out(m->act_a, nv, L.wo, L.norm1, moe_next);
         } else if (L.d.mixer == B200_MIX_STATE_SPACE) {
             const b200_state_space_desc& g = L.d.ssd;

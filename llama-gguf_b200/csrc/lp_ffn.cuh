@@ -208,13 +208,19 @@ __global__ void __launch_bounds__(256) lp_moe_up_sel_kernel(const T* __restrict_
 // y[r][c] = sum over the row's segments of down_e[c] . act segment; down_cat is [width][E eff + sff].  MD_SPLIT warps share one (row, c):
 // each takes every MD_SPLIT-th 16-byte group of every segment (more loads in flight per output: a decode step has only `width` of
 // them), the partial sums meet in shared memory and are added in warp order.  accum = 1: y += (y is the residual stream).
-constexpr int MD_SPLIT = 4;
+constexpr int MD_SPLIT = 4, MD_BATCH = 6;
 template <typename T>
 __global__ void __launch_bounds__(256) lp_moe_down_sel_kernel(const T* __restrict__ act, const T* __restrict__ down_cat, const int* __restrict__ sel,
                                                               int E, int top, int eff, int sff, int width, int R, float* __restrict__ y, RowsTail tail, int accum) {
     constexpr int VN = Vec8<T>::N, GROUPS = 8 / MD_SPLIT;
     __shared__ float part[8];
+    __shared__ int sel_s[256];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = warp / MD_SPLIT, sw = warp % MD_SPLIT;
+    const bool sel_in = R * top <= 256;
+    if (sel_in) {
+        for (int i = threadIdx.x; i < R * top; i += blockDim.x) sel_s[i] = sel[i];
+        __syncthreads();
+    }
     const int per_row = top * eff + sff, kd = E * eff + sff, total = R * width;
     for (int base = blockIdx.x * GROUPS; base < total; base += gridDim.x * GROUPS) {
         const int o = base + grp;
@@ -223,17 +229,28 @@ __global__ void __launch_bounds__(256) lp_moe_down_sel_kernel(const T* __restric
             const int r = o / width, c = o - r * width;
             const T* ar = act + (size_t)r * per_row;
             const T* dr = down_cat + (size_t)c * kd;
-            // the row's segments as one list of 16-byte groups (expert sizes are multiples of VN): no loop per segment, so that the
-            // loads of several groups are in flight
-#pragma unroll 4
-            for (int i = (sw * 32 + lane) * VN; i < per_row; i += MD_SPLIT * 32 * VN) {
-                const int k = min(i / eff, top);
-                const int e = k < top ? sel[(size_t)r * top + k] : E;
-                float wv[VN], xv[VN];
-                Vec8<T>::load(dr + (size_t)e * eff + (i - k * eff), wv);
-                Vec8<T>::load(ar + i, xv);
+            // the row's segments as one list of 16-byte groups (expert sizes are multiples of VN), MD_BATCH of them in flight per lane
+            for (int i0 = (sw * 32 + lane) * VN; i0 < per_row; i0 += MD_BATCH * MD_SPLIT * 32 * VN) {
+                uint4 wv[MD_BATCH], xv[MD_BATCH];
 #pragma unroll
-                for (int j = 0; j < VN; j++) acc = fmaf(wv[j], xv[j], acc);
+                for (int u = 0; u < MD_BATCH; u++) {
+                    const int i = i0 + u * MD_SPLIT * 32 * VN;
+                    wv[u] = xv[u] = make_uint4(0u, 0u, 0u, 0u);
+                    if (i < per_row) {
+                        const int k = min(i / eff, top);
+                        const int e = k < top ? (sel_in ? sel_s[r * top + k] : sel[(size_t)r * top + k]) : E;
+                        wv[u] = *reinterpret_cast<const uint4*>(dr + (size_t)e * eff + (i - k * eff));
+                        xv[u] = *reinterpret_cast<const uint4*>(ar + i);
+                    }
+                }
+#pragma unroll
+                for (int u = 0; u < MD_BATCH; u++) {
+                    float wf[VN], xf[VN];
+                    Vec8<T>::load(reinterpret_cast<const T*>(&wv[u]), wf);
+                    Vec8<T>::load(reinterpret_cast<const T*>(&xv[u]), xf);
+#pragma unroll
+                    for (int j = 0; j < VN; j++) acc = fmaf(wf[j], xf[j], acc);
+                }
             }
         }
         acc = wsum(acc);

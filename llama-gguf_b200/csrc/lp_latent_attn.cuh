@@ -132,30 +132,40 @@ __host__ __device__ inline int latent_lanes(int K, int VN) {
     while (l < 32 && l * VN < K) l <<= 1;
     return l;
 }
-// acc[i] = w . rows[i] over K values, summed over the `lanes` neighbouring lanes of the output (sub = place among them)
-template <typename T>
-__device__ __forceinline__ void latent_dot(const T* __restrict__ w, const float* rows, int ld, int nr, int K, int lanes, int sub, bool live, float* acc) {
+// acc[i] = w . rows[i] over K values, i < NR, summed over the `lanes` neighbouring lanes of the output (sub = place among them); rows past
+// nr are the last again.  rows: 16-byte aligned, ld a multiple of 4.
+template <typename T, int NR>
+__device__ __forceinline__ void latent_dot_n(const T* __restrict__ w, const float* rows, int ld, int nr, int K, int lanes, int sub, bool live, float* acc) {
     constexpr int VN = Vec8<T>::N;
 #pragma unroll
-    for (int i = 0; i < GV_ROWS; i++) acc[i] = 0.0f;
+    for (int i = 0; i < NR; i++) acc[i] = 0.0f;
     if (live) {
 #pragma unroll 2
         for (int k = sub * VN; k < K; k += lanes * VN) {
             float wv[VN];
             Vec8<T>::load(w + k, wv);
 #pragma unroll
-            for (int i = 0; i < GV_ROWS; i++) {
-                if (i < nr) {
+            for (int i = 0; i < NR; i++) {
+                const float* x = rows + (size_t)min(i, nr - 1) * ld + k;
 #pragma unroll
-                    for (int e = 0; e < VN; e++) acc[i] = fmaf(wv[e], rows[(size_t)i * ld + k + e], acc[i]);
+                for (int e = 0; e < VN; e += 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(x + e);
+                    acc[i] = fmaf(wv[e], v.x, acc[i]);
+                    acc[i] = fmaf(wv[e + 1], v.y, acc[i]);
+                    acc[i] = fmaf(wv[e + 2], v.z, acc[i]);
+                    acc[i] = fmaf(wv[e + 3], v.w, acc[i]);
                 }
             }
         }
     }
+    for (int o = lanes >> 1; o > 0; o >>= 1)
 #pragma unroll
-    for (int i = 0; i < GV_ROWS; i++)
-        if (i < nr)
-            for (int o = lanes >> 1; o > 0; o >>= 1) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], o);
+        for (int i = 0; i < NR; i++) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], o);
+}
+template <typename T>
+__device__ __forceinline__ void latent_dot(const T* __restrict__ w, const float* rows, int ld, int nr, int K, int lanes, int sub, bool live, float* acc) {
+    if (nr == 1) latent_dot_n<T, 1>(w, rows, ld, nr, K, lanes, sub, live, acc);
+    else latent_dot_n<T, GV_ROWS>(w, rows, ld, nr, K, lanes, sub, live, acc);
 }
 
 // Blocks [0, H nch): head n, a chunk of latent columns of all rows: qbuf[r][n][j] = W_uk[n]^T[j] . q_plain (ukT [H][kv_rank][dim]); the
@@ -165,7 +175,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) lp_latent_absorb_kernel(StepMeta sm, LatentGeom g, const float* __restrict__ Q, int ldq, const float* __restrict__ P, int ldp,
                                                                const T* __restrict__ ukT, const float* __restrict__ kvw, const double* __restrict__ freq,
                                                                float* __restrict__ qbuf, int R, int nch) {
-    extern __shared__ float la_sm[];     // product blocks: [R][dim] plain queries; [rot_n] angles
+    extern __shared__ __align__(16) float la_sm[];     // product blocks: [R][dim] plain queries; [rot_n] angles
     __shared__ float red[33];
     const int per = g.dim + g.rot_dim, D = g.kv_rank + g.rot_dim;
     if ((int)blockIdx.x >= g.H * nch) {
@@ -310,7 +320,7 @@ __global__ void __launch_bounds__(32 * LS_HEADS) lp_latent_split_kernel(StepMeta
 template <typename T>
 __global__ void __launch_bounds__(256) lp_latent_merge_kernel(LatentGeom g, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
                                                               const T* __restrict__ uv, const float* __restrict__ P, int ldp, T* __restrict__ out, int R, int nch) {
-    extern __shared__ float lm_sm[];
+    extern __shared__ __align__(16) float lm_sm[];
     float* lat = lm_sm;                                  // [R][kv_rank]
     float* wgt = lm_sm + (size_t)R * g.kv_rank;          // [R][splits]
     constexpr int VN = Vec8<T>::N;
@@ -368,6 +378,24 @@ __global__ void __launch_bounds__(256) lp_latent_merge_kernel(LatentGeom g, cons
                     out[(size_t)r * g.H * g.vdim + o] = from_f<T>(acc[i] * latent_gate(g, P + (size_t)r * ldp, o));
                 }
         }
+    }
+}
+
+// The merge alone: the latent of every (row, head) in the compute type -> out [R][H][kv_rank], the operand of the products with W_uv
+template <typename T>
+__global__ void __launch_bounds__(128) lp_latent_combine_kernel(LatentGeom g, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
+                                                                T* __restrict__ out) {
+    const size_t at = ((size_t)blockIdx.x * g.H + blockIdx.y) * splits;
+    float M = -INFINITY, L = 0.0f;
+    for (int s = 0; s < splits; s++) M = fmaxf(M, part_ml[2 * (at + s)]);
+    for (int s = 0; s < splits; s++) L = fmaf(part_ml[2 * (at + s) + 1], expf(part_ml[2 * (at + s)] - M), L);
+    for (int c = threadIdx.x; c < g.kv_rank; c += 128) {
+        float acc = 0.0f;
+        for (int s = 0; s < splits; s++) {
+            const float w = expf(part_ml[2 * (at + s)] - M);
+            if (w > 0.0f) acc = fmaf(w, part_o[(at + s) * g.kv_rank + c], acc);     // (an empty split has written nothing)
+        }
+        out[((size_t)blockIdx.x * g.H + blockIdx.y) * g.kv_rank + c] = from_f<T>(acc / L);
     }
 }
 
