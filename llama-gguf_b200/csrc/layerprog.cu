@@ -3120,8 +3120,10 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             launch(m, lp_add_vec_kernel, dim3(R), dim3(256), 0, m->x, add, W);
             add = nullptr;
         }
-        // the few-row expert kernels (16-byte loads: sizes multiples of 8 / 4, the rows in shared memory)
-        const bool moe_sel_ok = L.d.ff_kind == B200_FF_MOE && m->use_fuse && R <= 2 * GV_ROWS && W % (m->f32 ? 4 : 8) == 0 &&
+        // the few-row expert kernels (16-byte loads: sizes multiples of 8 / 4, the rows in shared memory), while the rows choose fewer experts
+        // than there are: beyond that the plain form reads every expert once for all rows (bf16: on the tensor pipe)
+        const bool many_choices = !m->f32 && m->use_gemv_mma && R >= 3 && L.d.ff_kind == B200_FF_MOE && R * L.d.moe.top > L.d.moe.experts && W % 32 == 0 && L.k_down % 32 == 0;
+        const bool moe_sel_ok = L.d.ff_kind == B200_FF_MOE && !many_choices && m->use_fuse && R <= 2 * GV_ROWS && W % (m->f32 ? 4 : 8) == 0 &&
                                 L.d.moe.expert_ff % (m->f32 ? 4 : 8) == 0 && L.d.moe.shared_ff % (m->f32 ? 4 : 8) == 0 && (size_t)R * W * elt(m) <= 40 * 1024;
         // (the fused tails know neither a router bias nor the always-on expert's gate)
         const LayerPlan* moe_next = ((few || sfew) && moe_sel_ok && !L.d.moe.router_bias && !L.d.moe.shared_gate) ? &L : nullptr;      // the mixer's output kernel also routes
