@@ -602,6 +602,32 @@ def test_decode_kernels_against_the_unfused_forms(b200, monkeypatch, env):
         gpu.close()
 
 
+@pytest.mark.parametrize("rows", [3, 7, 9, 16])
+def test_small_batches_on_the_tensor_pipe(b200, monkeypatch, rows):
+    # bf16 steps of 3 to 16 rows: products with K a multiple of 32 run on mma.sync (here every one; output counts that no tile of 16 divides
+    # included), and rows that choose more experts than there are take every expert once; B200_LP_GEMV_MMA=0 keeps the CUDA-core kernels
+    cfg = S.config([S.latent(heads=3, dim=16, rot_dim=8, vdim=32, mlp=S.moe(experts=4, top=2, ff=32, shared_ff=64)), S.latent(heads=2, vdim=16, mlp=S.dense(96))],
+                   width=96, vocab=101, taps=3, loop=(0, 1, 2))
+    w = S.random_weights(cfg, 48)
+    ref = Ref(cfg, w)
+    prompts = [tokens(2 + i % 5, cfg["vocab"], 80 + i) for i in range(rows)]
+    tails = [tokens(4, cfg["vocab"], 120 + i) for i in range(rows)]
+    out = {}
+    for mma in ("1", "0"):
+        monkeypatch.setenv("B200_LP_GEMV_MMA", mma)
+        gpu = S.gpu_model(cfg, w, "bfloat16", max_batch=rows, max_seq_len=32)
+        try:
+            gpu.step(list(enumerate(prompts)))
+            out[mma] = np.stack([gpu.decode_batch(list(range(rows)), [t[k] for t in tails]) for k in range(4)])
+        finally:
+            gpu.close()
+    d = np.array([[S.rel_err(out["1"][k][i], out["0"][k][i]) for i in range(rows)] for k in range(4)])
+    assert np.median(d) < 2e-2 and (d < 4e-2).mean() > 0.85
+    want = [ref.forward(prompts[i] + tails[i])[len(prompts[i]):] for i in range(rows)]
+    e = np.array([[S.rel_err(out["1"][k][i], want[i][k]) for i in range(rows)] for k in range(4)])
+    assert np.median(e) < BF16_TOL / 2
+
+
 def test_trace_runner_on_a_model_folder(b200, tmp_path):
     # config.json + model.safetensors (bf16) on disk -> registry -> bin/trace_run: two requests start together with unequal prompts, are
     # decoded together, the shorter one ends first; logits of the wanted rows come back in files
