@@ -317,10 +317,18 @@ B200_API const char* b200_batch_last_error(b200_batch* batch);   /* message of t
  * sigmoid(W_sg h), one number per token ('.shared.sg', [1, width]).
  * B200_FF_XIELU: W_down act(W_up h) of width ff with the two numbers (p, q) = '.act': act(z) = softplus(p) z^2 + z / 2 for z > 0,
  * (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 for z <= 0.
+ * B200_FF_GATED_RELU: W_down (relu(W_gate h) * W_up h) of width ff.
+ * sattn.v_from_k = 1: there is no W_v, a head's values are its keys as projected, before the norm (vdim = dim; with qk_norm NONE or
+ * HEAD_UNIT and no biases, convolution, rotation or value mixing): the cache holds those rows once, with one factor per row and head that
+ * makes the key of it.  sattn.q_temp_every > 0: the query of position p is multiplied by 1 + q_temp_coef ln(floor((p + 1) /
+ * q_temp_every) + 1) before its scores are taken.  latent.sink: as sattn.sink.
+ * moe.identity = n: the router has n more outputs behind the experts'; such an expert has no tensors, its output is what the feed-forward
+ * reads.  moe.correction = 1: '.correction' ([experts + identity]) is added to the scores that choose (B200_ROUTE_SOFTMAX_TOP: the
+ * probabilities, B200_ROUTE_SIGMOID_TOP: the sigmoids), the weights come from the scores without it.
  * parallel_ff = 1 (with post_norm = 0, streams = 0): a layer has one norm and its feed-forward reads the mixer's input,
  * h = norm1(x), x += mixer(h) + ff(h); the layer's input projection then also holds the feed-forward's ([gate | up] or the router).
- * Layer form (program): post_norm = 0: x += sublayer(norm(x)); post_norm = 1: x <- norm(residual_alpha * x + sublayer(x)), the
- * sublayers read x itself.  Norm weights are applied as (norm_weight_offset + w).  norm_kind = B200_NORM_LAYER: the layer norms and
+ * Layer form (program): post_norm = 0: x += sublayer(norm(x)); post_norm = 1: x <- norm(residual_alpha * x + sublayer(x));
+ * post_norm = 2: x <- residual_alpha * x + norm(sublayer(x)); in both the sublayers read x itself.  Norm weights are applied as (norm_weight_offset + w).  norm_kind = B200_NORM_LAYER: the layer norms and
  * the final norm subtract the mean first, (x - mean) / sqrt(var + eps) * w (no bias), instead of the RMS norm.
  * streams >= 1: the residual is `streams` copies x_1 .. x_s of the embedding; sublayer q of a layer (1 mixer, 2 feed-forward) reads
  * norm(sum_s hc<q>.in[s] x_s) and its output y updates all copies at once, x_t <- sum_s hc<q>.mix[s][t] x_s + residual_mult *
@@ -333,7 +341,8 @@ B200_API const char* b200_batch_last_error(b200_batch* batch);   /* message of t
  * ('l<i>.canon1' for the mixer, 'l<i>.canon2' for the feed-forward, [width, taps], conv(h)_t = sum_j w[:, j] h_(t - taps + 1 + j), zeros
  * before the sequence's start); a slot's state block keeps the last taps inputs per sublayer and layer run.  in_conv and loop_in belong to
  * the norm-first form with one residual stream and two norms per layer.
- * Embedding: row * embed_scale (+ sinusoidal position vector, pos_sinusoid); logits = head . norm(x) * logit_scale.
+ * Embedding: row * embed_scale (+ sinusoidal position vector, pos_sinusoid); logits = head . norm(x) * logit_scale; tied_head = 1: the
+ * head is the embedding table as stored, there is no 'head' tensor.
  * compute: 0 = bf16 weights and GEMM operands with f32 accumulation (residual stream, norms, softmax, gates and every recurrent
  * state stay f32), 1 = everything in f32 (FMA, no reduced-precision matrix mode). */
 enum { B200_MIX_WINDOW_MEMORY = 1, B200_MIX_GATED_DELTA = 2, B200_MIX_SOFTMAX_ATTN = 3, B200_MIX_LATENT_ATTN = 4, B200_MIX_STATE_SPACE = 5,
@@ -345,10 +354,11 @@ enum { B200_COMBINE_WEIGHTED = 0, B200_COMBINE_NORMED_MEAN = 1 };
 enum { B200_QKNORM_NONE = 0, B200_QKNORM_HEAD_WEIGHT = 1, B200_QKNORM_WHOLE_WEIGHT = 2, B200_QKNORM_HEAD_UNIT = 3 };
 enum { B200_GATE_NONE = 0, B200_GATE_CHANNEL = 1, B200_GATE_HEAD = 2 };
 enum { B200_VMIX_NONE = 0, B200_VMIX_SOURCE = 1, B200_VMIX_BLEND = 2 };
-enum { B200_FF_RELU2 = 0, B200_FF_GATED_GELU = 1, B200_FF_MOE = 2, B200_FF_CLAMPED_GLU = 3, B200_FF_XIELU = 4 };
+enum { B200_FF_RELU2 = 0, B200_FF_GATED_GELU = 1, B200_FF_MOE = 2, B200_FF_CLAMPED_GLU = 3, B200_FF_XIELU = 4, B200_FF_GATED_RELU = 5 };
 enum { B200_COMPUTE_BF16 = 0, B200_COMPUTE_F32 = 1 };
 enum { B200_NORM_RMS = 0, B200_NORM_LAYER = 1 };
-enum { B200_ACT_RELU2 = 0, B200_ACT_GELU = 1, B200_ACT_SILU_GLU = 2, B200_ACT_CLAMPED_GLU = 3 };
+enum { B200_FORM_NORM_FIRST = 0, B200_FORM_NORM_SUM = 1, B200_FORM_NORM_OUTPUT = 2 };   /* program.post_norm */
+enum { B200_ACT_RELU2 = 0, B200_ACT_GELU = 1, B200_ACT_SILU_GLU = 2, B200_ACT_CLAMPED_GLU = 3, B200_ACT_RELU_GLU = 4 };
 enum { B200_ROUTE_TOP_SOFTMAX = 0, B200_ROUTE_SOFTMAX_TOP = 1, B200_ROUTE_SIGMOID_TOP = 2 };
 enum { B200_TYPE_BF16 = 30 };   /* ggml's id; accepted by layer-program contexts only */
 typedef struct b200_window_attn_desc {
@@ -381,6 +391,9 @@ typedef struct b200_softmax_attn_desc {
     float v_rot_base;                /* > 0: values are turned by their position and the summed output is turned back */
     int32_t sink;                    /* B200_SINK_* */
     int32_t o_bias;                  /* 1 = '.o.b' is added by the output projection */
+    int32_t v_from_k;                /* 1 = the values are the projected keys before their norm */
+    float q_temp_coef;               /* query temperature (see above) */
+    int32_t q_temp_every;            /* 0 = none */
 } b200_softmax_attn_desc;
 typedef struct b200_moe_desc {
     int32_t experts, top, expert_ff, shared_ff;
@@ -391,6 +404,8 @@ typedef struct b200_moe_desc {
     float limit, shared_limit, slope;   /* B200_ACT_CLAMPED_GLU: clamps of the experts and of the always-on expert, slope of the gate */
     int32_t router_bias;             /* 1 = '.router.b' ([experts]) is added to the logits */
     int32_t shared_gate;             /* 1 = the always-on expert is multiplied by sigmoid('.shared.sg' h) */
+    int32_t identity;                /* router outputs behind the experts' whose expert is the input itself */
+    int32_t correction;              /* 1 = '.correction' is added to the scores that choose */
 } b200_moe_desc;
 /* Rotary frequencies: f_i = base^(-2i / dims), i < dims / 2.  yarn_factor > 0 stretches long wavelengths: with
  * d(t) = dims ln(yarn_original / (2 pi t)) / (2 ln base), lo = max(floor(d(yarn_fast)), 0), hi = min(ceil(d(yarn_slow)), dims - 1) and
@@ -410,6 +425,7 @@ typedef struct b200_latent_attn_desc {
     int32_t kv_from;                 /* -1: own W_dkv and cache rows; j: the rows of layer j */
     int32_t out_gate;                /* B200_GATE_* ('.g': [heads * vdim, width] or [heads, width]) */
     int32_t rot_pairs;               /* rotation layout: 0 = halves (i with i + dims / 2), 1 = neighbours (2i with 2i + 1) */
+    int32_t sink;                    /* B200_SINK_* ('.sink', [heads]) */
 } b200_latent_attn_desc;
 typedef struct b200_state_space_desc {
     int32_t heads, vdim, state, groups, conv, norm_groups;
@@ -444,8 +460,8 @@ typedef struct b200_program_desc {
     int32_t pos_sinusoid;                       /* 1 = add the sinusoidal position vector to the embedding */
     int32_t loop_start, loop_stop, loop_times;  /* layers [start, stop) run `times` times in a row; a step vector per pass */
     int32_t compute;                            /* B200_COMPUTE_* */
-    int32_t post_norm;                          /* 1 = norm after the residual sum (see "Layer form") */
-    float residual_alpha;                       /* post_norm: weight of x in the sum */
+    int32_t post_norm;                          /* B200_FORM_*: where the norms sit (see "Layer form") */
+    float residual_alpha;                       /* post_norm 1 and 2: weight of x in the sum */
     float norm_weight_offset;                   /* norm weights are stored minus this (0 or 1) */
     int32_t norm_kind;                          /* B200_NORM_* of the layer norms and the final norm */
     int32_t streams;                            /* 0: one residual stream in the forms above; >= 1: that many copies (see "streams") */
@@ -455,6 +471,7 @@ typedef struct b200_program_desc {
     int32_t embed_norm;                         /* 1 = the embedding is normed with 'embed.norm' */
     int32_t loop_in;                            /* 1 = 'loop.in' maps [x; x0] ahead of every pass of the repeated range */
     int32_t in_conv;                            /* taps of the convolution on every sublayer's input; 0 = none */
+    int32_t tied_head;                          /* 1 = the head is the embedding table */
 } b200_program_desc;
 B200_API int b200_ctx_create_layers(const b200_program_desc* prog, const b200_layer_desc* layers, int device, b200_ctx** out);
 /* One batch of token runs: run i continues sequence slot seqs[i] with lens[i] tokens (concatenated in `tokens`).  want_rows are

@@ -112,14 +112,15 @@ class SoftmaxAttnDesc(C.Structure):
                 ("rot_dims", C.c_int32), ("rot_base", C.c_float), ("softcap", C.c_float), ("dist_bias_exp", C.c_float),
                 ("v_mix", C.c_int32), ("out_gate", C.c_int32), ("yarn_factor", C.c_float), ("yarn_original", C.c_float),
                 ("yarn_fast", C.c_float), ("yarn_slow", C.c_float), ("rot_after_norm", C.c_int32), ("v_rot_base", C.c_float),
-                ("sink", C.c_int32), ("o_bias", C.c_int32)]
+                ("sink", C.c_int32), ("o_bias", C.c_int32), ("v_from_k", C.c_int32), ("q_temp_coef", C.c_float),
+                ("q_temp_every", C.c_int32)]
 
 
 class MoeDesc(C.Structure):
     """b200_moe_desc"""
     _fields_ = [("experts", C.c_int32), ("top", C.c_int32), ("expert_ff", C.c_int32), ("shared_ff", C.c_int32), ("act", C.c_int32),
                 ("route", C.c_int32), ("route_scale", C.c_float), ("weight_input", C.c_int32), ("limit", C.c_float), ("shared_limit", C.c_float),
-                ("slope", C.c_float), ("router_bias", C.c_int32), ("shared_gate", C.c_int32)]
+                ("slope", C.c_float), ("router_bias", C.c_int32), ("shared_gate", C.c_int32), ("identity", C.c_int32), ("correction", C.c_int32)]
 
 
 class RotaryDesc(C.Structure):
@@ -132,7 +133,7 @@ class LatentAttnDesc(C.Structure):
     """b200_latent_attn_desc"""
     _fields_ = [("heads", C.c_int32), ("dim", C.c_int32), ("rot_dim", C.c_int32), ("vdim", C.c_int32), ("q_rank", C.c_int32),
                 ("kv_rank", C.c_int32), ("mask_size", C.c_int32), ("scale", C.c_float), ("rot", RotaryDesc), ("kv_from", C.c_int32),
-                ("out_gate", C.c_int32), ("rot_pairs", C.c_int32)]
+                ("out_gate", C.c_int32), ("rot_pairs", C.c_int32), ("sink", C.c_int32)]
 
 
 class StateSpaceDesc(C.Structure):
@@ -167,12 +168,14 @@ class ProgramDesc(C.Structure):
                 ("pos_sinusoid", C.c_int32), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
                 ("compute", C.c_int32), ("post_norm", C.c_int32), ("residual_alpha", C.c_float), ("norm_weight_offset", C.c_float),
                 ("norm_kind", C.c_int32), ("streams", C.c_int32), ("residual_mult", C.c_float), ("parallel_ff", C.c_int32),
-                ("norm_scalar", C.c_int32), ("embed_norm", C.c_int32), ("loop_in", C.c_int32), ("in_conv", C.c_int32)]
+                ("norm_scalar", C.c_int32), ("embed_norm", C.c_int32), ("loop_in", C.c_int32), ("in_conv", C.c_int32),
+                ("tied_head", C.c_int32)]
 
 
 MIX_WINDOW_MEMORY, MIX_GATED_DELTA, MIX_SOFTMAX_ATTN, MIX_LATENT_ATTN, MIX_STATE_SPACE, MIX_ATTN_RECURRENT = 1, 2, 3, 4, 5, 6
 NORM_RMS, NORM_LAYER = 0, 1
-ACT_RELU2, ACT_GELU, ACT_SILU_GLU, ACT_CLAMPED_GLU = 0, 1, 2, 3
+FORM_NORM_FIRST, FORM_NORM_SUM, FORM_NORM_OUTPUT = 0, 1, 2
+ACT_RELU2, ACT_GELU, ACT_SILU_GLU, ACT_CLAMPED_GLU, ACT_RELU_GLU = 0, 1, 2, 3, 4
 ROUTE_TOP_SOFTMAX, ROUTE_SOFTMAX_TOP, ROUTE_SIGMOID_TOP = 0, 1, 2
 MASK_WINDOW, MASK_CHUNK, MASK_CAUSAL = 0, 1, 2
 SINK_NONE, SINK_LEARNED, SINK_ZERO = 0, 1, 2
@@ -181,7 +184,7 @@ COMBINE_WEIGHTED, COMBINE_NORMED_MEAN = 0, 1
 QKNORM_NONE, QKNORM_HEAD_WEIGHT, QKNORM_WHOLE_WEIGHT, QKNORM_HEAD_UNIT = 0, 1, 2, 3
 GATE_NONE, GATE_CHANNEL, GATE_HEAD = 0, 1, 2
 VMIX_NONE, VMIX_SOURCE, VMIX_BLEND = 0, 1, 2
-FF_RELU2, FF_GATED_GELU, FF_MOE, FF_CLAMPED_GLU, FF_XIELU = 0, 1, 2, 3, 4
+FF_RELU2, FF_GATED_GELU, FF_MOE, FF_CLAMPED_GLU, FF_XIELU, FF_GATED_RELU = 0, 1, 2, 3, 4, 5
 COMPUTE_BF16, COMPUTE_F32 = 0, 1
 BF16 = 30   # ggml's id; layer-program contexts only
 

@@ -62,10 +62,11 @@ struct StepMeta {
 
 // ------------------------------------------------------------------------------------------------ embedding
 // x[r] = table[token] * scale (+ sinusoidal position vector: entry 2i = sin(p w_i), entry 2i + 1 = cos(p w_i), w_i = 10000^(-2i/width)).
-// The angle and its sine are evaluated in double: at positions in the thousands an f32 angle alone is off by 1e-4.
+// The angle and its sine are evaluated in double: at positions in the thousands an f32 angle alone is off by 1e-4.  xc: the same in the
+// compute type, or null.
 template <typename T>
 __global__ void lp_embed_kernel(StepMeta sm, const T* __restrict__ table, const double* __restrict__ inv_freq, float* __restrict__ x,
-                                int width, float scale, int sinusoid) {
+                                int width, float scale, int sinusoid, T* __restrict__ xc) {
     const int r = blockIdx.x;
     const T* row = table + (size_t)sm.tok[r] * width;
     const double p = (double)sm.row_pos[r];
@@ -77,8 +78,15 @@ __global__ void lp_embed_kernel(StepMeta sm, const T* __restrict__ table, const 
             s = (float)ds;
             c = (float)dc;
         }
-        x[(size_t)r * width + 2 * i] = to_f(row[2 * i]) * scale + s;
-        if (2 * i + 1 < width) x[(size_t)r * width + 2 * i + 1] = to_f(row[2 * i + 1]) * scale + c;
+        const size_t o = (size_t)r * width + 2 * i;
+        const float v0 = to_f(row[2 * i]) * scale + s;
+        x[o] = v0;
+        if (xc) xc[o] = from_f<T>(v0);
+        if (2 * i + 1 < width) {
+            const float v1 = to_f(row[2 * i + 1]) * scale + c;
+            x[o + 1] = v1;
+            if (xc) xc[o + 1] = from_f<T>(v1);
+        }
     }
 }
 
@@ -133,17 +141,19 @@ __global__ void lp_rmsnorm_kernel(float* __restrict__ x, const float* __restrict
 // ------------------------------------------------------------------------------------------------ GEMM (CUDA cores)
 // Y[r][n] = epi(alpha * sum_k X[r][k] * W[n][k] + bias[n]); products of the stored operand values in f32, f32 accumulation
 // (bias: f32 per output column, or null).  act: the two numbers of the xIELU epilogue, (softplus(p), 1/2 + softplus(q)).
-enum { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2, EPI_GELU = 3, EPI_XIELU = 4, EPI_COUNT = 5 };
+// EPI_RELU_GLU: relu(v) * up, the unit of a gated layer from its two products (the kernels that have both at hand).
+enum { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2, EPI_GELU = 3, EPI_XIELU = 4, EPI_RELU_GLU = 5, EPI_COUNT = 6 };
 constexpr bool epi_is_act(int epi) { return epi >= EPI_RELU2; }
 // act.x z^2 + z / 2 above zero, act.y (exp(z) - 1 - z) + z / 2 below
 __device__ __forceinline__ float xielu_f(float z, float2 act) { return fmaf(0.5f, z, z > 0.0f ? act.x * z * z : act.y * (expm1f(z) - z)); }
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
 template <typename T, int EPI>
-__device__ __forceinline__ void epi_store(void* Y, size_t idx, float v, float2 act) {
+__device__ __forceinline__ void epi_store(void* Y, size_t idx, float v, float2 act, float up = 0.0f) {
     if (EPI == EPI_STORE) reinterpret_cast<float*>(Y)[idx] = v;
     else if (EPI == EPI_ADD) reinterpret_cast<float*>(Y)[idx] += v;
     else if (EPI == EPI_GELU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(gelu_erf_f(v));
     else if (EPI == EPI_XIELU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(xielu_f(v, act));
+    else if (EPI == EPI_RELU_GLU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(fmaxf(v, 0.0f) * up);
     else {
         const float z = fmaxf(v, 0.0f);
         reinterpret_cast<T*>(Y)[idx] = from_f<T>(z * z);
@@ -458,6 +468,7 @@ template <typename T, int NR> __device__ __forceinline__ void gemv_dot(const T* 
     }
 }
 #include "lp_input_conv.cuh"
+#include "lp_sublayer_norm.cuh"
 
 // the row count a few-row kernel is instantiated for: 1, 2, 4 or 8 (GV_ROWS) rows per pass over the weights
 #define LP_NR_DISPATCH(R, CALL)                                                                                        \
@@ -589,10 +600,11 @@ __global__ void __launch_bounds__(256) lp_gemv_mma_kernel(const bf16* __restrict
 // Every block repeats the norm (the rows are a few KB out of L2); a launch and a round trip through global memory go away.
 // ic.taps > 0 (decoding: one row per run): the normed row h becomes h + conv(h) before the rounding; every block reads the run's earlier
 // inputs, block 0 writes this position's (norm_conv_row; no other block reads that ring entry).
+// sn.on: instead of a norm, what lp_sub_norm_kernel does (the layer form with the norm on a sublayer's output).
 template <typename T, int EPI, int NR>
 __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restrict__ X, const int* __restrict__ gather, const float* __restrict__ nw,
                                                            float eps, const T* __restrict__ W, void* __restrict__ Y, int ldy, int R, int N, int K,
-                                                           float alpha, int center, T* __restrict__ hn_out, float2 act, InConv ic, StepMeta sm) {
+                                                           float alpha, int center, T* __restrict__ hn_out, float2 act, InConv ic, StepMeta sm, SubNorm sn) {
     extern __shared__ __align__(16) uint8_t gn_smem[];
     T* xs = reinterpret_cast<T*>(gn_smem);            // [R][K]
     __shared__ float red[8];
@@ -600,6 +612,10 @@ __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restri
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (blockIdx.x * 8 + warp < N) prefetch_row(W + (size_t)(blockIdx.x * 8 + warp) * K, K, lane);
     for (int r = 0; r < R; r++) {
+        if (sn.on) {         // (no gather; block 0 keeps the new stream, in another buffer than the one the blocks read)
+            sub_norm_row<T, 256>(sn, r, X + (size_t)r * K, blockIdx.x == 0 ? sn.xout + (size_t)r * K : (float*)nullptr, K, r & 1, xs + (size_t)r * K, (T*)nullptr);
+            continue;
+        }
         if (ic.taps > 0) {   // (RMS norm, no gather: checked by the host)
             norm_conv_row<T, 256>(ic, sm, r, X + (size_t)r * K, nw, K, eps, blockIdx.x == 0, xs + (size_t)r * K, nullptr);
             continue;
@@ -645,13 +661,14 @@ __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restri
         const T* wr = W + (size_t)n * K;
         for (int rb = 0; rb < R; rb += NR) {
             const int nr = min(NR, R - rb);
-            float acc[NR];
+            float acc[NR], accu[NR];
             gemv_dot<T, NR>(wr, xs + (size_t)rb * K, K, nr, K, lane, acc);
+            if (EPI == EPI_RELU_GLU) gemv_dot<T, NR>(wr + (size_t)N * K, xs + (size_t)rb * K, K, nr, K, lane, accu);     // (W: [gate | up], N units)
 #pragma unroll
             for (int i = 0; i < NR; i++) {
                 if (i < nr) {
-                    const float sum = wsum(acc[i]);
-                    if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + n, alpha * sum, act);
+                    const float sum = wsum(acc[i]), up = EPI == EPI_RELU_GLU ? wsum(accu[i]) : 0.0f;
+                    if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + n, alpha * sum, act, up);
                 }
             }
         }
@@ -674,11 +691,18 @@ struct AttnGeom {
     int chunk;                        // 1: the mask is chunks of `window` positions counted from position 0 instead of a sliding window
     float softcap;                    // > 0: score <- softcap tanh(score / softcap)
     float slope_exp;                  // > 0: score -= 2^(-slope_exp (h + 1) / H) (i - j)
-    int v_in_k;                       // 1: there are no value rows; a value is the first vdim entries of its (single, G = 1) key row
+    int v_in_k;                       // 1: there are no value rows; a value is the first vdim entries of its head's key row
+    int k_inv;                        // 1: keys and queries are over their root mean square; the rows hold the keys before that, their factors
+                                      //    [cap][G] sit behind the rows (v_in_k; lp_row_attn.cuh)
+    float temp_coef;                  // query temperature 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) at position p
+    int temp_every;                   // 0: none
     int sink_mode;                    // B200_SINK_*: one more term exp(c) in the softmax's denominator, without key or value
     const float* sink;                // [H]: c per head (B200_SINK_LEARNED)
     const float* vrot;                // [rows][vdim]: cos | sin of the angles that turn a row's summed values back, or null
 };
+__device__ __forceinline__ float attn_temp(const AttnGeom& a, int pos) {
+    return a.temp_every > 0 ? fmaf(a.temp_coef, logf((float)((pos + 1) / a.temp_every) + 1.0f), 1.0f) : 1.0f;
+}
 // the extra term of the denominator as the start of the running (maximum, sum): a key with score c and no value
 __device__ __forceinline__ bool attn_sink(const AttnGeom& a, int h, float* c) {
     if (a.sink_mode == B200_SINK_NONE) return false;
@@ -749,7 +773,8 @@ __global__ void __launch_bounds__(32 * ATT_WARPS) lp_window_attn_kernel(StepMeta
     const int g = h * a.G / a.H;
     const float* kc = reinterpret_cast<const float*>(sm.run_kv[run] + a.kv_off);
     const float* vc = a.v_in_k ? kc : kc + (size_t)a.cap * a.G * a.dim;
-    const int ldk = a.G * a.dim, ldv = a.v_in_k ? ldk : a.G * a.vdim;
+    const int ldk = a.G * a.dim, ldv = a.v_in_k ? ldk : a.G * a.vdim, gv = g * (a.v_in_k ? a.dim : a.vdim);
+    const float* kinv = a.k_inv ? kc + (size_t)a.cap * ldk + g : nullptr;
     if (a.fused_prep) {
         // what lp_attn_prep_kernel does, for this head and its K/V group only: warp 0 norms q into shared memory, warp 1 norms k
         // into the cache row of this position, the other warps copy v there.  Every head of a group writes the same values; a
@@ -836,6 +861,7 @@ __global__ void __launch_bounds__(32 * ATT_WARPS) lp_window_attn_kernel(StepMeta
             for (int d = 0; d < a.dim; d++) d0 = fmaf(qs[d], kr[d], d0);
             s = d0 * a.scale;
         }
+        if (kinv && j < end) s *= kinv[(size_t)j * a.G];
         if (j < end) s = attn_score(a, s, slope, i, j);
         const float m_new = fmaxf(m, wmax(s));
         const float p = j < end ? expf(s - m_new) : 0.0f;
@@ -853,7 +879,7 @@ __global__ void __launch_bounds__(32 * ATT_WARPS) lp_window_attn_kernel(StepMeta
             float vv[PVB][VCH];
 #pragma unroll
             for (int u = 0; u < PVB; u++) {
-                const float* vr = vc + (size_t)(j0 + min(jb + u, cnt - 1)) * ldv + g * a.vdim;
+                const float* vr = vc + (size_t)(j0 + min(jb + u, cnt - 1)) * ldv + gv;
 #pragma unroll
                 for (int c = 0; c < VCH; c++) {
                     const int ch = c * 32 + lane;
@@ -1442,6 +1468,7 @@ __global__ void lp_argmax_kernel(const float* __restrict__ logits, int vocab, in
 #include "lp_softmax_attn.cuh"
 #include "lp_ffn.cuh"
 #include "lp_streams.cuh"
+#include "lp_row_attn.cuh"
 #include "lp_latent_attn.cuh"
 #include "lp_state_space.cuh"
 #include "lp_gated_recurrent.cuh"
@@ -1514,12 +1541,13 @@ struct LayerPlan {
     int k_left = 0, k_right = 0;
     // parallel_ff: first column of the feed-forward's part ([gate | up], [up] or the router) in the layer's input projection
     int ff_off = -1;
+    const float* router_corr = nullptr;   // added to the scores that choose the experts
     int up_router_rows = 0;      // rows of the router at the head of w_up (0 when the router sits in the layer's input projection)
     // input convolutions of the two sublayers (ring_off: inside the run's state block), the xIELU numbers, the biases of the router's rows
     InConv ic[2];
     float2 act2 = float2{0.0f, 0.0f};
     const float* router_bias = nullptr;
-    int lat_splits = 0;          // latent attention: the largest row count x splits of the decoding kernels (0: they do not take these sizes)
+    int lat_splits = 0;          // attention over shared rows: the largest row count x splits of the decoding kernels (0: they do not take these sizes)
     // multi-stream layer form: [in | out | mix] of the two sublayers (null: identity)
     const float *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
 };
@@ -1551,13 +1579,13 @@ struct LpModel {
     uint8_t* h_meta = nullptr;          // pinned
     uint8_t* d_meta = nullptr;
     size_t meta_bytes = 0;
-    float *x = nullptr, *P = nullptr, *qbuf = nullptr, *O = nullptr, *conv = nullptr, *logits = nullptr;
+    float *x = nullptr, *x2 = nullptr, *P = nullptr, *qbuf = nullptr, *O = nullptr, *conv = nullptr, *logits = nullptr;
     float *y = nullptr, *vsrc = nullptr, *moe_w = nullptr, *moe_selw = nullptr;   // sublayer output (norm-after-sum layers), shared values, routing
     float* xs = nullptr;                // [rows][streams][width]: the residual copies of the multi-stream layer form
     void* cq = nullptr;                 // [rows][max_qrank] compute type: the normed query latent
     int max_qrank = 0;
     void* xcat = nullptr;               // [rows][2 width] compute type: [x; x0] ahead of a pass of the repeated range (program.loop_in)
-    float *lat_o = nullptr, *lat_ml = nullptr;   // decoding latent attention: the splits' sums and their (maximum, sum)
+    float *lat_o = nullptr, *lat_ml = nullptr;   // decoding attention over shared rows: the splits' sums and their (maximum, sum)
     size_t lat_o_floats = 0, lat_ml_floats = 0;
     size_t* ring_offs = nullptr;        // [n_convs] rings of the input convolutions inside a state block
     int n_convs = 0;
@@ -1598,7 +1626,7 @@ struct LpModel {
     int tc_min_rows = 17;
     bool use_gemv_mma = true;    // B200_LP_GEMV_MMA=0: small decode batches multiply on the CUDA cores
     int conv_fuse_rows = 1;      // B200_LP_CONV_FUSE_ROWS: decode steps of so many rows norm and convolve inside the projection
-    bool use_lat_split = true;   // B200_LP_LAT_SPLIT=0: decoding latent attention in the many-row kernels
+    bool use_lat_split = true;   // B200_LP_LAT_SPLIT=0: decoding attention over shared rows in the many-row kernels
     int* tc_err = nullptr;
     int* h_tc_err = nullptr;
     unsigned* tail_counter = nullptr;   // arrival counter of rows_tail (zero between kernels)
@@ -1841,12 +1869,12 @@ void rmsnorm(LpModel* m, float* x, const float* add, const float* w, void* out, 
 // written back into the stream).
 template <typename T>
 bool gemv_norm_t(LpModel* m, const float* x, const int* gather, const float* nw, const void* W, int N, int K, void* Y, int ldy, int R, float alpha,
-                 int epi, void* hn_out, float2 act, const InConv& ic, const StepMeta& sm) {
+                 int epi, void* hn_out, float2 act, const InConv& ic, const StepMeta& sm, const SubNorm& sn = SubNorm{}) {
     constexpr int VN = Vec8<T>::N;
     const size_t smem = (size_t)R * K * sizeof(T);
     if (R > 2 * GV_ROWS || K % VN || ((uintptr_t)W & 15) || smem > 96 * 1024) return false;
     if (sizeof(T) == 2 && R >= 3 && m->use_gemv_mma && K % 32 == 0) return false;      // (lp_gemv_mma_kernel behind a norm of its own)
-    if (epi != EPI_STORE && epi != EPI_RELU2 && epi != EPI_XIELU) return false;
+    if (epi != EPI_STORE && epi != EPI_RELU2 && epi != EPI_XIELU && epi != EPI_RELU_GLU) return false;
     static bool once[EPI_COUNT][GV_ROWS + 1][64] = {};
     int dev = 0;
     cudaGetDevice(&dev);
@@ -1863,16 +1891,19 @@ bool gemv_norm_t(LpModel* m, const float* x, const int* gather, const float* nw,
     const T* w = (const T*)W;
 #define LP_GN(E, NR)                                                                                                                       \
     if (!prep(lp_gemv_norm_kernel<T, E, NR>, E, NR)) return false;                                                                         \
-    launch(m, lp_gemv_norm_kernel<T, E, NR>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm)
+    launch(m, lp_gemv_norm_kernel<T, E, NR>, grid, block, smem, x, gather, nw, m->p.norm_eps, w, Y, ldy, R, N, K, alpha, norm_center(m), (T*)hn_out, act, ic, sm, sn)
 #define LP_GN_STORE(NR) LP_GN(EPI_STORE, NR)
 #define LP_GN_RELU2(NR) LP_GN(EPI_RELU2, NR)
 #define LP_GN_XIELU(NR) LP_GN(EPI_XIELU, NR)
+#define LP_GN_RELU_GLU(NR) LP_GN(EPI_RELU_GLU, NR)
     if (epi == EPI_STORE) LP_NR_DISPATCH(R, LP_GN_STORE);
     else if (epi == EPI_RELU2) LP_NR_DISPATCH(R, LP_GN_RELU2);
+    else if (epi == EPI_RELU_GLU) LP_NR_DISPATCH(R, LP_GN_RELU_GLU);
     else LP_NR_DISPATCH(R, LP_GN_XIELU);
 #undef LP_GN_STORE
 #undef LP_GN_RELU2
 #undef LP_GN_XIELU
+#undef LP_GN_RELU_GLU
 #undef LP_GN
     return true;
 }
@@ -1907,7 +1938,9 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
     const bool looped = p.loop_stop > p.loop_start;
     if (looped && (p.loop_start < 0 || p.loop_stop > p.n_layers || p.loop_times < 1)) return bad("bad repeated layer range");
     if (p.norm_kind != B200_NORM_RMS && p.norm_kind != B200_NORM_LAYER) return bad("unknown norm kind");
-    if (p.norm_kind == B200_NORM_LAYER && p.post_norm) return bad("the layer norm is not available in the norm-after-sum form");
+    if (p.post_norm < B200_FORM_NORM_FIRST || p.post_norm > B200_FORM_NORM_OUTPUT) return bad("unknown layer form (post_norm)");
+    if (p.post_norm == B200_FORM_NORM_OUTPUT && looped) return bad("the form with the norm on the output takes no repeated range");
+    if (p.norm_kind == B200_NORM_LAYER && p.post_norm == B200_FORM_NORM_SUM) return bad("the layer norm is not available in the norm-after-sum form");
     if (p.streams < 0 || p.streams > ST_MAX) return bad("streams must be 0 .. " + std::to_string(ST_MAX));
     if (p.streams > 0 && (p.post_norm || looped)) return bad("the multi-stream form takes neither the norm after the sum nor a repeated range");
     if (p.parallel_ff && (p.post_norm || p.streams > 0)) return bad("parallel_ff belongs to the norm-first form with one residual stream");
@@ -1946,7 +1979,13 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
             if (a.qk_norm < B200_QKNORM_NONE || a.qk_norm > B200_QKNORM_HEAD_UNIT) return bad(at + "unknown q/k norm");
             if (a.out_gate < B200_GATE_NONE || a.out_gate > B200_GATE_HEAD) return bad(at + "unknown output gate");
             if (a.v_mix < B200_VMIX_NONE || a.v_mix > B200_VMIX_BLEND) return bad(at + "unknown value mixing");
-            if (a.conv < 0 || a.softcap < 0.0f || a.dist_bias_exp < 0.0f) return bad(at + "negative attention constant");
+            if (a.conv < 0 || a.softcap < 0.0f || a.dist_bias_exp < 0.0f || a.q_temp_every < 0) return bad(at + "negative attention constant");
+            if (a.v_from_k) {
+                if (a.vdim != a.dim) return bad(at + "values taken from the keys have the keys' size");
+                if (L.mixer != B200_MIX_SOFTMAX_ATTN || a.qkv_bias || a.conv || a.rot_dims || a.v_rot_base > 0.0f || a.v_mix != B200_VMIX_NONE ||
+                    (a.qk_norm != B200_QKNORM_NONE && a.qk_norm != B200_QKNORM_HEAD_UNIT))
+                    return bad(at + "values taken from the keys go with neither biases, convolution, rotation, norm weights nor value mixing");
+            }
             if (a.v_mix == B200_VMIX_BLEND) {
                 int src = -1;
                 for (int j = 0; j < i; j++)
@@ -1975,6 +2014,7 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
             if (a.rot.yarn_factor < 0.0f || (a.rot.yarn_factor > 0.0f && !(a.rot.yarn_original > 0.0f && a.rot.yarn_fast > 0.0f && a.rot.yarn_slow > 0.0f)))
                 return bad(at + "bad rotary scaling");
             if (a.out_gate < B200_GATE_NONE || a.out_gate > B200_GATE_HEAD) return bad(at + "unknown output gate");
+            if (a.sink < B200_SINK_NONE || a.sink > B200_SINK_ZERO) return bad(at + "unknown sink kind");
             if (a.kv_from >= 0) {
                 if (a.kv_from >= i || layers[a.kv_from].mixer != B200_MIX_LATENT_ATTN || layers[a.kv_from].latent.kv_from >= 0)
                     return bad(at + "kv_from must name an earlier latent-attention layer with cache rows of its own");
@@ -1990,16 +2030,17 @@ int lp_create(const b200_program_desc* prog, const b200_layer_desc* layers, int 
         } else return bad(at + "unknown mixer");
         if (L.ff_kind == B200_FF_MOE) {
             const b200_moe_desc& e = L.moe;
-            if (e.experts <= 0 || e.top <= 0 || e.top > e.experts || e.expert_ff <= 0 || e.shared_ff < 0) return bad(at + "bad mixture-of-experts sizes");
-            if (e.act < B200_ACT_RELU2 || e.act > B200_ACT_CLAMPED_GLU || e.route < B200_ROUTE_TOP_SOFTMAX || e.route > B200_ROUTE_SIGMOID_TOP)
+            if (e.experts <= 0 || e.identity < 0 || e.top <= 0 || e.top > e.experts + e.identity || e.expert_ff <= 0 || e.shared_ff < 0) return bad(at + "bad mixture-of-experts sizes");
+            if (e.act < B200_ACT_RELU2 || e.act > B200_ACT_RELU_GLU || e.route < B200_ROUTE_TOP_SOFTMAX || e.route > B200_ROUTE_SIGMOID_TOP)
                 return bad(at + "unknown expert activation or routing rule");
             if (e.act == B200_ACT_CLAMPED_GLU && (!(e.limit > 0.0f) || (e.shared_ff > 0 && !(e.shared_limit > 0.0f)))) return bad(at + "clamped experts need positive limits");
+            if (e.correction && e.route == B200_ROUTE_TOP_SOFTMAX) return bad(at + "a correction of the choice needs scores (B200_ROUTE_SOFTMAX_TOP or B200_ROUTE_SIGMOID_TOP)");
             if (e.shared_gate && e.shared_ff <= 0) return bad(at + "a gate without an always-on expert");
             if (p.parallel_ff && (e.router_bias || e.shared_gate)) return bad(at + "parallel_ff takes no router bias and no gated always-on expert");
             if (e.weight_input && p.streams > 0) return bad(at + "weights on the experts' inputs are not available in the multi-stream form");
         } else if (L.ff_kind == B200_FF_CLAMPED_GLU) {
             if (L.ff > 0 && !(L.ff_limit > 0.0f)) return bad(at + "the clamped feed-forward needs a positive limit");
-        } else if (L.ff_kind != B200_FF_RELU2 && L.ff_kind != B200_FF_GATED_GELU && L.ff_kind != B200_FF_XIELU) return bad(at + "unknown feed-forward kind");
+        } else if (L.ff_kind != B200_FF_RELU2 && L.ff_kind != B200_FF_GATED_GELU && L.ff_kind != B200_FF_XIELU && L.ff_kind != B200_FF_GATED_RELU) return bad(at + "unknown feed-forward kind");
         if (L.ff < 0) return bad(at + "negative feed-forward width");
         if (L.ff_kind == B200_FF_XIELU && p.parallel_ff) return bad(at + "parallel_ff takes no xIELU feed-forward");
     }
@@ -2184,10 +2225,10 @@ int spread_norm(LpModel* m, const std::string& name, uint64_t n, std::string* er
 }
 double softplus_host(double z) { return std::max(z, 0.0) + std::log1p(std::exp(-std::fabs(z))); }
 
-// Splits of the decoding attention's keys for R rows: about two blocks per SM
-int latent_splits(int R, int heads) {
-    const int blocks = R * ((heads + LS_HEADS - 1) / LS_HEADS);
-    return std::max(1, std::min(64, 2 * 148 / blocks));
+// Splits of the decoding attention's keys for R rows: two blocks per SM, four of the smaller ones
+int row_splits(int R, int H, int G) {
+    const int per = H / G, nw = row_block_heads(per), blocks = R * G * ((per + nw - 1) / nw);
+    return std::max(1, std::min(64, (nw >= LS_HEADS ? 2 : 4) * 148 / blocks));
 }
 }  // namespace
 
@@ -2201,7 +2242,8 @@ int lp_finalize(LpModel* m, std::string* err) {
     void* dummy;
     if ((rc = need_mat(m, "embed", p.vocab, W, &dummy, err))) return rc;
     m->weight_bytes -= find(m, "embed")->bytes - W * elt(m);   // one row per token
-    if ((rc = need_mat(m, "head", p.vocab, W, &dummy, err))) return rc;
+    if (p.tied_head) m->weight_bytes += find(m, "embed")->bytes;
+    else if ((rc = need_mat(m, "head", p.vocab, W, &dummy, err))) return rc;
     const float* fv;
     if (p.norm_scalar) {
         std::vector<std::string> nm = {"final.norm", "embed.norm"};
@@ -2214,6 +2256,14 @@ int lp_finalize(LpModel* m, std::string* err) {
     if (p.embed_norm && (rc = need_vec(m, "embed.norm", W, &fv, err))) return rc;
     if (p.loop_in && (rc = need_mat(m, "loop.in", W, 2 * W, &dummy, err))) return rc;
     if (p.loop_stop > p.loop_start && (rc = need_vec(m, "loop.step", (uint64_t)p.loop_times * W, &fv, err))) return rc;
+    // room for the decoding kernels of attention over shared rows, when they take the layer's sizes
+    auto plan_row_splits = [&](LayerPlan& L) {
+        const AttnGeom& a = L.ag;
+        if (a.dim % 4 || row_split_smem(a.dim, row_block_heads(a.H / a.G)) > 200 * 1024) return;
+        for (int r = 1; r <= LS_ROWS; r++) L.lat_splits = std::max(L.lat_splits, r * row_splits(r, a.H, a.G));
+        m->lat_o_floats = std::max(m->lat_o_floats, (size_t)L.lat_splits * a.H * a.vdim);
+        m->lat_ml_floats = std::max(m->lat_ml_floats, (size_t)L.lat_splits * a.H * 2);
+    };
     for (int li = 0; li < p.n_layers; li++) {
         LayerPlan& L = m->plan[li];
         L.d = m->layers[li];
@@ -2274,8 +2324,9 @@ int lp_finalize(LpModel* m, std::string* err) {
             const bool dual = L.d.mixer == B200_MIX_ATTN_RECURRENT;
             const std::string x = pre + (dual ? "mix.left." : "mix."), rx = pre + "mix.right.";
             const uint64_t nq = (uint64_t)a.heads * a.dim, nk = (uint64_t)a.kv_heads * a.dim, nv = (uint64_t)a.kv_heads * a.vdim;
-            std::vector<std::string> names = {x + "q", x + "k", x + "v"};
-            std::vector<uint64_t> rows = {nq, nk, nv};
+            std::vector<std::string> names = {x + "q", x + "k"};
+            std::vector<uint64_t> rows = {nq, nk};
+            if (!a.v_from_k) { names.push_back(x + "v"); rows.push_back(nv); }
             if (a.out_gate) { names.push_back(x + "g"); rows.push_back(a.out_gate == B200_GATE_HEAD ? (uint64_t)a.heads : (uint64_t)a.heads * a.vdim); }
             const size_t n_left = names.size();
             if (dual && L.d.rec_kind == B200_REC_GATED_LINEAR) {
@@ -2292,8 +2343,9 @@ int lp_finalize(LpModel* m, std::string* err) {
             g.window = a.mask == B200_MASK_CAUSAL ? p.max_seq_len : a.mask_size;
             g.chunk = a.mask == B200_MASK_CHUNK ? 1 : 0; g.softcap = a.softcap; g.slope_exp = a.dist_bias_exp;
             g.qk_norm = 0; g.out_gate = a.out_gate; g.scale = a.scale; g.eps = p.norm_eps; g.cap = p.max_seq_len;
-            g.q_off = off[0]; g.k_off = off[1]; g.v_off = off[2]; g.g_off = a.out_gate ? off[3] : 0;
-            g.sink_mode = a.sink;
+            g.q_off = off[0]; g.k_off = off[1]; g.v_off = a.v_from_k ? off[1] : off[2]; g.g_off = a.out_gate ? off[a.v_from_k ? 2 : 3] : 0;
+            g.sink_mode = a.sink; g.temp_coef = a.q_temp_coef; g.temp_every = a.q_temp_every;
+            g.v_in_k = a.v_from_k ? 1 : 0; g.k_inv = a.v_from_k && a.qk_norm == B200_QKNORM_HEAD_UNIT ? 1 : 0;
             PrepGeom& q = L.pg;
             q.C = (int)(nq + nk + nv); q.taps = a.conv; q.qk_norm = a.qk_norm; q.rot_dims = a.rot_dims; q.v_mix = a.v_mix;
             q.rot_after_norm = a.rot_after_norm; q.rot_gain = 1.0f; q.v_rot = a.v_rot_base > 0.0f ? 1 : 0;
@@ -2346,7 +2398,8 @@ int lp_finalize(LpModel* m, std::string* err) {
             if (a.o_bias && (rc = need_vec(m, x + "o.b", W, &L.o_bias, err))) return rc;
             if (a.v_mix == B200_VMIX_BLEND && (rc = need_vec(m, x + "vmix", 1, &L.vmix, err))) return rc;
             L.k_left = a.heads * a.vdim;
-            L.kv_bytes = up16((size_t)p.max_seq_len * (nk + nv) * 4);
+            L.kv_bytes = up16((size_t)p.max_seq_len * (a.v_from_k ? nk + (uint64_t)a.kv_heads : nk + nv) * 4);
+            if (a.v_from_k && !a.out_gate) plan_row_splits(L);
             const size_t tail_bytes = q.taps > 1 ? up16((size_t)(q.taps - 1) * q.C * 4) : 0;
             L.rec_bytes = tail_bytes;
             m->max_q = std::max(m->max_q, (int)nq);
@@ -2447,7 +2500,8 @@ int lp_finalize(LpModel* m, std::string* err) {
             }
             AttnGeom& ag = L.ag;   // the cached rows as one K/V head: keys = the whole row, values = its first kv_rank entries
             ag.H = a.heads; ag.G = 1; ag.dim = (int)D; ag.vdim = a.kv_rank; ag.window = a.mask_size > 0 ? a.mask_size : p.max_seq_len;
-            ag.scale = a.scale; ag.eps = p.norm_eps; ag.cap = p.max_seq_len; ag.v_in_k = 1;
+            ag.scale = a.scale; ag.eps = p.norm_eps; ag.cap = p.max_seq_len; ag.v_in_k = 1; ag.sink_mode = a.sink;
+            if (a.sink == B200_SINK_LEARNED && (rc = need_vec(m, x + "sink", a.heads, &L.sink, err))) return rc;
             L.kv_bytes = own ? up16((size_t)p.max_seq_len * D * 4) : 0;
             L.kv_layer = own ? li : a.kv_from;
             m->max_act = std::max(m->max_act, (int)(H * std::max(std::max(a.dim, a.kv_rank), a.vdim)));
@@ -2457,11 +2511,7 @@ int lp_finalize(LpModel* m, std::string* err) {
             // decoding kernels: 16-byte loads of cached rows and weights, the rows in shared memory, two key tiles too
             const int vn = m->f32 ? 4 : 8;
             const size_t part = (size_t)2 * GV_ROWS * (std::max(a.dim, a.kv_rank) + std::max(64, a.rot.dims)) * 4;
-            if (D % 4 == 0 && a.kv_rank % vn == 0 && a.dim % vn == 0 && latent_split_smem((int)D) <= 200 * 1024 && part <= 190 * 1024) {
-                for (int r = 1; r <= LS_ROWS; r++) L.lat_splits = std::max(L.lat_splits, r * latent_splits(r, a.heads));
-                m->lat_o_floats = std::max(m->lat_o_floats, (size_t)L.lat_splits * a.heads * a.kv_rank);
-                m->lat_ml_floats = std::max(m->lat_ml_floats, (size_t)L.lat_splits * a.heads * 2);
-            }
+            if (a.kv_rank % vn == 0 && a.dim % vn == 0 && part <= 190 * 1024) plan_row_splits(L);
         } else if (L.d.mixer == B200_MIX_STATE_SPACE) {
             const b200_state_space_desc& g = L.d.ssd;
             const std::string x = pre + "mix.";
@@ -2571,20 +2621,22 @@ int lp_finalize(LpModel* m, std::string* err) {
             if (!par && (rc = need_vec(m, pre + "norm2", W, &L.norm2, err))) return rc;
             const bool glu = act_gated(e.act);
             const int per = glu ? 2 * e.expert_ff : e.expert_ff;   // rows of one expert's up matrix ([gate | up] when gated)
-            if (par && (rc = join_input({pre + "mlp.router"}, {(uint64_t)e.experts}))) return rc;
+            const int outs = e.experts + e.identity;               // outputs of the router
+            if (par && (rc = join_input({pre + "mlp.router"}, {(uint64_t)outs}))) return rc;
             std::vector<std::string> names, down;
             std::vector<uint64_t> rows;
-            if (!par) { names.push_back(pre + "mlp.router"); rows.push_back((uint64_t)e.experts); }
+            if (!par) { names.push_back(pre + "mlp.router"); rows.push_back((uint64_t)outs); }
             if (e.shared_gate) { names.push_back(pre + "mlp.shared.sg"); rows.push_back(1); }   // one more row of the router
-            L.up_router_rows = par ? 0 : e.experts + (e.shared_gate ? 1 : 0);
+            L.up_router_rows = par ? 0 : outs + (e.shared_gate ? 1 : 0);
+            if (e.correction && (rc = need_vec(m, pre + "mlp.correction", outs, &L.router_corr, err))) return rc;
             if (e.router_bias) {
                 const float* rb;
-                if ((rc = need_vec(m, pre + "mlp.router.b", e.experts, &rb, err))) return rc;
+                if ((rc = need_vec(m, pre + "mlp.router.b", outs, &rb, err))) return rc;
                 Tensor t;
                 t.rows = 1; t.cols = L.up_router_rows; t.bytes = t.cols * 4;
                 LCU_ALLOC(cudaMalloc(&t.d, up16(t.bytes)));
                 LCU(cudaMemset(t.d, 0, t.bytes));
-                LCU(cudaMemcpy(t.d, rb, (size_t)e.experts * 4, cudaMemcpyDeviceToDevice));
+                LCU(cudaMemcpy(t.d, rb, (size_t)outs * 4, cudaMemcpyDeviceToDevice));
                 m->tensors[pre + "mlp.router.b_cat"] = t;
                 L.router_bias = (const float*)t.d;
             }
@@ -2622,14 +2674,14 @@ int lp_finalize(LpModel* m, std::string* err) {
             Tensor t;
             t.d = L.w_down; t.matrix = true; t.rows = W; t.cols = L.k_down; t.bytes = W * (size_t)L.k_down * es;
             m->tensors[pre + "mlp.down_cat"] = t;
-            m->max_act = std::max(m->max_act, L.k_down);
+            m->max_act = std::max(m->max_act, std::max(L.k_down, e.top * e.expert_ff + e.shared_ff));   // (a row's choices side by side)
             m->max_in = std::max(m->max_in, std::max(L.n_up, e.experts * per));
-            m->weight_bytes -= (size_t)(e.experts - e.top) * (per + e.expert_ff) * W * es;   // a token reads its chosen experts only
-            m->max_experts = std::max(m->max_experts, e.experts);
+            m->weight_bytes -= (size_t)std::max(0, e.experts - e.top) * (per + e.expert_ff) * W * es;   // a token reads its chosen experts only
+            m->max_experts = std::max(m->max_experts, outs);
             m->max_top = std::max(m->max_top, e.top);
         } else if (L.d.ff > 0) {
             if (!par && (rc = need_vec(m, pre + "norm2", W, &L.norm2, err))) return rc;
-            const bool two = L.d.ff_kind == B200_FF_GATED_GELU || L.d.ff_kind == B200_FF_CLAMPED_GLU;
+            const bool two = L.d.ff_kind == B200_FF_GATED_GELU || L.d.ff_kind == B200_FF_CLAMPED_GLU || L.d.ff_kind == B200_FF_GATED_RELU;
             if (par) {
                 if (two) rc = join_input({pre + "mlp.gate", pre + "mlp.up"}, {(uint64_t)L.d.ff, (uint64_t)L.d.ff});
                 else rc = join_input({pre + "mlp.up"}, {(uint64_t)L.d.ff});
@@ -2656,14 +2708,14 @@ int lp_finalize(LpModel* m, std::string* err) {
             }
             L.k_down = L.d.ff;
             m->max_act = std::max(m->max_act, L.d.ff);
-        } else if (p.post_norm && find(m, pre + "norm2")) {   // a layer without feed-forward whose file still holds the second norm
+        } else if (p.post_norm == B200_FORM_NORM_SUM && find(m, pre + "norm2")) {   // a layer without feed-forward whose file still holds the second norm
             if ((rc = need_vec(m, pre + "norm2", W, &L.norm2, err))) return rc;
         }
     }
     {   // the preparation kernel of the softmax mixer keeps a row's q, k, v in shared memory
         size_t need = 0;
         for (const LayerPlan& L : m->plan)
-            if (L.d.mixer == B200_MIX_SOFTMAX_ATTN || L.d.mixer == B200_MIX_ATTN_RECURRENT)
+            if ((L.d.mixer == B200_MIX_SOFTMAX_ATTN || L.d.mixer == B200_MIX_ATTN_RECURRENT) && !L.d.sattn.v_from_k)
                 need = std::max(need, (size_t)(((L.pg.C + 3) & ~3) + L.pg.rot_dims + (L.pg.v_rot ? L.ag.vdim : 0)) * 4);
         if (need > 200 * 1024) return lp_fail(err, B200_ERR_UNSUPPORTED, "softmax mixer: q, k and v of one token exceed 200 KB of shared memory");
         if (need > 32 * 1024) LCU(cudaFuncSetAttribute(lp_attn_prep2_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)need));
@@ -2672,9 +2724,9 @@ int lp_finalize(LpModel* m, std::string* err) {
         LCU_ALLOC(cudaMalloc((void**)&m->lat_o, up16(m->lat_o_floats * 4)));
         LCU_ALLOC(cudaMalloc((void**)&m->lat_ml, up16(m->lat_ml_floats * 4)));
         const int sb = 200 * 1024, pb = 200 * 1024;
-        LCU(cudaFuncSetAttribute(lp_latent_split_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
-        LCU(cudaFuncSetAttribute(lp_latent_split_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
-        LCU(cudaFuncSetAttribute(lp_latent_split_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
+        LCU(cudaFuncSetAttribute(lp_row_split_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
+        LCU(cudaFuncSetAttribute(lp_row_split_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
+        LCU(cudaFuncSetAttribute(lp_row_split_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, sb));
         LCU(cudaFuncSetAttribute(lp_latent_absorb_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, pb));
         LCU(cudaFuncSetAttribute(lp_latent_absorb_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, pb));
         LCU(cudaFuncSetAttribute(lp_latent_merge_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, pb));
@@ -2707,7 +2759,7 @@ int lp_finalize(LpModel* m, std::string* err) {
         m->weight_bytes += 0;
         if (L.d.mixer == B200_MIX_WINDOW_MEMORY) m->kv_bytes_per_pos += (size_t)L.d.attn.kv_heads * (L.d.attn.dim + L.d.attn.vdim) * 4;
         if (L.d.mixer == B200_MIX_SOFTMAX_ATTN || L.d.mixer == B200_MIX_ATTN_RECURRENT)
-            m->kv_bytes_per_pos += (size_t)L.d.sattn.kv_heads * (L.d.sattn.dim + L.d.sattn.vdim) * 4;
+            m->kv_bytes_per_pos += (size_t)L.d.sattn.kv_heads * (L.d.sattn.dim + (L.d.sattn.v_from_k ? 1 : L.d.sattn.vdim)) * 4;
         if (L.d.mixer == B200_MIX_LATENT_ATTN && L.d.latent.kv_from < 0) m->kv_bytes_per_pos += (size_t)(L.d.latent.kv_rank + L.d.latent.rot_dim) * 4;
     }
     if (p.in_conv > 1) {   // the rings of all layer runs: convolution i of the order in which a step meets them
@@ -2767,7 +2819,7 @@ void lp_destroy(LpModel* m) {
     for (SlotMem& s : m->pool) { cudaFree(s.kv); cudaFree(s.rec); }
     for (void* ptr : {(void*)m->inv_freq, (void*)m->d_meta, (void*)m->x, (void*)m->P, (void*)m->qbuf, (void*)m->O, (void*)m->conv, (void*)m->logits,
                       m->hn, m->act_a, m->hw, (void*)m->pick, (void*)m->taps, (void*)m->glin_carry, (void*)m->y, (void*)m->vsrc, (void*)m->moe_w, (void*)m->moe_selw,
-                      (void*)m->moe_sel, (void*)m->moe_pos, (void*)m->moe_seg, m->moe_xp, (void*)m->moe_yp, (void*)m->xs, m->cq, (void*)m->vrot, m->xcat,
+                      (void*)m->moe_sel, (void*)m->moe_pos, (void*)m->moe_seg, m->moe_xp, (void*)m->moe_yp, (void*)m->xs, (void*)m->x2, m->cq, (void*)m->vrot, m->xcat,
                       (void*)m->lat_o, (void*)m->lat_ml, (void*)m->moe_shw, (void*)m->ring_offs, (void*)m->conv_pend})
         cudaFree(ptr);
     if (m->h_meta) cudaFreeHost(m->h_meta);
@@ -2828,6 +2880,7 @@ int ensure_scratch(LpModel* m, int R, int n_runs, int n_want, std::string* err) 
     if (R > m->cap_rows) {
         const int cap = std::max(R, std::min(2 * m->cap_rows, 1 << 20));
         if ((rc = grow(&m->x, (size_t)cap * W * 4, err))) return rc;
+        if (m->p.post_norm == B200_FORM_NORM_OUTPUT && (rc = grow(&m->x2, (size_t)cap * W * 4, err))) return rc;
         if ((rc = grow(&m->P, (size_t)cap * m->max_in * 4, err))) return rc;
         if ((rc = grow(&m->qbuf, (size_t)cap * std::max(m->max_q, 1) * 4, err))) return rc;
         if ((rc = grow(&m->O, (size_t)cap * std::max(m->max_o, 1) * 4, err))) return rc;
@@ -2898,27 +2951,28 @@ bool attn_tile(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int ldp, int 
     return attn_tile_launch<128, 256>(m, sm, ag, ldp, n_runs, max_len);
 }
 
-// The same for latent attention (lp_latent_tile_kernel): cached rows a multiple of 16 wide up to 320, latents a multiple of 8 up to 256
+// The same over rows that hold keys and values (lp_row_tile_kernel): rows a multiple of 16 wide up to 320, values a multiple of 8 up to 256
 template <int DK, int DV>
-bool latent_tile_launch(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int n_runs, int max_len) {
+bool row_tile_launch(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int n_runs, int max_len) {
     static bool once[64] = {};
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64 || !once[dev]) {
-        if (cudaFuncSetAttribute(lp_latent_tile_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_tile_smem<DK>()) != cudaSuccess) {
+        if (cudaFuncSetAttribute(lp_row_tile_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)row_tile_smem<DK>()) != cudaSuccess) {
             cudaGetLastError();
             return false;
         }
         if (dev >= 0 && dev < 64) once[dev] = true;
     }
-    launch(m, lp_latent_tile_kernel<DK, DV>, dim3((unsigned)(((size_t)max_len * ag.H + LT_ROWS - 1) / LT_ROWS), n_runs), dim3(256), latent_tile_smem<DK>(), sm, ag,
+    launch(m, lp_row_tile_kernel<DK, DV>, dim3((unsigned)(((size_t)max_len * (ag.H / ag.G) + LT_ROWS - 1) / LT_ROWS), n_runs, ag.G), dim3(256), row_tile_smem<DK>(), sm, ag,
            (const float*)m->qbuf, (bf16*)m->act_a);
     return true;
 }
-bool latent_tile(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int n_runs, int max_len) {
-    if (m->f32 || !m->use_attn_tile || max_len < 16 || ag.dim % 16 || ag.vdim % 8) return false;
-    if (ag.dim <= 128 && ag.vdim <= 128) return latent_tile_launch<128, 128>(m, sm, ag, n_runs, max_len);
-    if (ag.dim <= 320 && ag.vdim <= 256) return latent_tile_launch<320, 256>(m, sm, ag, n_runs, max_len);
+bool row_tile(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int n_runs, int max_len) {
+    if (m->f32 || !m->use_attn_tile || max_len < 16 || ag.dim % 16 || ag.vdim % 8 || ag.chunk || ag.keep_first || ag.slope_exp > 0.0f || ag.out_gate) return false;
+    if (ag.dim <= 64 && ag.vdim <= 64) return row_tile_launch<64, 64>(m, sm, ag, n_runs, max_len);
+    if (ag.dim <= 128 && ag.vdim <= 128) return row_tile_launch<128, 128>(m, sm, ag, n_runs, max_len);
+    if (ag.dim <= 320 && ag.vdim <= 256) return row_tile_launch<320, 256>(m, sm, ag, n_runs, max_len);
     return false;
 }
 
@@ -2947,6 +3001,20 @@ void attn_rows(LpModel* m, const StepMeta& sm, const AttnGeom& ag, const LayerPl
 #undef LP_ATTN
 }
 
+// Decoding over shared rows: the split kernel (with P: the preparation of the row in it) and the merge into m->act_a
+void row_split(LpModel* m, const StepMeta& sm, const AttnGeom& ag, const float* P, int ldp, int R, int splits) {
+    const int per = ag.H / ag.G, nw = row_block_heads(per);
+    const dim3 grid(splits, R, ag.G * ((per + nw - 1) / nw)), block(32 * nw);
+    const size_t smem = row_split_smem(ag.dim, nw);
+#define LP_RS(V) launch(m, lp_row_split_kernel<V>, grid, block, smem, sm, ag, (const float*)m->qbuf, P, ldp, m->lat_o, m->lat_ml)
+    if (ag.vdim <= 128) LP_RS(4); else if (ag.vdim <= 256) LP_RS(8); else LP_RS(16);
+#undef LP_RS
+}
+void row_combine(LpModel* m, const AttnGeom& ag, int R, int splits) {
+    if (m->f32) launch(m, lp_row_combine_kernel<float>, dim3(R, ag.H), dim3(128), 0, ag.H, ag.vdim, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (float*)m->act_a, ag.out_ld);
+    else launch(m, lp_row_combine_kernel<bf16>, dim3(R, ag.H), dim3(128), 0, ag.H, ag.vdim, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (bf16*)m->act_a, ag.out_ld);
+}
+
 // Every kernel of one step, in order, on the model's stream: eagerly, or while the stream is being captured into a CUDA graph (a
 // decode step: one row per run, nothing allocated).  head: 0 = no logits, 1 = logits of the wanted rows, 2 = their greedy picks.
 void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want, int head, int taps_len, int max_len) {
@@ -2954,19 +3022,41 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
     const int W = p.width;
     const float* loop_step = p.loop_stop > p.loop_start ? (const float*)find(m, "loop.step")->d : nullptr;
     // embedding
-    if (m->f32) launch(m, lp_embed_kernel<float>, dim3(R), dim3(128), 0, sm, (const float*)find(m, "embed")->d, m->inv_freq, m->x, W, p.embed_scale, p.pos_sinusoid);
-    else launch(m, lp_embed_kernel<bf16>, dim3(R), dim3(128), 0, sm, (const bf16*)find(m, "embed")->d, m->inv_freq, m->x, W, p.embed_scale, p.pos_sinusoid);
+    void* xc0 = p.post_norm ? m->hn : nullptr;      // (the forms whose sublayers read the stream itself: its copy in the compute type)
+    if (m->f32) launch(m, lp_embed_kernel<float>, dim3(R), dim3(128), 0, sm, (const float*)find(m, "embed")->d, m->inv_freq, m->x, W, p.embed_scale, p.pos_sinusoid, (float*)xc0);
+    else launch(m, lp_embed_kernel<bf16>, dim3(R), dim3(128), 0, sm, (const bf16*)find(m, "embed")->d, m->inv_freq, m->x, W, p.embed_scale, p.pos_sinusoid, (bf16*)xc0);
     if (p.embed_norm || p.loop_in) {   // the embedding's norm; with loop_in its copy x0 for the passes of the repeated range
         const float* g = p.embed_norm ? (const float*)find(m, "embed.norm")->d : nullptr;
         if (m->f32) launch(m, lp_embed_norm_kernel<float>, dim3(R), dim3(256), 0, m->x, g, W, p.norm_eps, p.embed_norm, (float*)m->xcat);
         else launch(m, lp_embed_norm_kernel<bf16>, dim3(R), dim3(256), 0, m->x, g, W, p.norm_eps, p.embed_norm, (bf16*)m->xcat);
     }
-    // The two layer forms.  Norm first: a sublayer reads norm(x) and its output projection adds into x.  Norm after the sum
-    // (post_norm): a sublayer reads x itself -- m->hn holds x in the compute type -- its output projection goes to m->y, and
-    // lp_postnorm_kernel makes x <- norm(alpha x + y) and the next copy.
+    // The layer forms.  Norm first: a sublayer reads norm(x) and its output projection adds into x.  Norm after the sum
+    // (post_norm 1): a sublayer reads x itself -- m->hn holds x in the compute type -- its output projection goes to m->y, and
+    // lp_postnorm_kernel makes x <- norm(alpha x + y) and the next copy.  Norm on the output (post_norm 2): the same with x <- alpha x +
+    // norm(y), which waits in `sub_pend` until somebody asks for x: the next projection of a few rows makes the new x itself (into
+    // m->x2, the two buffers then change places), otherwise lp_sub_norm_kernel.
     // Multi-stream form (p.streams >= 1): the copies live in m->xs; a sublayer's output goes to m->y and waits in `pend` until the
     // next sublayer (or the head) asks for its input: lp_streams_kernel then updates the copies and norms their weighted sum into m->hn.
-    const bool post = p.post_norm != 0, streams = p.streams > 0;
+    const bool post = p.post_norm != 0, streams = p.streams > 0, out_norm = p.post_norm == B200_FORM_NORM_OUTPUT;
+    SubNorm sub_pend{};
+    // x as the sublayer before left it, and its copy in m->hn; with a router: its logits and the choice (one token per run or few rows)
+    auto settle = [&](const StepRoute& rt) {
+        if (!sub_pend.y && !rt.router) return;
+        SubNorm sn = sub_pend;
+        sn.xout = m->x;
+        const size_t smem = rt.router ? (size_t)W * elt(m) : 0;
+        if (rt.router) {
+            if (m->f32) launch(m, lp_sub_norm_kernel<float, 512>, dim3(R), dim3(512), smem, sn, (const float*)m->x, W, (float*)m->hn, rt);
+            else launch(m, lp_sub_norm_kernel<bf16, 512>, dim3(R), dim3(512), smem, sn, (const float*)m->x, W, (bf16*)m->hn, rt);
+        } else {
+            if (m->f32) launch(m, lp_sub_norm_kernel<float, 256>, dim3(R), dim3(256), smem, sn, (const float*)m->x, W, (float*)m->hn, rt);
+            else launch(m, lp_sub_norm_kernel<bf16, 256>, dim3(R), dim3(256), smem, sn, (const float*)m->x, W, (bf16*)m->hn, rt);
+        }
+        sub_pend.y = nullptr;
+    };
+    auto pend_output = [&](const float* nw) {
+        sub_pend.on = 1; sub_pend.y = m->y; sub_pend.w = nw; sub_pend.alpha = p.residual_alpha; sub_pend.eps = p.norm_eps; sub_pend.center = norm_center(m);
+    };
     struct {
         const float *y, *mix, *out;
         bool src;
@@ -3068,12 +3158,25 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         } else if (streams) {
             boundary(cur->hc_in[sub], nw, nullptr);
             gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, nullptr, act);
+        } else if (out_norm) {
+            if (sub_pend.y && m->use_fuse) {
+                SubNorm sn = sub_pend;
+                sn.xout = m->x2;
+                if (m->f32 ? gemv_norm_t<float>(m, m->x, nullptr, nullptr, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, act, InConv{}, sm, sn)
+                           : gemv_norm_t<bf16>(m, m->x, nullptr, nullptr, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, act, InConv{}, sm, sn)) {
+                    std::swap(m->x, m->x2);
+                    sub_pend.y = nullptr;
+                    return;
+                }
+            }
+            settle(StepRoute{});
+            gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, nullptr, act);
         } else if (post) gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, nullptr, act);
         else norm_gemm(m, m->x, add, nullptr, nw, m->hn, Wm, N, Y, ldy, R, 1.0f, epi, p.parallel_ff != 0, act);   // (parallel_ff: the experts read m->hn later)
     };
     // Few rows (decoding) in the norm-after-sum form: the kernel that writes m->y also does what follows it -- its last block norms the
     // rows and, when `moe` follows, computes the router's logits and choices (rows_tail) -- instead of two or three more launches.
-    const bool few = post && m->use_fuse && R <= 2 * GV_ROWS;
+    const bool few = post && !out_norm && m->use_fuse && R <= 2 * GV_ROWS;
     auto make_tail = [&](const float* nw, const LayerPlan* moe) {
         RowsTail t{};
         t.on = 1; t.x = m->x; t.y = m->y; t.w = nw; t.xc = m->hn; t.width = W; t.R = R; t.alpha = p.residual_alpha; t.eps = p.norm_eps;
@@ -3095,12 +3198,14 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         } else if (few) {
             const RowsTail t = make_tail(nw, moe);
             gemm(m, X, K, Wm, W, K, m->y, W, R, 1.0f, EPI_STORE, &t, bias);
+        } else if (out_norm) {
+            gemm(m, X, K, Wm, W, K, m->y, W, R, 1.0f, EPI_STORE, nullptr, bias);
+            pend_output(nw);
         } else if (post) {
             gemm(m, X, K, Wm, W, K, m->y, W, R, 1.0f, EPI_STORE, nullptr, bias);
             cast_x(m->y, nw);
         } else gemm(m, X, K, Wm, W, K, m->x, W, R, 1.0f, EPI_ADD, nullptr, bias);
     };
-    if (post) cast_x(nullptr, nullptr);
     for (size_t run = 0; run < m->runs.size(); run++) {
         LayerPlan& L = m->plan[m->runs[run]];
         const float* add = m->run_pass[run] >= 0 ? loop_step + (size_t)m->run_pass[run] * W : nullptr;
@@ -3125,14 +3230,35 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
         const bool many_choices = !m->f32 && m->use_gemv_mma && R >= 3 && L.d.ff_kind == B200_FF_MOE && R * L.d.moe.top > L.d.moe.experts && W % 32 == 0 && L.k_down % 32 == 0;
         const bool moe_sel_ok = L.d.ff_kind == B200_FF_MOE && !many_choices && m->use_fuse && R <= 2 * GV_ROWS && W % (m->f32 ? 4 : 8) == 0 &&
                                 L.d.moe.expert_ff % (m->f32 ? 4 : 8) == 0 && L.d.moe.shared_ff % (m->f32 ? 4 : 8) == 0 && (size_t)R * W * elt(m) <= 40 * 1024;
-        // (the fused tails know neither a router bias nor the always-on expert's gate)
-        const LayerPlan* moe_next = ((few || sfew) && moe_sel_ok && !L.d.moe.router_bias && !L.d.moe.shared_gate) ? &L : nullptr;      // the mixer's output kernel also routes
+        // (the fused tails know neither a router bias, the always-on expert's gate, a correction nor identity experts)
+        const bool tail_routes = !L.d.moe.router_bias && !L.d.moe.shared_gate && !L.d.moe.correction && !L.d.moe.identity;
+        const LayerPlan* moe_next = ((few || sfew) && moe_sel_ok && tail_routes) ? &L : nullptr;      // the mixer's output kernel also routes
         cur = &L;
         sub = 0;
         cur_run = run;
-        cur_moe_sel = moe_sel_ok && !L.d.moe.router_bias && !L.d.moe.shared_gate;
+        cur_moe_sel = moe_sel_ok && tail_routes;
         project_in(add, L.norm1, L.w_in, L.n_in, m->P, L.n_in, EPI_STORE);
-        if (L.d.mixer == B200_MIX_SOFTMAX_ATTN || L.d.mixer == B200_MIX_ATTN_RECURRENT) {
+        if (L.d.mixer == B200_MIX_SOFTMAX_ATTN && L.d.sattn.v_from_k) {
+            // keys and values in the same rows (lp_row_attn.cuh)
+            AttnGeom ag = L.ag;
+            ag.kv_off = m->run_kv_off[run];
+            ag.out_ld = L.k_left;
+            ag.out_scale = 1.0f;
+            ag.sink = L.sink;
+            const bool v4 = ag.dim % 4 == 0 && L.n_in % 4 == 0;
+            const bool split = m->use_fuse && m->use_lat_split && max_len == 1 && R <= LS_ROWS && L.lat_splits > 0;
+            if (!(split && v4)) {
+                const dim3 pgrid((unsigned)(((size_t)R * (ag.H + ag.G) + 7) / 8));
+                if (v4) launch(m, lp_row_prep_kernel<4>, pgrid, dim3(256), 0, sm, ag, (const float*)m->P, L.n_in, m->qbuf, R);
+                else launch(m, lp_row_prep_kernel<1>, pgrid, dim3(256), 0, sm, ag, (const float*)m->P, L.n_in, m->qbuf, R);
+            }
+            if (split) {
+                const int splits = row_splits(R, ag.H, ag.G);
+                row_split(m, sm, ag, v4 ? m->P : nullptr, L.n_in, R, splits);
+                row_combine(m, ag, R, splits);
+            } else if (!row_tile(m, sm, ag, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
+            project_out(m->act_a, ag.out_ld, L.wo, L.norm1, moe_next, L.o_bias);
+        } else if (L.d.mixer == B200_MIX_SOFTMAX_ATTN || L.d.mixer == B200_MIX_ATTN_RECURRENT) {
             const bool dual = L.d.mixer == B200_MIX_ATTN_RECURRENT, weighted = dual && L.d.combine == B200_COMBINE_WEIGHTED;
             AttnGeom ag = L.ag;
             ag.kv_off = m->run_kv_off[run];
@@ -3250,18 +3376,17 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             ag.out_ld = a.heads * a.kv_rank;
             ag.out_scale = 1.0f;
             ag.fused_prep = 0;
-#define LP_LS(V) launch(m, lp_latent_split_kernel<V>, sgrid, dim3(32 * LS_HEADS), latent_split_smem(D), sm, ag, (const float*)m->qbuf, m->lat_o, m->lat_ml)
-#define LP_LS_ANY() do { if (a.kv_rank <= 128) LP_LS(4); else if (a.kv_rank <= 256) LP_LS(8); else LP_LS(16); } while (0)
+            ag.sink = L.sink;
             if (few_lat) {
                 const float* Q = direct ? m->P + lg.q_off : m->O;
-                const int ldq = direct ? L.n_in : a.heads * per, vn = m->f32 ? 4 : 8, splits = latent_splits(R, a.heads);
+                const int ldq = direct ? L.n_in : a.heads * per, vn = m->f32 ? 4 : 8, splits = row_splits(R, a.heads, 1);
                 const int uk_cols = 8 * (32 / latent_lanes(a.dim, vn)), uk_ch = (a.kv_rank + uk_cols - 1) / uk_cols;
                 const int uv_cols = 8 * (32 / latent_lanes(a.kv_rank, vn)), uv_ch = (a.vdim + uv_cols - 1) / uv_cols;
-                const dim3 agrid(a.heads * uk_ch + (direct && own ? R : 0)), sgrid(splits, R, (a.heads + LS_HEADS - 1) / LS_HEADS), ugrid(a.heads * uv_ch);
+                const dim3 agrid(a.heads * uk_ch + (direct && own ? R : 0)), ugrid(a.heads * uv_ch);
                 const size_t asm_ = (size_t)(R * a.dim + lg.rot_n) * 4, usm = ((size_t)R * (a.kv_rank + splits) + 1024 + 4) * 4;
                 if (m->f32) launch(m, lp_latent_absorb_kernel<float>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const float*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
                 else launch(m, lp_latent_absorb_kernel<bf16>, agrid, dim3(256), asm_, sm, lg, Q, ldq, (const float*)m->P, L.n_in, (const bf16*)L.w_ukT, L.dkv_norm, L.rot_freq, m->qbuf, R, uk_ch);
-                LP_LS_ANY();
+                row_split(m, sm, ag, nullptr, 0, R, splits);
                 if (m->f32) launch(m, lp_latent_merge_kernel<float>, ugrid, dim3(256), usm, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (const float*)L.w_uv, (const float*)m->P, L.n_in, (float*)m->act_a, R, uv_ch);
                 else launch(m, lp_latent_merge_kernel<bf16>, ugrid, dim3(256), usm, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (const bf16*)L.w_uv, (const float*)m->P, L.n_in, (bf16*)m->act_a, R, uv_ch);
             } else {
@@ -3271,20 +3396,16 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                 }
                 gemm_heads(m, m->act_a, a.heads * a.dim, a.dim, L.w_ukT, a.heads, a.kv_rank, a.dim, m->qbuf, a.heads * D, D, R);
                 if (split) {
-                    const int splits = latent_splits(R, a.heads);
-                    const dim3 sgrid(splits, R, (a.heads + LS_HEADS - 1) / LS_HEADS);
-                    LP_LS_ANY();
-                    if (m->f32) launch(m, lp_latent_combine_kernel<float>, dim3(R, a.heads), dim3(128), 0, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (float*)m->act_a);
-                    else launch(m, lp_latent_combine_kernel<bf16>, dim3(R, a.heads), dim3(128), 0, lg, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (bf16*)m->act_a);
-                } else if (!latent_tile(m, sm, ag, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
+                    const int splits = row_splits(R, a.heads, 1);
+                    row_split(m, sm, ag, nullptr, 0, R, splits);
+                    row_combine(m, ag, R, splits);
+                } else if (!row_tile(m, sm, ag, n_runs, max_len)) attn_rows(m, sm, ag, L, R);
                 gemm_heads(m, m->act_a, a.heads * a.kv_rank, a.kv_rank, L.w_uv, a.heads, a.vdim, a.kv_rank, m->O, nv, a.vdim, R);
 #define LP_LG(T, N) launch(m, lp_latent_gate_kernel<T, N>, dim3(R), dim3(256), 0, lg, (const float*)m->O, (const float*)m->P, L.n_in, (T*)m->act_a)
                 if (m->f32) { if (a.vdim % 4) LP_LG(float, 1); else LP_LG(float, 4); }
                 else { if (a.vdim % 4) LP_LG(bf16, 1); else LP_LG(bf16, 4); }
 #undef LP_LG
             }
-#undef LP_LS_ANY
-#undef LP_LS
             project_out(m->act_a, nv, L.wo, L.norm1, moe_next);
         } else if (L.d.mixer == B200_MIX_STATE_SPACE) {
             const b200_state_space_desc& g = L.d.ssd;
@@ -3340,31 +3461,40 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             const int per = act_gated(e.act) ? 2 * e.expert_ff : e.expert_ff;                // rows of one expert's up matrix
             const bool own_act = act_gated(e.act) || e.weight_input != 0;                      // the hidden units need a kernel of their own
             const ExpertAct ea{e.act, e.weight_input, e.limit, e.shared_limit, e.slope};
-            const int rrows = e.experts + (e.shared_gate ? 1 : 0);                             // logits of a row: the experts', then the always-on gate's
+            const int outs = e.experts + e.identity;                                            // what the router chooses among
+            const int rrows = outs + (e.shared_gate ? 1 : 0);                                  // logits of a row: these, then the always-on gate's
+            // (an identity expert's output is what the feed-forward reads: the stream in f32 where that is it, else m->hn)
+            const float* hf = post ? m->x : nullptr;
             float* shw = e.shared_gate ? m->moe_shw : nullptr;
             sub = 1;
             bool routed = par || moe_next != nullptr;
-            if (p.in_conv > 0) {
+            if (p.in_conv > 0 || out_norm) {
                 StepRoute rt{};
-                if (ring_step && R <= LS_ROWS) {       // few rows: the block that norms a row also routes it
-                    rt.router = L.w_up; rt.bias = L.router_bias; rt.rows = rrows; rt.E = e.experts; rt.top = e.top; rt.mode = e.route; rt.scale = e.route_scale;
+                if (R <= LS_ROWS && (out_norm ? m->use_fuse && (size_t)W * es <= 40 * 1024 : ring_step)) {       // few rows: the block that norms a row also routes it
+                    rt.router = L.w_up; rt.bias = L.router_bias; rt.corr = L.router_corr; rt.rows = rrows; rt.E = outs; rt.top = e.top; rt.mode = e.route; rt.scale = e.route_scale;
                     rt.logits = m->P; rt.wts = m->moe_w; rt.sel = m->moe_sel; rt.selw = m->moe_selw; rt.shw = shw;
                     routed = true;
                 }
-                conv_in(L.ic[1], L.norm2, rt);
+                if (out_norm) settle(rt);
+                else conv_in(L.ic[1], L.norm2, rt);
             } else if (streams) boundary(L.hc_in[1], L.norm2, nullptr);
             else if (!post && !par) rmsnorm(m, m->x, nullptr, L.norm2, m->hn, nullptr, R);
             if (par) {
-                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P + L.ff_off, L.n_in, e.experts, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale, (float*)nullptr);
+                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P + L.ff_off, L.n_in, outs, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale, (float*)nullptr, L.router_corr);
             } else if (!routed) {
                 gemm(m, m->hn, W, L.w_up, rrows, W, m->P, rrows, R, 1.0f, EPI_STORE, nullptr, L.router_bias);
-                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P, rrows, e.experts, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale, shw);
+                launch(m, lp_moe_route_kernel, dim3((R + 3) / 4), dim3(128), 0, (const float*)m->P, rrows, outs, e.top, m->moe_w, m->moe_sel, m->moe_selw, R, e.route, e.route_scale, shw, L.router_corr);
             }
             const size_t hbytes = (size_t)R * W * es;
             const uint8_t* up_experts = (const uint8_t*)L.w_up + (size_t)L.up_router_rows * W * es;
             const bool direct = !post && !streams;     // x += : the experts' sum goes straight into the residual stream
             float* ydst = direct ? m->x : m->y;
             bool normed = false;
+            auto identity_add = [&](int add) {
+                if (!e.identity) return;
+                if (m->f32) launch(m, lp_moe_identity_kernel<float>, dim3(R), dim3(256), 0, (const float*)m->moe_w, e.experts, e.identity, (const float*)m->hn, hf, W, add, ydst);
+                else launch(m, lp_moe_identity_kernel<bf16>, dim3(R), dim3(256), 0, (const float*)m->moe_w, e.experts, e.identity, (const bf16*)m->hn, hf, W, add, ydst);
+            };
             if (moe_sel_ok) {
                 // few rows (decoding): kernels that walk each row's choices and read those experts' weights only
                 const int per_row = e.top * e.expert_ff + e.shared_ff;
@@ -3374,18 +3504,18 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                 if (sfew) pre_done = true;
                 if (m->f32) {
                     launch(m, lp_moe_up_sel_kernel<float>, ugrid, dim3(256), hbytes, (const float*)m->hn, (const float*)up_experts, (const int*)m->moe_sel, (const float*)m->moe_selw, (const float*)shw, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, (float*)m->act_a, ea);
-                    launch(m, lp_moe_down_sel_kernel<float>, dgrid, dim3(256), 0, (const float*)m->act_a, (const float*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, direct ? 1 : 0);
+                    launch(m, lp_moe_down_sel_kernel<float>, dgrid, dim3(256), 0, (const float*)m->act_a, (const float*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, direct ? 1 : 0, (const float*)m->moe_selw, (const float*)m->hn, hf, e.identity);
                 } else {
                     launch(m, lp_moe_up_sel_kernel<bf16>, ugrid, dim3(256), hbytes, (const bf16*)m->hn, (const bf16*)up_experts, (const int*)m->moe_sel, (const float*)m->moe_selw, (const float*)shw, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, (bf16*)m->act_a, ea);
-                    launch(m, lp_moe_down_sel_kernel<bf16>, dgrid, dim3(256), 0, (const bf16*)m->act_a, (const bf16*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, direct ? 1 : 0);
+                    launch(m, lp_moe_down_sel_kernel<bf16>, dgrid, dim3(256), 0, (const bf16*)m->act_a, (const bf16*)L.w_down, (const int*)m->moe_sel, e.experts, e.top, e.expert_ff, e.shared_ff, W, R, ydst, t, direct ? 1 : 0, (const float*)m->moe_selw, (const bf16*)m->hn, hf, e.identity);
                 }
             } else if (m->use_fuse && R > 2 * GV_ROWS) {
                 // many rows: the (token, choice) pairs in expert order, one product pair per expert over its block of rows (the row
                 // counts stay on the device), the always-on expert over all rows, then the weighted sum per token
                 const int pairs = R * e.top;
-                launch(m, lp_moe_sort_kernel, dim3(1), dim3(1024), (size_t)2 * e.experts * 4, (const int*)m->moe_sel, pairs, e.experts, m->moe_seg, m->moe_pos);
-                if (m->f32) launch(m, lp_moe_gather_kernel<float>, dim3(pairs), dim3(128), 0, (const float*)m->hn, (const int*)m->moe_pos, e.top, W, (float*)m->moe_xp);
-                else launch(m, lp_moe_gather_kernel<bf16>, dim3(pairs), dim3(128), 0, (const bf16*)m->hn, (const int*)m->moe_pos, e.top, W, (bf16*)m->moe_xp);
+                launch(m, lp_moe_sort_kernel, dim3(1), dim3(1024), (size_t)2 * outs * 4, (const int*)m->moe_sel, pairs, outs, m->moe_seg, m->moe_pos);
+                if (m->f32) launch(m, lp_moe_gather_kernel<float>, dim3(pairs), dim3(128), 0, (const float*)m->hn, (const int*)m->moe_pos, (const int*)m->moe_sel, e.experts, e.top, W, (float*)m->moe_xp);
+                else launch(m, lp_moe_gather_kernel<bf16>, dim3(pairs), dim3(128), 0, (const bf16*)m->hn, (const int*)m->moe_pos, (const int*)m->moe_sel, e.experts, e.top, W, (bf16*)m->moe_xp);
                 const uint8_t* down = (const uint8_t*)L.w_down;
                 uint8_t* act_sh = (uint8_t*)m->act_a + (size_t)pairs * e.expert_ff * es;     // the always-on expert's activations behind the others
                 if (own_act) {
@@ -3393,7 +3523,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                     gemm_grouped(m, m->moe_xp, W, up_experts, W, (size_t)per * W, e.experts, per, W, m->P, per, R, EPI_STORE, m->moe_seg);
                     const int V = e.expert_ff % 4 ? 1 : 4;
                     const unsigned nb = (unsigned)(((size_t)pairs * (e.expert_ff / V) + 255) / 256);
-#define LP_PA(T, V) launch(m, lp_moe_pair_act_kernel<T, V>, dim3(nb), dim3(256), 0, (const float*)m->P, per, (const int*)m->moe_pos, (const float*)m->moe_selw, e.expert_ff, (T*)m->act_a, pairs, ea)
+#define LP_PA(T, V) launch(m, lp_moe_pair_act_kernel<T, V>, dim3(nb), dim3(256), 0, (const float*)m->P, per, (const int*)m->moe_pos, (const int*)m->moe_sel, (const float*)m->moe_selw, e.experts, e.expert_ff, (T*)m->act_a, pairs, ea)
                     if (m->f32) { if (V == 4) LP_PA(float, 4); else LP_PA(float, 1); }
                     else { if (V == 4) LP_PA(bf16, 4); else LP_PA(bf16, 1); }
 #undef LP_PA
@@ -3415,23 +3545,38 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                     } else gemm(m, m->hn, W, up_sh, e.shared_ff, W, act_sh, e.shared_ff, R, 1.0f, act_epi);
                     gemm_ld(m, act_sh, e.shared_ff, down + (size_t)e.experts * e.expert_ff * es, L.k_down, W, e.shared_ff, ydst, W, R, direct ? EPI_ADD : EPI_STORE);
                 }
-                launch(m, lp_moe_combine_kernel, dim3(R), dim3(256), 0, (const float*)m->moe_yp, (const int*)m->moe_pos, own_act ? (const float*)nullptr : (const float*)m->moe_selw, e.top, W,
-                       (direct || e.shared_ff > 0) ? 1 : 0, ydst);
+                // (with kernels of their own for the units the experts' weights are in there already, an identity expert's is not)
+                const float* cw = own_act ? (const float*)nullptr : (const float*)m->moe_selw;
+                if (out_norm && e.shared_ff == 0 && !(cw == nullptr && e.identity)) {       // the sum, its norm and the residual in one pass
+                    pend_output(L.norm2);
+                    SubNorm sn = sub_pend;
+                    sn.xout = m->x;
+                    sub_pend.y = nullptr;
+                    normed = true;
+                    if (m->f32) launch(m, lp_sub_norm_moe_kernel<float>, dim3(R), dim3(256), 0, sn, (const float*)m->x, W, (float*)m->hn, (const float*)m->moe_yp, (const int*)m->moe_pos, (const int*)m->moe_sel, cw, e.top, e.experts);
+                    else launch(m, lp_sub_norm_moe_kernel<bf16>, dim3(R), dim3(256), 0, sn, (const float*)m->x, W, (bf16*)m->hn, (const float*)m->moe_yp, (const int*)m->moe_pos, (const int*)m->moe_sel, cw, e.top, e.experts);
+                } else {
+                    launch(m, lp_moe_combine_kernel, dim3(R), dim3(256), 0, (const float*)m->moe_yp, (const int*)m->moe_pos, (const int*)m->moe_sel, cw, e.top, e.experts, W,
+                           (direct || e.shared_ff > 0) ? 1 : 0, ydst);
+                    identity_add(1);
+                }
             } else {
                 // the plain form: every expert's up projection for every row, activations times their expert's weight (0 for experts
                 // that were not chosen), one product with the down matrices side by side
                 const int n_exp = L.n_up - L.up_router_rows;
                 gemm(m, m->hn, W, up_experts, n_exp, W, m->P, n_exp, R, 1.0f, EPI_STORE);
                 const unsigned nb = (unsigned)(((size_t)R * L.k_down + 255) / 256);
-                if (m->f32) launch(m, lp_moe_act_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, (const float*)shw, e.experts, e.expert_ff, e.shared_ff, (float*)m->act_a, R, ea);
-                else launch(m, lp_moe_act_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, (const float*)shw, e.experts, e.expert_ff, e.shared_ff, (bf16*)m->act_a, R, ea);
-                gemm(m, m->act_a, L.k_down, L.w_down, W, L.k_down, ydst, W, R, 1.0f, direct ? EPI_ADD : EPI_STORE);
+                if (m->f32) launch(m, lp_moe_act_kernel<float>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, outs, (const float*)shw, e.experts, e.expert_ff, e.shared_ff, (float*)m->act_a, R, ea);
+                else launch(m, lp_moe_act_kernel<bf16>, dim3(nb), dim3(256), 0, (const float*)m->P, n_exp, 0, (const float*)m->moe_w, outs, (const float*)shw, e.experts, e.expert_ff, e.shared_ff, (bf16*)m->act_a, R, ea);
+                identity_add(direct ? 1 : 0);
+                gemm(m, m->act_a, L.k_down, L.w_down, W, L.k_down, ydst, W, R, 1.0f, direct || e.identity ? EPI_ADD : EPI_STORE);
             }
             if (normed || direct) {
             } else if (streams) {
                 pend.y = m->y; pend.mix = L.hc_mix[1]; pend.out = L.hc_out[1];
-            } else cast_x(m->y, L.norm2);
-        } else if (L.d.ff > 0 && (L.d.ff_kind == B200_FF_GATED_GELU || L.d.ff_kind == B200_FF_CLAMPED_GLU)) {
+            } else if (out_norm) pend_output(L.norm2);
+            else cast_x(m->y, L.norm2);
+        } else if (L.d.ff > 0 && (L.d.ff_kind == B200_FF_GATED_GELU || L.d.ff_kind == B200_FF_CLAMPED_GLU || L.d.ff_kind == B200_FF_GATED_RELU)) {
             // [gate | up] in one product (with parallel_ff: columns ff_off .. of the layer's input projection), the gated units, W_down
             sub = 1;
             const float* ffP = m->P;
@@ -3439,7 +3584,18 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             if (par) { ffP = m->P + L.ff_off; ff_ld = L.n_in; }
             else project_in(nullptr, L.norm2, L.w_up, L.n_up, m->P, L.n_up, EPI_STORE);
             const unsigned nb = (unsigned)(((size_t)R * L.d.ff + 255) / 256);
-            if (L.d.ff_kind == B200_FF_CLAMPED_GLU) {
+            if (L.d.ff_kind == B200_FF_GATED_RELU) {      // (an always-on expert's units without a gate)
+                const ExpertAct ea{B200_ACT_RELU_GLU, 0, 0.0f, 0.0f, 0.0f};
+                const bool v4 = L.d.ff % 4 == 0 && ff_ld % 4 == 0 && ((uintptr_t)ffP & 15) == 0;
+                const unsigned nb4 = (unsigned)(((size_t)R * (L.d.ff / 4) + 255) / 256);
+                if (m->f32) {
+                    if (v4) launch(m, lp_moe_shared_act_kernel<float, 4>, dim3(nb4), dim3(256), 0, ffP, ff_ld, (const float*)nullptr, L.d.ff, (float*)m->act_a, R, ea);
+                    else launch(m, lp_moe_shared_act_kernel<float, 1>, dim3(nb), dim3(256), 0, ffP, ff_ld, (const float*)nullptr, L.d.ff, (float*)m->act_a, R, ea);
+                } else {
+                    if (v4) launch(m, lp_moe_shared_act_kernel<bf16, 4>, dim3(nb4), dim3(256), 0, ffP, ff_ld, (const float*)nullptr, L.d.ff, (bf16*)m->act_a, R, ea);
+                    else launch(m, lp_moe_shared_act_kernel<bf16, 1>, dim3(nb), dim3(256), 0, ffP, ff_ld, (const float*)nullptr, L.d.ff, (bf16*)m->act_a, R, ea);
+                }
+            } else if (L.d.ff_kind == B200_FF_CLAMPED_GLU) {
                 const bool v4 = L.d.ff % 4 == 0 && ff_ld % 4 == 0 && ((uintptr_t)ffP & 15) == 0;
                 const unsigned nb4 = (unsigned)(((size_t)R * (L.d.ff / 4) + 255) / 256);
                 if (m->f32) {
@@ -3465,17 +3621,19 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             sub = 1;
             project_in(nullptr, L.norm2, L.w_up, L.d.ff, m->act_a, L.d.ff, L.d.ff_kind == B200_FF_XIELU ? EPI_XIELU : EPI_RELU2);
             project_out(m->act_a, L.d.ff, L.w_down, L.norm2, nullptr);
-        } else if (post && L.norm2) {
+        } else if (post && !out_norm && L.norm2) {
             cast_x(nullptr, L.norm2);
         }
         if (streams && taps_len > 0) boundary(nullptr, nullptr, m->x);   // the taps are the sum of the copies
+        if (taps_len > 0 && out_norm) settle(StepRoute{});
         if (taps_len > 0) cudaMemcpyAsync(m->taps + run * (size_t)taps_len * W, m->x, (size_t)taps_len * W * 4, cudaMemcpyDeviceToDevice, m->stream);
     }
+    if (out_norm) settle(StepRoute{});
     if (streams) boundary(nullptr, nullptr, m->x);   // the head reads the sum of the copies
     if (p.in_conv > 1 && !ring_step)
         launch(m, lp_ring_commit_kernel, dim3(m->n_convs, n_runs, p.in_conv - 1), dim3(256), 0, sm, (const size_t*)m->ring_offs, (const float*)m->conv_pend, p.in_conv, W);
     if (head) {
-        norm_gemm(m, m->x, nullptr, sm.want, (const float*)find(m, "final.norm")->d, m->hw, find(m, "head")->d, p.vocab, m->logits, p.vocab, n_want,
+        norm_gemm(m, m->x, nullptr, sm.want, (const float*)find(m, "final.norm")->d, m->hw, find(m, p.tied_head ? "embed" : "head")->d, p.vocab, m->logits, p.vocab, n_want,
                   p.logit_scale, EPI_STORE);
         if (head == 2) launch(m, lp_argmax_kernel, dim3(n_want), dim3(1024), 0, (const float*)m->logits, p.vocab, m->pick);
     }

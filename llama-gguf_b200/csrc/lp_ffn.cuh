@@ -64,10 +64,10 @@ __global__ void lp_relu2_kernel(const float* __restrict__ P, int ldp, OutT* __re
 
 // Router: one warp per row of the f32 logits P[r][0 .. E) (route_row, lp_rows_tail.cuh)
 __global__ void lp_moe_route_kernel(const float* __restrict__ P, int ldp, int E, int top, float* __restrict__ wts, int* __restrict__ sel,
-                                    float* __restrict__ selw, int R, int mode, float scale, float* __restrict__ shw) {
+                                    float* __restrict__ selw, int R, int mode, float scale, float* __restrict__ shw, const float* __restrict__ corr) {
     const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (r >= R) return;
-    route_row(P + (size_t)r * ldp, E, top, wts + (size_t)r * E, sel + (size_t)r * top, selw + (size_t)r * top, lane, mode, scale);
+    route_row(P + (size_t)r * ldp, E, top, wts + (size_t)r * E, sel + (size_t)r * top, selw + (size_t)r * top, lane, mode, scale, corr);
     if (shw && lane == 0) shw[r] = sigmoid_f(P[(size_t)r * ldp + E]);      // the always-on expert's gate: the logit behind the experts'
 }
 
@@ -78,13 +78,13 @@ __device__ __forceinline__ float expert_act(float z, int act) {
     return z * z;
 }
 
-// What an expert's hidden units are made of.  The gated kinds (B200_ACT_SILU_GLU, B200_ACT_CLAMPED_GLU) have two pre-activations per unit,
+// What an expert's hidden units are made of.  The gated kinds (B200_ACT_SILU_GLU, B200_ACT_CLAMPED_GLU, B200_ACT_RELU_GLU) have two pre-activations per unit,
 // their up matrix is [gate | up] rows.
 struct ExpertAct {
     int kind, win;               // B200_ACT_*; 1: the expert's weight goes onto its input
     float limit, shared_limit, slope;
 };
-__host__ __device__ inline bool act_gated(int kind) { return kind == B200_ACT_SILU_GLU || kind == B200_ACT_CLAMPED_GLU; }
+__host__ __device__ inline bool act_gated(int kind) { return kind == B200_ACT_SILU_GLU || kind == B200_ACT_CLAMPED_GLU || kind == B200_ACT_RELU_GLU; }
 __device__ __forceinline__ int expert_rows(int eff, int kind) { return act_gated(kind) ? 2 * eff : eff; }
 // min(z, limit) sigmoid(slope .) (clamp(zu, +-limit) + 1)
 __device__ __forceinline__ float clamped_glu_f(float z, float zu, float limit, float slope) {
@@ -95,7 +95,8 @@ __device__ __forceinline__ float clamped_glu_f(float z, float zu, float limit, f
 // where W (w h) = w (W h) puts it on the pre-activations
 __device__ __forceinline__ float expert_unit(float z, float zu, float w, const ExpertAct& a, float limit) {
     if (a.win) { z *= w; zu *= w; }
-    const float v = a.kind == B200_ACT_CLAMPED_GLU ? clamped_glu_f(z, zu, limit, a.slope) : a.kind == B200_ACT_SILU_GLU ? z * sigmoid_f(z) * zu : expert_act(z, a.kind);
+    const float v = a.kind == B200_ACT_CLAMPED_GLU ? clamped_glu_f(z, zu, limit, a.slope) : a.kind == B200_ACT_SILU_GLU ? z * sigmoid_f(z) * zu
+                  : a.kind == B200_ACT_RELU_GLU ? fmaxf(z, 0.0f) * zu : expert_act(z, a.kind);
     return a.win ? v : v * w;
 }
 // the always-on expert: the same form, its weight (1 without a gate) always on the output
@@ -105,10 +106,10 @@ __device__ __forceinline__ float shared_unit(float z, float zu, float w, ExpertA
 }
 
 // out[r][c] = hidden unit c of the row: expert e = c / eff with its weight (0 = not chosen: the unit is 0), the always-on expert's
-// units behind them with weight shw[r] (null: 1).  P holds every expert's pre-activations side by side (expert_rows per expert).
+// units behind them with weight shw[r] (null: 1).  wts: [R][ldw].  P holds every expert's pre-activations side by side (expert_rows per expert).
 template <typename OutT>
-__global__ void lp_moe_act_kernel(const float* __restrict__ P, int ldp, int off, const float* __restrict__ wts, const float* __restrict__ shw, int E, int eff,
-                                  int sff, OutT* __restrict__ out, int R, ExpertAct a) {
+__global__ void lp_moe_act_kernel(const float* __restrict__ P, int ldp, int off, const float* __restrict__ wts, int ldw, const float* __restrict__ shw, int E,
+                                  int eff, int sff, OutT* __restrict__ out, int R, ExpertAct a) {
     const int total = E * eff + sff;
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (size_t)R * total) return;
@@ -119,7 +120,7 @@ __global__ void lp_moe_act_kernel(const float* __restrict__ P, int ldp, int off,
     float v = 0.0f;
     if (c < E * eff) {
         const int e = c / eff, n = c - e * eff;
-        const float w = wts[(size_t)r * E + e];
+        const float w = wts[(size_t)r * ldw + e];
         if (w != 0.0f) v = expert_unit(p[e * per + n], glu ? p[e * per + eff + n] : 0.0f, w, a, a.limit);
     } else {
         const int n = c - E * eff;
@@ -130,12 +131,14 @@ __global__ void lp_moe_act_kernel(const float* __restrict__ P, int ldp, int off,
 
 // The same for (token, choice) pairs in expert order: pair i = (row i / top, choice i % top) sits at row pos[i] of P (its expert's
 // pre-activations, expert_rows wide) and of out (eff wide); its weight is selw[i].  V units per thread (4: eff a multiple of 4).
+// Pairs of an identity expert have neither.
 template <typename OutT, int V>
-__global__ void lp_moe_pair_act_kernel(const float* __restrict__ P, int ldp, const int* __restrict__ pos, const float* __restrict__ selw, int eff,
-                                       OutT* __restrict__ out, int n_pairs, ExpertAct a) {
+__global__ void lp_moe_pair_act_kernel(const float* __restrict__ P, int ldp, const int* __restrict__ pos, const int* __restrict__ sel, const float* __restrict__ selw,
+                                       int E, int eff, OutT* __restrict__ out, int n_pairs, ExpertAct a) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (size_t)n_pairs * (eff / V)) return;
     const int pr = (int)(i / (eff / V)), n = (int)(i - (size_t)pr * (eff / V)) * V;
+    if (sel[pr] >= E) return;
     const float* p = P + (size_t)pos[pr] * ldp;
     const FloatV<V> z = load_v<V>(p + n), zu = act_gated(a.kind) ? load_v<V>(p + eff + n) : z;
     FloatV<V> o;
@@ -162,7 +165,7 @@ __global__ void lp_moe_shared_act_kernel(const float* __restrict__ P, int ldp, c
 // columns (a gated expert: [gate | up], expert_rows each); segment k < top of a row's activations belongs to expert sel[r][k],
 // segment `top` to the always-on expert.
 //   act[r][k eff + n] = unit(up_e[n] . h_r, selw[r][k])        act[r][top eff + n] = unit(up_shared[n] . h_r, shw[r] or 1)
-// One warp per (row, segment, n); h rows are staged in shared memory once per block.
+// A choice e >= E is an identity expert: its segment is not written.  One warp per (row, segment, n); h rows are staged in shared memory once per block.
 template <typename T>
 __global__ void __launch_bounds__(256) lp_moe_up_sel_kernel(const T* __restrict__ H, const T* __restrict__ up_exp, const int* __restrict__ sel,
                                                             const float* __restrict__ selw, const float* __restrict__ shw, int E, int top, int eff, int sff,
@@ -182,6 +185,7 @@ __global__ void __launch_bounds__(256) lp_moe_up_sel_kernel(const T* __restrict_
         const int k = c < top * eff ? c / eff : top;
         const int n = c - k * eff;
         const int e = k < top ? sel[(size_t)r * top + k] : E;
+        if (k < top && e >= E) continue;
         const T* wr = up_exp + ((size_t)e * per + n) * width;
         const T* wu = wr + (size_t)(k < top ? eff : sff) * width;          // (gated experts: the up row of the same unit)
         const T* hr = hs + (size_t)r * width;
@@ -207,11 +211,13 @@ __global__ void __launch_bounds__(256) lp_moe_up_sel_kernel(const T* __restrict_
 
 // y[r][c] = sum over the row's segments of down_e[c] . act segment; down_cat is [width][E eff + sff].  MD_SPLIT warps share one (row, c):
 // each takes every MD_SPLIT-th 16-byte group of every segment (more loads in flight per output: a decode step has only `width` of
-// them), the partial sums meet in shared memory and are added in warp order.  accum = 1: y += (y is the residual stream).
+// them), the partial sums meet in shared memory and are added in warp order.  accum = 1: y += (y is the residual stream).  Identity experts
+// (choices e >= E) have no segment: they add their weight times what the feed-forward reads, hf in f32 or, when that is null, h.
 constexpr int MD_SPLIT = 4, MD_BATCH = 6;
 template <typename T>
 __global__ void __launch_bounds__(256) lp_moe_down_sel_kernel(const T* __restrict__ act, const T* __restrict__ down_cat, const int* __restrict__ sel,
-                                                              int E, int top, int eff, int sff, int width, int R, float* __restrict__ y, RowsTail tail, int accum) {
+                                                              int E, int top, int eff, int sff, int width, int R, float* __restrict__ y, RowsTail tail, int accum,
+                                                              const float* __restrict__ selw, const T* __restrict__ h, const float* hf, int identity) {
     constexpr int VN = Vec8<T>::N, GROUPS = 8 / MD_SPLIT;
     __shared__ float part[8];
     __shared__ int sel_s[256];
@@ -236,9 +242,9 @@ __global__ void __launch_bounds__(256) lp_moe_down_sel_kernel(const T* __restric
                 for (int u = 0; u < MD_BATCH; u++) {
                     const int i = i0 + u * MD_SPLIT * 32 * VN;
                     wv[u] = xv[u] = make_uint4(0u, 0u, 0u, 0u);
-                    if (i < per_row) {
-                        const int k = min(i / eff, top);
-                        const int e = k < top ? (sel_in ? sel_s[r * top + k] : sel[(size_t)r * top + k]) : E;
+                    const int k = i < per_row ? min(i / eff, top) : 0;
+                    const int e = i >= per_row ? 0 : k < top ? (sel_in ? sel_s[r * top + k] : sel[(size_t)r * top + k]) : E;
+                    if (i < per_row && (k == top || e < E)) {
                         wv[u] = *reinterpret_cast<const uint4*>(dr + (size_t)e * eff + (i - k * eff));
                         xv[u] = *reinterpret_cast<const uint4*>(ar + i);
                     }
@@ -260,6 +266,11 @@ __global__ void __launch_bounds__(256) lp_moe_down_sel_kernel(const T* __restric
             float t = part[grp * MD_SPLIT];
 #pragma unroll
             for (int i = 1; i < MD_SPLIT; i++) t += part[grp * MD_SPLIT + i];
+            if (identity) {
+                const int r = o / width;
+                for (int k = 0; k < top; k++)
+                    if (sel[(size_t)r * top + k] >= E) t = fmaf(selw[(size_t)r * top + k], hf ? hf[o] : to_f(h[o]), t);
+            }
             y[o] = accum ? y[o] + t : t;
         }
         __syncthreads();
@@ -291,10 +302,11 @@ __global__ void __launch_bounds__(1024) lp_moe_sort_kernel(const int* __restrict
     for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) pos[i] = atomicAdd(&cur[sel[i]], 1);
 }
 
-// Xp[pos[i]] = H[i / top]: one block per pair
+// Xp[pos[i]] = H[i / top]: one block per pair (pairs of an identity expert, sel[i] >= E, need no row)
 template <typename T>
-__global__ void lp_moe_gather_kernel(const T* __restrict__ H, const int* __restrict__ pos, int top, int width, T* __restrict__ Xp) {
+__global__ void lp_moe_gather_kernel(const T* __restrict__ H, const int* __restrict__ pos, const int* __restrict__ sel, int E, int top, int width, T* __restrict__ Xp) {
     const int i = blockIdx.x;
+    if (sel[i] >= E) return;
     const T* src = H + (size_t)(i / top) * width;
     T* dst = Xp + (size_t)pos[i] * width;
     constexpr int VN = Vec8<T>::N;
@@ -305,14 +317,60 @@ __global__ void lp_moe_gather_kernel(const T* __restrict__ H, const int* __restr
     }
 }
 
-// y[r] (+)= sum_k selw[r][k] Yp[pos[r top + k]], choices in the order they were taken; add = 1 when y already holds something to add
-// to (the always-on expert's output, or the residual stream); selw = null: plain sum (the weights went into the experts' inputs)
-__global__ void lp_moe_combine_kernel(const float* __restrict__ Yp, const int* __restrict__ pos, const float* __restrict__ selw, int top, int width,
-                                      int add, float* __restrict__ y) {
+// Channels c .. c + V - 1 of sum_k selw[r][k] out_k, choices in the order they were taken: out_k = Yp[pos[r top + k]], or the row hr itself
+// when choice k is an identity expert (sel >= E); selw = null: plain sum (the weights went into the experts' inputs)
+template <int V>
+__device__ __forceinline__ FloatV<V> moe_sum(const float* __restrict__ Yp, const int* __restrict__ pos, const int* __restrict__ sel, const float* __restrict__ selw, int top,
+                                             int E, int width, int r, int c, const float* hr) {
+    FloatV<V> sum;
+#pragma unroll
+    for (int e = 0; e < V; e++) sum.v[e] = 0.0f;
+    for (int k = 0; k < top; k++) {
+        const size_t at = (size_t)r * top + k;
+        const FloatV<V> v = load_v<V>(sel[at] >= E ? hr + c : Yp + (size_t)pos[at] * width + c);
+        const float w = selw ? selw[at] : 1.0f;
+#pragma unroll
+        for (int e = 0; e < V; e++) sum.v[e] = fmaf(w, v.v[e], sum.v[e]);
+    }
+    return sum;
+}
+// x <- alpha x + norm(that sum): the end of a mixture in the layer form with the norm on a sublayer's output (lp_sublayer_norm.cuh).  One block per row.
+template <typename T>
+__global__ void __launch_bounds__(256) lp_sub_norm_moe_kernel(SubNorm sn, const float* x, int width, T* __restrict__ out, const float* __restrict__ Yp,
+                                                              const int* __restrict__ pos, const int* __restrict__ sel, const float* __restrict__ selw, int top, int E) {
+    const int r = blockIdx.x;
+    const float* xr = x + (size_t)r * width;
+    float* xo = sn.xout + (size_t)r * width;
+    T* o = out + (size_t)r * width;
+    if (width & 3) {
+        sub_norm_row_v<T, 256, 1>(sn, xr, xo, width, 0, o, (T*)nullptr, [&](int c) { return moe_sum<1>(Yp, pos, sel, selw, top, E, width, r, c, xr); });
+    } else {
+        sub_norm_row_v<T, 256, 4>(sn, xr, xo, width, 0, o, (T*)nullptr, [&](int c) { return moe_sum<4>(Yp, pos, sel, selw, top, E, width, r, c, xr); });
+    }
+}
+// y[r] (+)= sum_k selw[r][k] Yp[pos[r top + k]], selw = null: plain sum; add = 1 when y already holds something to add to (the always-on expert's output, or the residual stream).
+// Identity experts are left out (lp_moe_identity_kernel adds them).
+__global__ void lp_moe_combine_kernel(const float* __restrict__ Yp, const int* __restrict__ pos, const int* __restrict__ sel, const float* __restrict__ selw, int top, int E,
+                                      int width, int add, float* __restrict__ y) {
     const int r = blockIdx.x;
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float acc = add ? y[(size_t)r * width + c] : 0.0f, sum = 0.0f;
-        for (int k = 0; k < top; k++) sum = fmaf(selw ? selw[(size_t)r * top + k] : 1.0f, Yp[(size_t)pos[(size_t)r * top + k] * width + c], sum);
+        for (int k = 0; k < top; k++) {
+            const size_t at = (size_t)r * top + k;
+            if (sel[at] < E) sum = fmaf(selw ? selw[at] : 1.0f, Yp[(size_t)pos[at] * width + c], sum);
+        }
         y[(size_t)r * width + c] = acc + sum;
+    }
+}
+// y[r] (+)= (sum of the row's weights for identity experts, wts[r][E .. E + n)) * what the feed-forward reads: hf in f32 or, when null, h
+template <typename T>
+__global__ void lp_moe_identity_kernel(const float* __restrict__ wts, int E, int n, const T* __restrict__ h, const float* hf, int width, int add, float* __restrict__ y) {
+    const int r = blockIdx.x;
+    float w = 0.0f;
+    for (int e = 0; e < n; e++) w += wts[(size_t)r * (E + n) + E + e];
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const size_t o = (size_t)r * width + c;
+        const float v = w == 0.0f ? 0.0f : w * (hf ? hf[o] : to_f(h[o]));
+        y[o] = add ? y[o] + v : v;
     }
 }

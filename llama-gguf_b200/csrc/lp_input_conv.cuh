@@ -131,25 +131,17 @@ __device__ __forceinline__ float block_sum_sq(const float* xr, int width, float*
 struct StepRoute {
     const void* router = nullptr;   // null: no routing
     const float* bias = nullptr;    // [rows]
+    const float* corr = nullptr;    // [E] added to the scores that choose
     int rows = 0, E = 0, top = 0, mode = 0;
     float scale = 0.0f;
     float *logits = nullptr, *wts = nullptr, *selw = nullptr, *shw = nullptr;
     int* sel = nullptr;
 };
 
-// One token per run (decoding), one block per row: norm, convolution, the row in the compute type; then, before a mixture of experts,
-// the router's logits on that row (a warp per logit) and the choice.
+// The router's logits on a row in shared memory (a warp per logit) and the choice, by the whole block
 template <typename T>
-__global__ void __launch_bounds__(512) lp_norm_conv_step_kernel(StepMeta sm, InConv ic, const float* __restrict__ x, const float* __restrict__ g, int width,
-                                                                float eps, T* __restrict__ out, StepRoute rt) {
-    extern __shared__ __align__(16) uint8_t nc_smem[];
-    T* hs = reinterpret_cast<T*>(nc_smem);     // [width] (with routing only)
-    const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-    if (rt.router)
-        for (int e = warp; e < rt.rows; e += nw) prefetch_row(reinterpret_cast<const T*>(rt.router) + (size_t)e * width, width, lane);
-    norm_conv_row<T, 512>(ic, sm, r, x + (size_t)r * width, g, width, eps, true, out + (size_t)r * width, rt.router ? hs : (T*)nullptr);
-    if (!rt.router) return;
-    __syncthreads();
+__device__ __forceinline__ void step_route(const StepRoute& rt, const T* hs, int r, int width) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     constexpr int VN = Vec8<T>::N;
     const T* rw = reinterpret_cast<const T*>(rt.router);
     float* z = rt.logits + (size_t)r * rt.rows;
@@ -173,9 +165,25 @@ __global__ void __launch_bounds__(512) lp_norm_conv_step_kernel(StepMeta sm, InC
     }
     __syncthreads();
     if (warp == 0) {
-        route_row(z, rt.E, rt.top, rt.wts + (size_t)r * rt.E, rt.sel + (size_t)r * rt.top, rt.selw + (size_t)r * rt.top, lane, rt.mode, rt.scale);
+        route_row(z, rt.E, rt.top, rt.wts + (size_t)r * rt.E, rt.sel + (size_t)r * rt.top, rt.selw + (size_t)r * rt.top, lane, rt.mode, rt.scale, rt.corr);
         if (rt.shw && lane == 0) rt.shw[r] = sigmoid_f(z[rt.E]);
     }
+}
+
+// One token per run (decoding), one block per row: norm, convolution, the row in the compute type; then, before a mixture of experts,
+// the router's logits on that row (a warp per logit) and the choice.
+template <typename T>
+__global__ void __launch_bounds__(512) lp_norm_conv_step_kernel(StepMeta sm, InConv ic, const float* __restrict__ x, const float* __restrict__ g, int width,
+                                                                float eps, T* __restrict__ out, StepRoute rt) {
+    extern __shared__ __align__(16) uint8_t nc_smem[];
+    T* hs = reinterpret_cast<T*>(nc_smem);     // [width] (with routing only)
+    const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+    if (rt.router)
+        for (int e = warp; e < rt.rows; e += nw) prefetch_row(reinterpret_cast<const T*>(rt.router) + (size_t)e * width, width, lane);
+    norm_conv_row<T, 512>(ic, sm, r, x + (size_t)r * width, g, width, eps, true, out + (size_t)r * width, rt.router ? hs : (T*)nullptr);
+    if (!rt.router) return;
+    __syncthreads();
+    step_route<T>(rt, hs, r, width);
 }
 
 // Runs of any length: a block of 8 warps takes NC_ROWS rows; the warps first sum the squares of those rows and of the taps - 1 rows before

@@ -3,7 +3,7 @@
 // of layerprog.cu read it as ONE K/V head whose keys are the whole row and whose values are the row's first kv_rank entries
 // (AttnGeom.v_in_k).  For that, head n's query is carried into the latent: qbuf[r][n] = [W_uk[n]^T q_plain | rotated q part], and the
 // summed latent comes back through W_uv[n] afterwards (two products batched over the heads).  Included by layerprog.cu inside its
-// anonymous namespace, behind lp_input_conv.cuh (block_sum_sq).  Norms, angles and the rotation are f32 (the angle, its sine and cosine in double).
+// anonymous namespace, behind lp_input_conv.cuh (block_sum_sq) and lp_row_attn.cuh (the attention itself).  Norms, angles and the rotation are f32 (the angle, its sine and cosine in double).
 #pragma once
 
 struct LatentGeom {
@@ -123,8 +123,7 @@ __global__ void lp_latent_gate_kernel(LatentGeom g, const float* __restrict__ V,
 
 // ------------------------------------------------------------------------------------------------ few rows, one token per run (decoding)
 // Three kernels take a layer from its input projection to the operand of W_o: the query into the latent (with the rotations and the cache
-// row), the attention with the keys cut into splits and all heads of a row on the same staged rows, and the merge of the splits with W_uv
-// and the gate.  Everything between the two products is f32.
+// row), the attention with the keys cut into splits (lp_row_split_kernel), and the merge of the splits with W_uv and the gate.  Everything between the two products is f32.
 
 // Lanes that share one output of a per-head product of length K: the smallest power of two with VN values each, at most a warp
 __host__ __device__ inline int latent_lanes(int K, int VN) {
@@ -225,96 +224,6 @@ __global__ void __launch_bounds__(256) lp_latent_absorb_kernel(StepMeta sm, Late
     }
 }
 
-// Attention of one row over its cached rows, the keys cut into gridDim.x splits of whole 32-key tiles; a block stages its tiles in shared
-// memory (two in flight, 16-byte cp.async) and its LS_HEADS warps each take one head: a key per lane for the scores, online softmax, the
-// latent channels dealt over the lanes for the weighted sum.  part_o [R][H][splits][kv_rank] receives the unnormalised sums, part_ml
-// the running maximum and sum (an empty split: -inf, 0).
-constexpr int LS_HEADS = 8, LS_KEYS = 32, LS_ROWS = 64;   // (LS_ROWS: the most rows these kernels take)
-__host__ __device__ inline size_t latent_split_smem(int D) { return (size_t)(LS_HEADS * D + 2 * LS_KEYS * (D + 4)) * 4; }
-template <int VCH>
-__global__ void __launch_bounds__(32 * LS_HEADS) lp_latent_split_kernel(StepMeta sm, AttnGeom a, const float* __restrict__ qbuf, float* __restrict__ part_o,
-                                                                        float* __restrict__ part_ml) {
-    extern __shared__ __align__(16) float ls_sm[];
-    const int D = a.dim, pitch = D + 4;
-    float* qs = ls_sm;                         // [LS_HEADS][D]
-    float* ks = ls_sm + LS_HEADS * D;          // [2][LS_KEYS][pitch]
-    const int split = blockIdx.x, splits = gridDim.x, r = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int h = blockIdx.z * LS_HEADS + warp;
-    const int i = sm.row_pos[r], lo = attn_lo(a, i);
-    const float* rows = reinterpret_cast<const float*>(sm.run_kv[sm.row_run[r]] + a.kv_off);
-    const int tiles = (i + 1 - lo + LS_KEYS - 1) / LS_KEYS, each = (tiles + splits - 1) / splits;
-    const int t_beg = min(tiles, split * each), t_end = min(tiles, t_beg + each);
-    const int vec = D / 4;
-    auto stage = [&](int t, int buf) {
-        const int j0 = lo + t * LS_KEYS;
-        for (int u = threadIdx.x; u < LS_KEYS * vec; u += 32 * LS_HEADS) {
-            const int key = u / vec, c = (u - key * vec) * 4, j = j0 + key;
-            cp_async16(smem_u32(ks + ((size_t)buf * LS_KEYS + key) * pitch + c), rows + (size_t)min(j, i) * D + c, j <= i ? 16u : 0u);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    if (t_beg < t_end) {
-        stage(t_beg, 0);
-        if (h < a.H)
-            for (int d = lane * 4; d < D; d += 128)
-                *reinterpret_cast<float4*>(qs + warp * D + d) = *reinterpret_cast<const float4*>(qbuf + ((size_t)r * a.H + h) * D + d);
-    }
-    float m = -INFINITY, l = 0.0f, acc[VCH];
-#pragma unroll
-    for (int c = 0; c < VCH; c++) acc[c] = 0.0f;
-    for (int t = t_beg; t < t_end; t++) {
-        const int buf = (t - t_beg) & 1;
-        if (t + 1 < t_end) {
-            stage(t + 1, buf ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();
-        if (h < a.H) {
-            const float* kt = ks + (size_t)buf * LS_KEYS * pitch;
-            const int j = lo + t * LS_KEYS + lane;
-            const float* kr = kt + (size_t)lane * pitch;
-            const float* q = qs + warp * D;
-            float s0 = 0.0f, s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
-#pragma unroll 8
-            for (int d = 0; d < D; d += 4) {
-                const float4 kv = *reinterpret_cast<const float4*>(kr + d), qv = *reinterpret_cast<const float4*>(q + d);
-                s0 = fmaf(qv.x, kv.x, s0);
-                s1 = fmaf(qv.y, kv.y, s1);
-                s2 = fmaf(qv.z, kv.z, s2);
-                s3 = fmaf(qv.w, kv.w, s3);
-            }
-            const float s = j <= i ? ((s0 + s1) + (s2 + s3)) * a.scale : -INFINITY;
-            const float mn = fmaxf(m, wmax(s));       // (a tile of the split holds a visible key: mn is finite)
-            const float p = expf(s - mn), corr = expf(m - mn);
-            l = l * corr + wsum(p);
-            m = mn;
-#pragma unroll
-            for (int c = 0; c < VCH; c++) acc[c] *= corr;
-#pragma unroll 8
-            for (int k = 0; k < LS_KEYS; k++) {
-                const float pk = __shfl_sync(0xffffffffu, p, k);
-#pragma unroll
-                for (int c = 0; c < VCH; c++) {
-                    const int chn = c * 32 + lane;
-                    if (chn < a.vdim) acc[c] = fmaf(pk, kt[(size_t)k * pitch + chn], acc[c]);
-                }
-            }
-        }
-        __syncthreads();
-    }
-    if (h >= a.H) return;
-    const size_t at = ((size_t)r * a.H + h) * splits + split;
-    if (lane == 0) {
-        part_ml[2 * at] = m;
-        part_ml[2 * at + 1] = l;
-    }
-    if (t_beg < t_end) {
-#pragma unroll
-        for (int c = 0; c < VCH; c++)
-            if (c * 32 + lane < a.vdim) part_o[at * a.vdim + c * 32 + lane] = acc[c];
-    }
-}
-
 // The splits' parts of a head's rows summed into the latent (shared memory, f32), then a chunk of the head's value columns: W_uv[n] times
 // the latent, times the gate, in the compute type: out[r][n vdim + c].
 template <typename T>
@@ -377,191 +286,6 @@ __global__ void __launch_bounds__(256) lp_latent_merge_kernel(LatentGeom g, cons
                     const int r = rb + i, o = n * g.vdim + c;
                     out[(size_t)r * g.H * g.vdim + o] = from_f<T>(acc[i] * latent_gate(g, P + (size_t)r * ldp, o));
                 }
-        }
-    }
-}
-
-// The merge alone: the latent of every (row, head) in the compute type -> out [R][H][kv_rank], the operand of the products with W_uv
-template <typename T>
-__global__ void __launch_bounds__(128) lp_latent_combine_kernel(LatentGeom g, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
-                                                                T* __restrict__ out) {
-    const size_t at = ((size_t)blockIdx.x * g.H + blockIdx.y) * splits;
-    float M = -INFINITY, L = 0.0f;
-    for (int s = 0; s < splits; s++) M = fmaxf(M, part_ml[2 * (at + s)]);
-    for (int s = 0; s < splits; s++) L = fmaf(part_ml[2 * (at + s) + 1], expf(part_ml[2 * (at + s)] - M), L);
-    for (int c = threadIdx.x; c < g.kv_rank; c += 128) {
-        float acc = 0.0f;
-        for (int s = 0; s < splits; s++) {
-            const float w = expf(part_ml[2 * (at + s)] - M);
-            if (w > 0.0f) acc = fmaf(w, part_o[(at + s) * g.kv_rank + c], acc);     // (an empty split has written nothing)
-        }
-        out[((size_t)blockIdx.x * g.H + blockIdx.y) * g.kv_rank + c] = from_f<T>(acc / L);
-    }
-}
-
-// ------------------------------------------------------------------------------------------------ prompt rows (bf16)
-// All heads of a token meet the same cached rows, so the (token, head) pairs of a run are ONE list of query rows, [tokens * H][D] as qbuf
-// holds them: a block of 8 warps takes LT_ROWS neighbours of the list (16 per warp) against tiles of LT_KEYS cached rows.  A tile is
-// staged once, as bf16 [key][channel], and serves both products on the tensor pipe (mma.sync m16n8k16, f32 accumulators): ldmatrix gives
-// its keys for the scores, ldmatrix.trans its first vdim channels as the values.  Two tiles in shared memory: the next one is loaded
-// (DK <= 128: into registers, ahead of the products) while this one is used.  Mask, online softmax and normalisation in f32.  DK / DV:
-// upper bounds of the row and of the latent.  Blocks start with the last tokens, which see the most keys.
-constexpr int LT_ROWS = 128, LT_KEYS = 64;
-template <int DK> constexpr size_t latent_tile_smem() { return (size_t)(LT_ROWS + 2 * LT_KEYS) * (DK + 8) * 2; }
-__device__ __forceinline__ void ldsm4(uint32_t* r, uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t* r, uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-template <int DK, int DV>
-__global__ void __launch_bounds__(256) lp_latent_tile_kernel(StepMeta sm, AttnGeom a, const float* __restrict__ qbuf, bf16* __restrict__ out) {
-    constexpr int PITCH = DK + 8, NU = LT_KEYS * (DK / 4) / 256;
-    constexpr bool AHEAD = DK <= 128;
-    extern __shared__ __align__(16) uint8_t lt_sm[];
-    bf16* Qs = reinterpret_cast<bf16*>(lt_sm);          // [LT_ROWS][PITCH]
-    bf16* Ks = Qs + LT_ROWS * PITCH;                    // [2][LT_KEYS][PITCH]
-    const int run = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
-    const int r0 = sm.run_start[run], len = sm.run_start[run + 1] - r0, p0 = sm.run_pos0[run];
-    const int rows = len * a.H, nb = (rows + LT_ROWS - 1) / LT_ROWS;
-    if ((int)blockIdx.x >= nb) return;
-    const int f0 = (nb - 1 - (int)blockIdx.x) * LT_ROWS, D = a.dim;
-    const float* cache = reinterpret_cast<const float*>(sm.run_kv[run] + a.kv_off);
-    const float* q = qbuf + ((size_t)r0 * a.H + f0) * D;
-    for (int u = threadIdx.x; u < LT_ROWS * (DK / 4); u += 256) {
-        const int f = u / (DK / 4), d = (u - f * (DK / 4)) * 4;
-        const float4 v = (f0 + f < rows && d < D) ? *reinterpret_cast<const float4*>(q + (size_t)f * D + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-        *reinterpret_cast<uint2*>(Qs + f * PITCH + d) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
-    }
-    const int last = p0 + min(f0 + LT_ROWS - 1, rows - 1) / a.H, lo = attn_lo(a, p0 + f0 / a.H);
-    const int tiles = (last - lo) / LT_KEYS + 1;
-    auto get = [&](int t, int u) {
-        const int i = threadIdx.x + u * 256, key = i / (DK / 4), d = (i - key * (DK / 4)) * 4, j = lo + t * LT_KEYS + key;
-        return (j <= last && d < D) ? *reinterpret_cast<const float4*>(cache + (size_t)j * D + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-    };
-    auto put = [&](int t, int u, const float4& v) {
-        const int i = threadIdx.x + u * 256, key = i / (DK / 4), d = (i - key * (DK / 4)) * 4;
-        *reinterpret_cast<uint2*>(Ks + ((t & 1) * LT_KEYS + key) * PITCH + d) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
-    };
-    auto stage = [&](int t) {
-#pragma unroll
-        for (int u0 = 0; u0 < NU; u0 += 4) {
-            float4 v[4];
-#pragma unroll
-            for (int u = 0; u < 4; u++) v[u] = get(t, u0 + u);
-#pragma unroll
-            for (int u = 0; u < 4; u++) put(t, u0 + u, v[u]);
-        }
-    };
-    stage(0);
-    // this thread's two rows of the warp's 16, their positions, and the warp's first and last position
-    const int fa = f0 + warp * 16 + gid, fb = fa + 8;
-    const int ia = p0 + min(fa, rows - 1) / a.H, ib = p0 + min(fb, rows - 1) / a.H;
-    const int w_first = p0 + min(f0 + warp * 16, rows - 1) / a.H, w_last = p0 + min(f0 + warp * 16 + 15, rows - 1) / a.H;
-    const uint32_t q_addr = smem_u32(Qs + (warp * 16 + (lane & 15)) * PITCH + (lane >> 4) * 8);
-    const uint32_t k_off = (uint32_t)(((lane & 7) + ((lane >> 4) << 3)) * PITCH + ((lane >> 3) & 1) * 8) * 2;
-    const uint32_t v_off = (uint32_t)(((lane & 7) + (((lane >> 3) & 1) << 3)) * PITCH + (lane >> 4) * 8) * 2;
-    const float sl = a.scale * 1.4426950408889634f;      // scores in powers of two
-    float o[DV / 8][4];
-#pragma unroll
-    for (int n = 0; n < DV / 8; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
-    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
-    __syncthreads();
-    for (int t = 0; t < tiles; t++) {
-        const int j0 = lo + t * LT_KEYS;
-        float4 nx[AHEAD ? NU : 1];
-        if (AHEAD && t + 1 < tiles) {
-#pragma unroll
-            for (int u = 0; u < NU; u++) nx[u % (AHEAD ? NU : 1)] = get(t + 1, u);
-        }
-        if (j0 <= w_last && j0 + LT_KEYS - 1 > w_first - a.window) {      // (some row of the warp sees some key of the tile)
-            const uint32_t kt = smem_u32(Ks + (t & 1) * LT_KEYS * PITCH);
-            float sc[LT_KEYS / 8][4];
-#pragma unroll
-            for (int n = 0; n < LT_KEYS / 8; n++) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.0f;
-#pragma unroll
-            for (int kb = 0; kb < DK / 16; kb++) {
-                if (kb * 16 < D) {
-                    uint32_t qa[4];
-                    ldsm4(qa, q_addr + kb * 32);
-#pragma unroll
-                    for (int n = 0; n < LT_KEYS / 16; n++) {
-                        uint32_t b[4];
-                        ldsm4(b, kt + k_off + (uint32_t)(n * 16 * PITCH + kb * 16) * 2);
-                        mma_bf16(sc[2 * n], qa, b[0], b[1]);
-                        mma_bf16(sc[2 * n + 1], qa, b[2], b[3]);
-                    }
-                }
-            }
-            const bool all = j0 + LT_KEYS - 1 <= w_first && j0 > w_last - a.window;     // nothing of the tile is masked
-            float x0 = -INFINITY, x1 = -INFINITY;
-#pragma unroll
-            for (int n = 0; n < LT_KEYS / 8; n++) {
-#pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    const int j = j0 + n * 8 + 2 * tig + (e & 1), i = (e & 2) ? ib : ia;
-                    sc[n][e] = (all || (j <= i && i - j < a.window)) ? sc[n][e] * sl : -INFINITY;
-                }
-                x0 = fmaxf(x0, fmaxf(sc[n][0], sc[n][1]));
-                x1 = fmaxf(x1, fmaxf(sc[n][2], sc[n][3]));
-            }
-            x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1));
-            x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
-            x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1));
-            x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-            const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
-            const float b0 = n0 == -INFINITY ? 0.0f : n0, b1 = n1 == -INFINITY ? 0.0f : n1;      // (a row without a visible key yet: all weights 0)
-            const float c0 = exp2f(m0 - b0), c1 = exp2f(m1 - b1);
-            m0 = n0;
-            m1 = n1;
-            float s0 = 0.0f, s1 = 0.0f;
-            uint32_t pa[LT_KEYS / 16][4];
-#pragma unroll
-            for (int n = 0; n < LT_KEYS / 8; n++) {
-                const float e0 = exp2f(sc[n][0] - b0), e1 = exp2f(sc[n][1] - b0), e2 = exp2f(sc[n][2] - b1), e3 = exp2f(sc[n][3] - b1);
-                s0 += e0 + e1;
-                s1 += e2 + e3;
-                pa[n >> 1][(n & 1) * 2] = pack_bf2(e0, e1);
-                pa[n >> 1][(n & 1) * 2 + 1] = pack_bf2(e2, e3);
-            }
-            l0 = l0 * c0 + s0;
-            l1 = l1 * c1 + s1;
-#pragma unroll
-            for (int n = 0; n < DV / 8; n++) {
-                o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1;
-            }
-#pragma unroll
-            for (int n = 0; n < DV / 16; n++) {
-                if (n * 16 < a.vdim) {
-#pragma unroll
-                    for (int k = 0; k < LT_KEYS / 16; k++) {
-                        uint32_t b[4];
-                        ldsm4_t(b, kt + v_off + (uint32_t)(k * 16 * PITCH + n * 16) * 2);
-                        mma_bf16(o[2 * n], pa[k], b[0], b[1]);
-                        mma_bf16(o[2 * n + 1], pa[k], b[2], b[3]);
-                    }
-                }
-            }
-        }
-        if (t + 1 < tiles) {
-            if (AHEAD) {
-#pragma unroll
-                for (int u = 0; u < NU; u++) put(t + 1, u, nx[u % (AHEAD ? NU : 1)]);
-            } else stage(t + 1);
-        }
-        __syncthreads();
-    }
-    l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
-    l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
-    l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
-    l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-    const float v0 = 1.0f / l0, v1 = 1.0f / l1;
-#pragma unroll
-    for (int n = 0; n < DV / 8; n++) {
-        const int c = n * 8 + 2 * tig;
-        if (c < a.vdim) {        // (vdim is even: c + 1 < vdim)
-            if (fa < rows) *reinterpret_cast<uint32_t*>(out + ((size_t)r0 * a.H + fa) * a.vdim + c) = pack_bf2(o[n][0] * v0, o[n][1] * v0);
-            if (fb < rows) *reinterpret_cast<uint32_t*>(out + ((size_t)r0 * a.H + fb) * a.vdim + c) = pack_bf2(o[n][2] * v1, o[n][3] * v1);
         }
     }
 }

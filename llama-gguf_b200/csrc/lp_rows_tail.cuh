@@ -7,16 +7,16 @@
 // Router of a mixture of experts for one row, by one warp: the `top` largest of z[0 .. E) are taken one after the other (of equal
 // logits the lower index first); their weights are the softmax over the chosen logits only (mode B200_ROUTE_TOP_SOFTMAX), or their
 // share of the softmax over ALL experts times `scale`, not renormalised (B200_ROUTE_SOFTMAX_TOP), or their own sigmoid, not
-// renormalised, times `scale` when that is not 0 (B200_ROUTE_SIGMOID_TOP).  w[e] receives the weight of
+// renormalised, times `scale` when that is not 0 (B200_ROUTE_SIGMOID_TOP).  corr: [E] added to the scores (the probability, the sigmoid)
+// that choose, not to the weights; null: the logits choose.  w[e] receives the weight of
 // expert e (0 when it is not chosen); sel[k] / selw[k] list the chosen experts in the order they were taken.
 __device__ __forceinline__ void route_row(const float* __restrict__ z, int E, int top, float* __restrict__ w, int* __restrict__ sel,
-                                          float* __restrict__ selw, int lane, int mode, float scale) {
+                                          float* __restrict__ selw, int lane, int mode, float scale, const float* __restrict__ corr = nullptr) {
     for (int e = lane; e < E; e += 32) w[e] = 0.0f;
     __syncwarp();
     float zmax = 0.0f, sum = 0.0f;
-    float all = 0.0f;
+    float all = 0.0f, mx = -INFINITY;
     if (mode == B200_ROUTE_SOFTMAX_TOP) {
-        float mx = -INFINITY;
         for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
         mx = wmax(mx);
         for (int e = lane; e < E; e += 32) all += expf(z[e] - mx);
@@ -26,7 +26,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ z, int E, in
         float best = -INFINITY;
         int bi = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            const float v = z[e];
+            const float v = !corr ? z[e] : (mode == B200_ROUTE_SIGMOID_TOP ? sigmoid_f(z[e]) : expf(z[e] - mx) / all) + corr[e];
             if (w[e] == 0.0f && (v > best || (v == best && e < bi))) { best = v; bi = e; }   // (chosen experts carry a mark != 0)
         }
 #pragma unroll
@@ -35,8 +35,10 @@ __device__ __forceinline__ void route_row(const float* __restrict__ z, int E, in
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
         }
-        if (k == 0) zmax = best;
-        const float p = mode == B200_ROUTE_SIGMOID_TOP ? sigmoid_f(best) : expf(best - zmax);
+        bi = min(bi, E - 1);            // (no score compares: not a number)
+        const float zb = z[bi];
+        if (k == 0) zmax = mode == B200_ROUTE_SOFTMAX_TOP ? mx : zb;
+        const float p = mode == B200_ROUTE_SIGMOID_TOP ? sigmoid_f(zb) : expf(zb - zmax);
         sum += p;
         if (lane == 0) {
             w[bi] = -1.0f - p;          // mark; turned into the weight below

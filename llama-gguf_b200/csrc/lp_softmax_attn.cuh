@@ -129,7 +129,8 @@ __global__ void __launch_bounds__(256) lp_attn_prep2_kernel(StepMeta sm, AttnGeo
     }
     float* kc = reinterpret_cast<float*>(sm.run_kv[run] + a.kv_off) + (size_t)pos * nk;
     float* vc = reinterpret_cast<float*>(sm.run_kv[run] + a.kv_off) + (size_t)a.cap * nk + (size_t)pos * a.G * a.vdim;
-    for (int c = threadIdx.x; c < nq; c += blockDim.x) qbuf[(size_t)r * nq + c] = y[c];
+    const float temp = attn_temp(a, pos);
+    for (int c = threadIdx.x; c < nq; c += blockDim.x) qbuf[(size_t)r * nq + c] = y[c] * temp;
     for (int c = threadIdx.x; c < nk; c += blockDim.x) kc[c] = y[nq + c];
     const int nv = a.G * a.vdim;
     const float lam = g.v_mix == B200_VMIX_BLEND ? *lam_p : 0.0f;

@@ -34,7 +34,12 @@ def _fizesun(path, **kw):
     return fizesun.load(path, **kw)
 
 
-LOADERS = {"Lazilorn": _lazilorn, "Mefurax": _mefurax, "Madudra": _madudra, "Marosun": _marosun, "Fizesun": _fizesun}
+def _gefovik(path, **kw):
+    from . import gefovik
+    return gefovik.load(path, **kw)
+
+
+LOADERS = {"Lazilorn": _lazilorn, "Mefurax": _mefurax, "Madudra": _madudra, "Marosun": _marosun, "Fizesun": _fizesun, "Gefovik": _gefovik}
 
 
 def architecture_of(path):
