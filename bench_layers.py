@@ -1,10 +1,11 @@
-"""bench.py --design lazilorn | mefurax | madudra | marosun | fizesun: prefill and decode throughput of a layer-program design at sizes that resemble a real model's
+"""bench.py --design lazilorn | mefurax | madudra | marosun | fizesun | gefovik: prefill and decode throughput of a layer-program design at sizes that resemble a real model's
 layers (random weights), beside the library's closest existing model -- a llama-architecture transformer of the same width, depth
 and parameter count in Q8_0 blocks (the densest weight type its tensor-core prompt path takes); Mefurax also beside Lazilorn at
 the same width and depth (the other bf16 layer program, whose attention and GEMM kernels it shares); Madudra beside Lazilorn (the
 other hybrid of attention and recurrent scans) and Mefurax (the other mixture of experts) at the same width and depth; Marosun beside
 the same two (Lazilorn: attention beside a matrix memory; Mefurax: softmax mixers with rotation and experts); Fizesun beside Madudra (the other latent attention) and Mefurax (the other mixture with an
-always-on expert) at the same width and as many layer runs.
+always-on expert) at the same width and as many layer runs; Gefovik beside Mefurax (soft-capped grouped attention, experts, norms outside
+the sublayers' inputs) and Fizesun (latent attention without a query latent, gated experts) at the same width and depth.
 
 Per size and model: prompt tokens/s for one prompt of --prefill-len tokens, decode tokens/s at batch 1 and at --batch sequences
 after prompts of --prompt-len tokens.  Every number is host wall clock around the library call (each call ends with a stream
@@ -139,6 +140,31 @@ def fizesun_config(s):
             "loop": {"start": a, "stop": b, "times": t}, "layers": layers}
 
 
+GEFOVIK_SIZES = {
+    # name: width, layers (a = softmax attention with values from the keys, l = latent attention; D = dense gated relu, M = mixture of gated
+    # experts with identity experts), heads / kv heads, dense ff, experts / identity / chosen / expert ff
+    "w1024": dict(width=1024, pattern=["aD", "lM", "aM", "lD", "aM", "lM"], heads=8, kv_heads=2, ff=4096, experts=8, identity=2, top=2, eff=1024, vocab=32000),
+    "w2048": dict(width=2048, pattern=["aD", "lM", "aM", "lM", "aD", "lM", "aM", "lM"], heads=16, kv_heads=4, ff=8192, experts=8, identity=2, top=2, eff=2048,
+                  vocab=32000),
+}
+
+
+def gefovik_config(s):
+    # heads of 128 (softmax) and of 96 query / key and 128 value channels over a latent of 128 (the cached row of madudra_config's width)
+    layers = []
+    for ch, ff in s["pattern"]:
+        mlp = {"kind": "dense", "ff": s["ff"]} if ff == "D" else {"kind": "moe", "router": {"experts": s["experts"], "identity": s["identity"], "top": s["top"]},
+                                                                  "expert": {"ff": s["eff"]}}
+        if ch == "a":
+            layers.append({"type": "attention", "mlp": mlp,
+                           "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+                                     "q_temp": {"coef": 0.1, "every": 1024}}})
+        else:
+            layers.append({"type": "latent_attention", "mlp": mlp,
+                           "mixer": {"heads": s["heads"], "dim": 96, "vdim": 128, "kv_rank": 128, "scale": 96 ** -0.5}})
+    return {"architecture": "Gefovik", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": layers}
+
+
 def lazilorn_feeder(cfg, seed, tensor_shapes=None):
     """upload(name, type, ne, data) for every tensor of cfg: bf16 bit patterns of N(0, 1/fan_in) matrices, f32 vectors."""
     import llama_gguf_b200 as B
@@ -167,6 +193,8 @@ def lazilorn_feeder(cfg, seed, tensor_shapes=None):
                 a = rng.uniform(1.0, 4.0, shape)
             elif last == "lower":
                 a = rng.uniform(0.0, 0.9, shape)
+            elif last == "correction":
+                a = 0.1 * rng.standard_normal(shape)
             elif last in ("A_log", "dt_bias", "b") and len(shape) == 1:
                 a = rng.uniform(-2.0, 0.5, shape)
             elif (last in ("norm1", "norm2", "vmix") or name == "final.norm") and cfg["architecture"] in ("Mefurax", "Marosun"):
@@ -178,8 +206,8 @@ def lazilorn_feeder(cfg, seed, tensor_shapes=None):
 
 
 def design_module(cfg):
-    from llama_gguf_b200 import fizesun, lazilorn, madudra, marosun, mefurax
-    return {"Lazilorn": lazilorn, "Mefurax": mefurax, "Madudra": madudra, "Marosun": marosun, "Fizesun": fizesun}[cfg["architecture"]]
+    from llama_gguf_b200 import fizesun, gefovik, lazilorn, madudra, marosun, mefurax
+    return {"Gefovik": gefovik, "Lazilorn": lazilorn, "Mefurax": mefurax, "Madudra": madudra, "Marosun": marosun, "Fizesun": fizesun}[cfg["architecture"]]
 
 
 def n_params(cfg):
@@ -275,6 +303,8 @@ def main(args):
         return main_marosun(args)
     if args.design == "fizesun":
         return main_fizesun(args)
+    if args.design == "gefovik":
+        return main_gefovik(args)
     sizes = [x for x in (args.sizes.split(",") if args.sizes else SIZES) if x]
     max_seq = max(args.prefill_len, args.prompt_len + args.warmup + args.steps + 8) + 8
     res = {}
@@ -386,4 +416,28 @@ def main_fizesun(args):
     print(json.dumps({"bench": "design", "design": "fizesun", "unit": "tok/s", "prefill_len": args.prefill_len, "prompt_len": args.prompt_len,
                       "batch": args.batch, "steps": args.steps, "warmup": args.warmup, "timing": "host wall clock around the library calls",
                       "dtype": "bf16 (fizesun, madudra, mefurax at the same width and number of layer runs)", "data": "synthetic", "sizes": res}))
+    return 0
+
+
+def main_gefovik(args):
+    sizes = [x for x in (args.sizes.split(",") if args.sizes else GEFOVIK_SIZES) if x]
+    max_seq = max(args.prefill_len, args.prompt_len + args.warmup + args.steps + 8) + 8
+    res = {}
+    for name in sizes:
+        s = GEFOVIK_SIZES[name]
+        cfg = gefovik_config(s)
+        params = n_params(cfg)
+        n_moe = sum(1 for p in s["pattern"] if p[1] == "M")
+        # (a token whose choices are all real experts; an identity expert has no parameters)
+        active = params - n_moe * (s["experts"] - s["top"]) * 3 * s["width"] * s["eff"]
+        r = {"params_without_embedding": params, "active_params_without_embedding": active, "layers": ",".join(s["pattern"]),
+             "gefovik_bf16": bench_lazilorn(cfg, args, max_seq)}
+        print(name, json.dumps(r), file=sys.stderr, flush=True)
+        r["mefurax_bf16"] = bench_lazilorn(mefurax_config(MEFURAX_SIZES[name]), args, max_seq)
+        r["fizesun_bf16"] = bench_lazilorn(fizesun_config(FIZESUN_SIZES[name]), args, max_seq)
+        res[name] = r
+        print(name, json.dumps(r), file=sys.stderr, flush=True)
+    print(json.dumps({"bench": "design", "design": "gefovik", "unit": "tok/s", "prefill_len": args.prefill_len, "prompt_len": args.prompt_len,
+                      "batch": args.batch, "steps": args.steps, "warmup": args.warmup, "timing": "host wall clock around the library calls",
+                      "dtype": "bf16 (gefovik, mefurax, fizesun at the same width and number of layer runs)", "data": "synthetic", "sizes": res}))
     return 0

@@ -141,8 +141,10 @@ __global__ void lp_rmsnorm_kernel(float* __restrict__ x, const float* __restrict
 // ------------------------------------------------------------------------------------------------ GEMM (CUDA cores)
 // Y[r][n] = epi(alpha * sum_k X[r][k] * W[n][k] + bias[n]); products of the stored operand values in f32, f32 accumulation
 // (bias: f32 per output column, or null).  act: the two numbers of the xIELU epilogue, (softplus(p), 1/2 + softplus(q)).
-// EPI_RELU_GLU: relu(v) * up, the unit of a gated layer from its two products (the kernels that have both at hand).
-enum { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2, EPI_GELU = 3, EPI_XIELU = 4, EPI_RELU_GLU = 5, EPI_COUNT = 6 };
+// EPI_RELU_GLU, EPI_SILU_GLU: the unit of a gated layer, relu(v) * up or silu(v) * up, from its two products, N units out of a matrix of 2 N
+// rows [gate | up] (lp_gemm_tc_kernel, lp_gemv_mma_kernel, lp_gemv_norm_kernel).
+enum { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2, EPI_GELU = 3, EPI_XIELU = 4, EPI_RELU_GLU = 5, EPI_SILU_GLU = 6, EPI_COUNT = 7 };
+constexpr bool epi_is_glu(int epi) { return epi == EPI_RELU_GLU || epi == EPI_SILU_GLU; }
 constexpr bool epi_is_act(int epi) { return epi >= EPI_RELU2; }
 // act.x z^2 + z / 2 above zero, act.y (exp(z) - 1 - z) + z / 2 below
 __device__ __forceinline__ float xielu_f(float z, float2 act) { return fmaf(0.5f, z, z > 0.0f ? act.x * z * z : act.y * (expm1f(z) - z)); }
@@ -154,6 +156,7 @@ __device__ __forceinline__ void epi_store(void* Y, size_t idx, float v, float2 a
     else if (EPI == EPI_GELU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(gelu_erf_f(v));
     else if (EPI == EPI_XIELU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(xielu_f(v, act));
     else if (EPI == EPI_RELU_GLU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(fmaxf(v, 0.0f) * up);
+    else if (EPI == EPI_SILU_GLU) reinterpret_cast<T*>(Y)[idx] = from_f<T>(v * sigmoid_f(v) * up);
     else {
         const float z = fmaxf(v, 0.0f);
         reinterpret_cast<T*>(Y)[idx] = from_f<T>(z * z);
@@ -236,6 +239,8 @@ __global__ void __launch_bounds__(256) lp_gemm_kernel(const T* __restrict__ X, i
 // stage's mbarrier; a stage is refilled when that commit has arrived.  Epilogue: warp w reads TMEM lanes 32w .. 32w + 31 (= weight
 // rows) 32 token columns at a time; a warp's stores of one token are 32 consecutive outputs.  Every mbarrier wait is bounded: a
 // wait that gives up sets *err and the CTA drains its copies, frees its TMEM columns and returns.
+// Gated epilogues: the tile's 128 weight rows are 64 units' gate rows and the same units' up rows; the two halves of the CTA exchange half
+// of their tokens' sums through the (drained) stages and each makes the units of the other half.
 constexpr int TC_M = 128, TC_K = 64, TC_STAGES = 4;
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 // K-major SWIZZLE_128B shared-memory matrix descriptor: start >> 4, LBO (unused) = 1, SBO = 1024 bytes between 8-row groups,
@@ -266,6 +271,18 @@ __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, uint32
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
 }
 
+// 32 columns of this warp's 32 TMEM lanes
+__device__ __forceinline__ void tc_ld32(uint32_t* v, uint32_t taddr) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
+          "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]), "=r"(v[17]), "=r"(v[18]),
+          "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]),
+          "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
+        : "r"(taddr));
+}
+
 template <int TN, int EPI>
 __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict__ X, int ldx, const bf16* __restrict__ W, int ldw,
                                                          void* __restrict__ Y, int ldy, int R, int N, int K, float alpha, int* err,
@@ -291,7 +308,8 @@ __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict_
     constexpr int kStage = (TC_M + TN) * 128;
     uint8_t* base = tc_smem + ((1024u - (smem_u32(tc_smem) & 1023u)) & 1023u);   // the swizzle is on absolute address bits
     const int tid = threadIdx.x, warp = tid >> 5;
-    const int n0 = blockIdx.x * TC_M, t0 = blockIdx.y * TN;
+    constexpr bool GLU = epi_is_glu(EPI);
+    const int n0 = blockIdx.x * (GLU ? TC_M / 2 : TC_M), t0 = blockIdx.y * TN;
     const uint32_t bar = smem_u32(&s_bar[0]);
     constexpr int kCols = TN < 32 ? 32 : TN;
     if (tid == 0) {
@@ -317,9 +335,10 @@ __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict_
         const int k0 = st * TC_K;
 #pragma unroll
         for (int u = 0; u < 8; u++) {
-            const int i = tid + u * 128, r = i >> 3, c = i & 7, n = n0 + r, k = k0 + 8 * c;
+            const int i = tid + u * 128, r = i >> 3, c = i & 7, n = n0 + (GLU ? r & (TC_M / 2 - 1) : r), k = k0 + 8 * c;
             const bool in = n < N && k < K;
-            cp_async16(smem_u32(tA + tc_sw128(r, c)), in ? (const void*)(W + (size_t)n * ldw + k) : (const void*)W, in ? 16u : 0u);
+            const size_t wrow = GLU && r >= TC_M / 2 ? (size_t)N + n : (size_t)n;
+            cp_async16(smem_u32(tA + tc_sw128(r, c)), in ? (const void*)(W + wrow * ldw + k) : (const void*)W, in ? 16u : 0u);
         }
 #pragma unroll
         for (int u = 0; u < TN / 16; u++) {
@@ -372,22 +391,40 @@ __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict_
         if (err) atomicExch(err, 2);
     }
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    const int n = n0 + tid;
+    const int n = n0 + (GLU ? tid & (TC_M / 2 - 1) : tid);
     const float bn = (bias && n < N) ? bias[n] : 0.0f;
-    if (alive) {
+    if constexpr (GLU) {
+        float* ex = reinterpret_cast<float*>(base);        // [2 halves][16 tokens][64 units]
+        const bool up = tid >= TC_M / 2;
+        __syncthreads();                                    // every thread's copies have landed, every MMA has read its stage
+#pragma unroll 1
+        for (int c0 = 0; c0 < TN; c0 += 32) {
+            if (t0 + c0 >= R) break;   // CTA-uniform
+            uint32_t v[32];
+#pragma unroll
+            for (int c = 0; c < 32; c++) v[c] = 0u;
+            if (alive) {
+                tc_ld32(v, tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0);
+                asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+            }
+#pragma unroll
+            for (int c = 0; c < 16; c++) ex[(up ? 0 : 16 * 64) + c * 64 + (tid & 63)] = __uint_as_float(v[up ? c : 16 + c]);
+            __syncthreads();
+#pragma unroll
+            for (int c = 0; c < 16; c++) {
+                const float mine = alpha * __uint_as_float(v[up ? 16 + c : c]), other = alpha * ex[(up ? 16 * 64 : 0) + c * 64 + (tid & 63)];
+                const int t = t0 + c0 + (up ? 16 + c : c);
+                if (alive && n < N && t < R) epi_store<bf16, EPI>(Y, (size_t)t * ldy + n, up ? other : mine, act, up ? mine : other);
+            }
+            __syncthreads();
+        }
+    } else if (alive) {
 #pragma unroll 1
         for (int c0 = 0; c0 < TN; c0 += 32) {
             if (t0 + c0 >= R) break;   // CTA-uniform
             uint32_t v[32];
             const uint32_t taddr = tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0;
-            asm volatile(
-                "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-                "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-                : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
-                  "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]), "=r"(v[17]), "=r"(v[18]),
-                  "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]),
-                  "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-                : "r"(taddr));
+            tc_ld32(v, taddr);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             if (EPI == EPI_ADD && n < N) {   // all 32 sums are read before the first one is written
                 float old[32];
@@ -548,7 +585,7 @@ __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b
 // B = 8 activation rows, NT of them), because the CUDA cores would spend a multiply and an unpack per weight and row.  A block takes 16
 // weight rows, its 8 warps take K in chunks of 32 in turn; a lane's 16-byte load holds 8 consecutive k of one row, for both operands
 // alike, so the order of k inside a chunk does not matter to the sum.  The warps' 16 x 8 NT parts meet in shared memory, warp order.
-// K a multiple of 32, rows 16-byte aligned.
+// K a multiple of 32, rows 16-byte aligned.  Gated epilogues: the block's 16 weight rows are 8 units' gate rows and their up rows.
 template <int EPI, int NT>
 __global__ void __launch_bounds__(256) lp_gemv_mma_kernel(const bf16* __restrict__ X, int ldx, const bf16* __restrict__ W, int ldw, void* __restrict__ Y, int ldy,
                                                           int R, int N, int K, float alpha, RowsTail tail, const float* __restrict__ bias, float2 act) {
@@ -557,9 +594,10 @@ __global__ void __launch_bounds__(256) lp_gemv_mma_kernel(const bf16* __restrict
     const bf16* xr[NT];
 #pragma unroll
     for (int t = 0; t < NT; t++) xr[t] = X + (size_t)min(t * 8 + gid, R - 1) * ldx + tig * 8;
-    for (int n0 = blockIdx.x * 16; n0 < N; n0 += gridDim.x * 16) {
+    constexpr int NB = epi_is_glu(EPI) ? 8 : 16;
+    for (int n0 = blockIdx.x * NB; n0 < N; n0 += gridDim.x * NB) {
         const bf16* wa = W + (size_t)min(n0 + gid, N - 1) * ldw + tig * 8;
-        const bf16* wb = W + (size_t)min(n0 + gid + 8, N - 1) * ldw + tig * 8;
+        const bf16* wb = W + (epi_is_glu(EPI) ? (size_t)N + min(n0 + gid, N - 1) : (size_t)min(n0 + gid + 8, N - 1)) * ldw + tig * 8;
         float c[NT][4];
 #pragma unroll
         for (int t = 0; t < NT; t++) c[t][0] = c[t][1] = c[t][2] = c[t][3] = 0.0f;
@@ -584,12 +622,16 @@ __global__ void __launch_bounds__(256) lp_gemv_mma_kernel(const bf16* __restrict
             d[24] = c[t][3];
         }
         __syncthreads();
-        for (int i = threadIdx.x; i < 16 * R; i += 256) {
-            const int r = i >> 4, n = n0 + (i & 15);
-            float v = 0.0f;
+        for (int i = threadIdx.x; i < NB * R; i += 256) {
+            const int r = i / NB, n = n0 + i % NB, at = r * 16 + i % NB;
+            float v = 0.0f, u = 0.0f;
 #pragma unroll
-            for (int w = 0; w < 8; w++) v += red[w][i];
-            if (n < N) epi_store<bf16, EPI>(Y, (size_t)r * ldy + n, alpha * v + (bias ? bias[n] : 0.0f), act);
+            for (int w = 0; w < 8; w++) v += red[w][at];
+            if (epi_is_glu(EPI)) {
+#pragma unroll
+                for (int w = 0; w < 8; w++) u += red[w][at + 8];
+            }
+            if (n < N) epi_store<bf16, EPI>(Y, (size_t)r * ldy + n, alpha * v + (bias ? bias[n] : 0.0f), act, alpha * u);
         }
     }
     if (tail.on) rows_tail<bf16>(tail);
@@ -663,11 +705,11 @@ __global__ void __launch_bounds__(256) lp_gemv_norm_kernel(const float* __restri
             const int nr = min(NR, R - rb);
             float acc[NR], accu[NR];
             gemv_dot<T, NR>(wr, xs + (size_t)rb * K, K, nr, K, lane, acc);
-            if (EPI == EPI_RELU_GLU) gemv_dot<T, NR>(wr + (size_t)N * K, xs + (size_t)rb * K, K, nr, K, lane, accu);     // (W: [gate | up], N units)
+            if (epi_is_glu(EPI)) gemv_dot<T, NR>(wr + (size_t)N * K, xs + (size_t)rb * K, K, nr, K, lane, accu);     // (W: [gate | up], N units)
 #pragma unroll
             for (int i = 0; i < NR; i++) {
                 if (i < nr) {
-                    const float sum = wsum(acc[i]), up = EPI == EPI_RELU_GLU ? wsum(accu[i]) : 0.0f;
+                    const float sum = wsum(acc[i]), up = epi_is_glu(EPI) ? wsum(accu[i]) : 0.0f;
                     if (lane == 0) epi_store<T, EPI>(Y, (size_t)(rb + i) * ldy + n, alpha * sum, act, up);
                 }
             }
@@ -1736,7 +1778,8 @@ bool tc_launch(LpModel* m, const bf16* x, int ldx, const bf16* w, int ldw, int N
         if (dev >= 0 && dev < 64) once[e][dev] = true;
         return true;
     };
-    dim3 grid((N + TC_M - 1) / TC_M, (R + TN - 1) / TN, groups), block(128);
+    const int per_cta = epi_is_glu(epi) ? TC_M / 2 : TC_M;
+    dim3 grid((N + per_cta - 1) / per_cta, (R + TN - 1) / TN, groups), block(128);
 #define LP_TC(E)                                                                                                                       \
     do {                                                                                                                               \
         if (!prep(lp_gemm_tc_kernel<TN, E>, E)) return false;                                                                          \
@@ -1746,14 +1789,19 @@ bool tc_launch(LpModel* m, const bf16* x, int ldx, const bf16* w, int ldw, int N
     else if (epi == EPI_ADD) LP_TC(EPI_ADD);
     else if (epi == EPI_GELU) LP_TC(EPI_GELU);
     else if (epi == EPI_XIELU) LP_TC(EPI_XIELU);
+    else if (epi == EPI_RELU_GLU) LP_TC(EPI_RELU_GLU);
+    else if (epi == EPI_SILU_GLU) LP_TC(EPI_SILU_GLU);
     else LP_TC(EPI_RELU2);
 #undef LP_TC
     return true;
 }
+bool tc_takes(const LpModel* m, const void* X, int ldx, const void* W, int ldw, int K, int R, size_t wz, ZStride zs) {
+    if (m->f32 || !m->use_tc || R < m->tc_min_rows) return false;
+    return !(K % 8 || ldx % 8 || ldw % 8 || wz % 8 || zs.x % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15));
+}
 bool tc_gemm(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, int K, void* Y, int ldy, int R, float alpha, int epi, const int* seg,
              int groups, size_t wz, ZStride zs, const float* bias, float2 act) {
-    if (m->f32 || !m->use_tc || R < m->tc_min_rows) return false;
-    if (K % 8 || ldx % 8 || ldw % 8 || wz % 8 || zs.x % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return false;
+    if (!tc_takes(m, X, ldx, W, ldw, K, R, wz, zs)) return false;
     const bf16* x = (const bf16*)X;
     const bf16* w = (const bf16*)W;
     if (R <= 64) return tc_launch<64>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias, act);
@@ -1761,6 +1809,13 @@ bool tc_gemm(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, 
     return tc_launch<256>(m, x, ldx, w, ldw, N, K, Y, ldy, R, alpha, epi, seg, groups, wz, zs, bias, act);
 }
 
+// Whether gemm / project_in can end with a gated epilogue for these rows (K: the products' length; few: the input is made by the projection)
+bool glu_takes(const LpModel* m, const void* X, const void* W, int K, int R) {
+    if (!m->use_fuse || m->f32) return false;
+    if (R <= 2 || (!m->use_gemv_mma && R <= 2 * GV_ROWS)) return false;
+    if (R <= 2 * GV_ROWS) return K % 32 == 0 && ((uintptr_t)X % 16) == 0 && ((uintptr_t)W % 16) == 0;
+    return tc_takes(m, X, K, W, K, K, R, 0, ZStride{0, 0});
+}
 // Y = epi(alpha X W^T): rows of the step against a [N][K] matrix in the compute type.  Without `seg`, groups > 1 batches the product
 // over heads: head z multiplies columns [z zs.x, z zs.x + K) of X with rows [z N, (z + 1) N) of W (wz = N ldw) into columns
 // [z zs.y, z zs.y + N) of Y.
@@ -1777,7 +1832,8 @@ void gemm_t(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, i
         if constexpr (sizeof(T) == 2) {
             if (R >= 3 && m->use_gemv_mma && !heads && vec_ok && K % 32 == 0) {
                 const RowsTail tl = tail ? *tail : RowsTail{};
-                const dim3 g((unsigned)std::min((N + 15) / 16, 8 * 148)), b(256);
+                const int nb = epi_is_glu(epi) ? 8 : 16;
+                const dim3 g((unsigned)std::min((N + nb - 1) / nb, 8 * 148)), b(256);
 #define LP_GT(E)                                                                                                                            \
     do {                                                                                                                                    \
         if (R <= 8) launch(m, lp_gemv_mma_kernel<E, 1>, g, b, 0, x, ldx, w, ldw, Y, ldy, R, N, K, alpha, tl, bias, act);                    \
@@ -1787,6 +1843,7 @@ void gemm_t(LpModel* m, const void* X, int ldx, const void* W, int ldw, int N, i
                 else if (epi == EPI_ADD) LP_GT(EPI_ADD);
                 else if (epi == EPI_GELU) LP_GT(EPI_GELU);
                 else if (epi == EPI_XIELU) LP_GT(EPI_XIELU);
+                else if (epi == EPI_RELU_GLU) LP_GT(EPI_RELU_GLU);
                 else LP_GT(EPI_RELU2);
 #undef LP_GT
                 return;
@@ -3011,8 +3068,10 @@ void row_split(LpModel* m, const StepMeta& sm, const AttnGeom& ag, const float* 
 #undef LP_RS
 }
 void row_combine(LpModel* m, const AttnGeom& ag, int R, int splits) {
-    if (m->f32) launch(m, lp_row_combine_kernel<float>, dim3(R, ag.H), dim3(128), 0, ag.H, ag.vdim, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (float*)m->act_a, ag.out_ld);
-    else launch(m, lp_row_combine_kernel<bf16>, dim3(R, ag.H), dim3(128), 0, ag.H, ag.vdim, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (bf16*)m->act_a, ag.out_ld);
+#define LP_RC(T, V) launch(m, lp_row_combine_kernel<T, V>, dim3(R, ag.H), dim3(256), 0, ag.H, ag.vdim, (const float*)m->lat_o, (const float*)m->lat_ml, splits, (T*)m->act_a, ag.out_ld)
+    if (m->f32) { if (ag.vdim % 4) LP_RC(float, 1); else LP_RC(float, 4); }
+    else { if (ag.vdim % 4) LP_RC(bf16, 1); else LP_RC(bf16, 4); }
+#undef LP_RC
 }
 
 // Every kernel of one step, in order, on the model's stream: eagerly, or while the stream is being captured into a CUDA graph (a
@@ -3143,6 +3202,11 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
 #undef LP_NC
         conv_at++;
     };
+    // form with the norm on the output: the next projection of a few rows makes its own input (gemv_norm_t's conditions)
+    auto few_in = [&](const void* Wm) {
+        return out_norm && sub_pend.y && m->use_fuse && R <= (m->f32 || !m->use_gemv_mma || W % 32 ? 2 * GV_ROWS : 2) && W % (m->f32 ? 4 : 8) == 0 &&
+               ((uintptr_t)Wm & 15) == 0 && (size_t)R * W * elt(m) <= 96 * 1024;
+    };
     auto project_in = [&](const float* add, const float* nw, const void* Wm, int N, void* Y, int ldy, int epi) {
         const float2 act = cur->act2;
         if (p.in_conv > 0) {
@@ -3159,7 +3223,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             boundary(cur->hc_in[sub], nw, nullptr);
             gemm(m, m->hn, W, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, nullptr, act);
         } else if (out_norm) {
-            if (sub_pend.y && m->use_fuse) {
+            if (few_in(Wm)) {
                 SubNorm sn = sub_pend;
                 sn.xout = m->x2;
                 if (m->f32 ? gemv_norm_t<float>(m, m->x, nullptr, nullptr, Wm, N, W, Y, ldy, R, 1.0f, epi, nullptr, act, InConv{}, sm, sn)
@@ -3457,9 +3521,12 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             // Router logits (f32) -> the choice per row -> the experts -> m->y -> the residual.
             const b200_moe_desc& e = L.d.moe;
             const size_t es = elt(m);
-            const int act_epi = e.act == B200_ACT_GELU ? EPI_GELU : EPI_RELU2;
+            const int act_epi = e.act == B200_ACT_GELU ? EPI_GELU : e.act == B200_ACT_SILU_GLU ? EPI_SILU_GLU : e.act == B200_ACT_RELU_GLU ? EPI_RELU_GLU : EPI_RELU2;
             const int per = act_gated(e.act) ? 2 * e.expert_ff : e.expert_ff;                // rows of one expert's up matrix
-            const bool own_act = act_gated(e.act) || e.weight_input != 0;                      // the hidden units need a kernel of their own
+            // gated experts whose weights go onto their outputs: the units in the grouped product's epilogue
+            const bool glu_epi = (e.act == B200_ACT_SILU_GLU || e.act == B200_ACT_RELU_GLU) && !e.weight_input && m->use_fuse &&
+                                 tc_takes(m, m->moe_xp, W, (const uint8_t*)L.w_up + (size_t)L.up_router_rows * W * es, W, W, R, (size_t)per * W, ZStride{0, 0});
+            const bool own_act = (act_gated(e.act) && !glu_epi) || e.weight_input != 0;        // the hidden units need a kernel of their own
             const ExpertAct ea{e.act, e.weight_input, e.limit, e.shared_limit, e.slope};
             const int outs = e.experts + e.identity;                                            // what the router chooses among
             const int rrows = outs + (e.shared_gate ? 1 : 0);                                  // logits of a row: these, then the always-on gate's
@@ -3528,7 +3595,7 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
                     else { if (V == 4) LP_PA(bf16, 4); else LP_PA(bf16, 1); }
 #undef LP_PA
                 } else {
-                    gemm_grouped(m, m->moe_xp, W, up_experts, W, (size_t)e.expert_ff * W, e.experts, e.expert_ff, W, m->act_a, e.expert_ff, R, act_epi, m->moe_seg);
+                    gemm_grouped(m, m->moe_xp, W, up_experts, W, (size_t)per * W, e.experts, e.expert_ff, W, m->act_a, e.expert_ff, R, act_epi, m->moe_seg);
                 }
                 gemm_grouped(m, m->act_a, e.expert_ff, down, L.k_down, (size_t)e.expert_ff, e.experts, W, e.expert_ff, m->moe_yp, W, R, EPI_STORE, m->moe_seg);
                 if (e.shared_ff > 0) {
@@ -3582,9 +3649,12 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             const float* ffP = m->P;
             int ff_ld = L.n_up;
             if (par) { ffP = m->P + L.ff_off; ff_ld = L.n_in; }
-            else project_in(nullptr, L.norm2, L.w_up, L.n_up, m->P, L.n_up, EPI_STORE);
+            const bool gated_epi = L.d.ff_kind == B200_FF_GATED_RELU && !par && out_norm && (few_in(L.w_up) || glu_takes(m, m->hn, L.w_up, W, R));
+            if (gated_epi) project_in(nullptr, L.norm2, L.w_up, L.d.ff, m->act_a, L.d.ff, EPI_RELU_GLU);       // (the units in the product's epilogue)
+            else if (!par) project_in(nullptr, L.norm2, L.w_up, L.n_up, m->P, L.n_up, EPI_STORE);
             const unsigned nb = (unsigned)(((size_t)R * L.d.ff + 255) / 256);
-            if (L.d.ff_kind == B200_FF_GATED_RELU) {      // (an always-on expert's units without a gate)
+            if (gated_epi) {
+            } else if (L.d.ff_kind == B200_FF_GATED_RELU) {      // (an always-on expert's units without a gate)
                 const ExpertAct ea{B200_ACT_RELU_GLU, 0, 0.0f, 0.0f, 0.0f};
                 const bool v4 = L.d.ff % 4 == 0 && ff_ld % 4 == 0 && ((uintptr_t)ffP & 15) == 0;
                 const unsigned nb4 = (unsigned)(((size_t)R * (L.d.ff / 4) + 255) / 256);

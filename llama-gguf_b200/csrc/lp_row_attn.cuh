@@ -18,7 +18,13 @@ __global__ void __launch_bounds__(256) lp_row_prep_kernel(StepMeta sm, AttnGeom 
     float* rows = reinterpret_cast<float*>(sm.run_kv[run] + a.kv_off);
     float* dst = isq ? qbuf + ((size_t)r * a.H + h) * a.dim : rows + ((size_t)pos * a.G + g) * a.dim;
     float ss = 0.0f;
-    for (int d = lane * V; d < a.dim; d += 32 * V) {
+    FloatV<V> f0;
+#pragma unroll
+    for (int e = 0; e < V; e++) f0.v[e] = 0.0f;
+    if (lane * V < a.dim) f0 = load_v<V>(src + lane * V);
+#pragma unroll
+    for (int e = 0; e < V; e++) ss = fmaf(f0.v[e], f0.v[e], ss);
+    for (int d = (lane + 32) * V; d < a.dim; d += 32 * V) {
         const FloatV<V> f = load_v<V>(src + d);
 #pragma unroll
         for (int e = 0; e < V; e++) ss = fmaf(f.v[e], f.v[e], ss);
@@ -26,7 +32,7 @@ __global__ void __launch_bounds__(256) lp_row_prep_kernel(StepMeta sm, AttnGeom 
     const float inv = a.k_inv ? 1.0f / sqrtf(wsum(ss) / (float)a.dim + a.eps) : 1.0f;
     const float mul = isq ? inv * attn_temp(a, pos) : 1.0f;
     for (int d = lane * V; d < a.dim; d += 32 * V) {
-        FloatV<V> f = load_v<V>(src + d);
+        FloatV<V> f = d == lane * V ? f0 : load_v<V>(src + d);
 #pragma unroll
         for (int e = 0; e < V; e++) f.v[e] *= mul;
         store_v<V>(dst + d, f);
@@ -170,31 +176,54 @@ __global__ void __launch_bounds__(32 * LS_HEADS) lp_row_split_kernel(StepMeta sm
     }
 }
 
-// The merge of the splits: every (row, head)'s weighted values in the compute type -> out[r][h vdim ..] (rows out_ld apart)
-template <typename T>
-__global__ void __launch_bounds__(128) lp_row_combine_kernel(int H, int vdim, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
+// The merge of the splits: every (row, head)'s weighted values in the compute type -> out[r][h vdim ..] (rows out_ld apart).  The block's
+// warps deal the splits among themselves; V channels per lane (4: vdim a multiple of 4), LC_BATCH splits in flight.
+constexpr int LC_BATCH = 8;
+template <typename T, int V>
+__global__ void __launch_bounds__(256) lp_row_combine_kernel(int H, int vdim, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
                                                              T* __restrict__ out, int out_ld) {
-    __shared__ float wgt[64];              // (splits <= 64)
-    const int lane = threadIdx.x & 31;
+    __shared__ float wgt[64], part[8][32 * V];              // (splits <= 64)
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const size_t at = ((size_t)blockIdx.x * H + blockIdx.y) * splits;
-    if (threadIdx.x < 32) {
-        float M = -INFINITY, L = 0.0f;
-        for (int s = lane; s < splits; s += 32) M = fmaxf(M, part_ml[2 * (at + s)]);
-        M = wmax(M);
-        for (int s = lane; s < splits; s += 32) L = fmaf(part_ml[2 * (at + s) + 1], expf(part_ml[2 * (at + s)] - M), L);
-        L = wsum(L);
-        for (int s = lane; s < splits; s += 32) wgt[s] = expf(part_ml[2 * (at + s)] - M) / L;
+    if (warp == 0) {
+        const float2* ml = reinterpret_cast<const float2*>(part_ml) + at;
+        const float2 none = make_float2(-INFINITY, 0.0f);
+        const float2 a = lane < splits ? ml[lane] : none, b = lane + 32 < splits ? ml[lane + 32] : none;
+        const float M = wmax(fmaxf(a.x, b.x));
+        const float wa = expf(a.x - M), wb = expf(b.x - M);
+        const float L = wsum(a.y * wa + b.y * wb);
+        wgt[lane] = wa / L;
+        wgt[lane + 32] = wb / L;
     }
     __syncthreads();
-    for (int c = threadIdx.x; c < vdim; c += 128) {
-        float acc = 0.0f;
-#pragma unroll 8
-        for (int s = 0; s < splits; s++) {
-            const float w = wgt[s];
-            const float o = w > 0.0f ? part_o[(at + s) * vdim + c] : 0.0f;     // (an empty split has written nothing)
-            acc = fmaf(w, o, acc);
+    for (int c0 = 0; c0 < vdim; c0 += 32 * V) {
+        const int c = c0 + lane * V;
+        FloatV<V> acc;
+#pragma unroll
+        for (int e = 0; e < V; e++) acc.v[e] = 0.0f;
+        for (int s0 = warp; s0 < splits; s0 += 8 * LC_BATCH) {
+            FloatV<V> o[LC_BATCH];
+#pragma unroll
+            for (int u = 0; u < LC_BATCH; u++) {
+                const int s = s0 + 8 * u;
+#pragma unroll
+                for (int e = 0; e < V; e++) o[u].v[e] = 0.0f;
+                if (s < splits && c < vdim && wgt[s] > 0.0f) o[u] = load_v<V>(part_o + (at + s) * vdim + c);     // (an empty split has written nothing)
+            }
+#pragma unroll
+            for (int u = 0; u < LC_BATCH; u++)
+#pragma unroll
+                for (int e = 0; e < V; e++) acc.v[e] = fmaf(wgt[min(s0 + 8 * u, 63)], o[u].v[e], acc.v[e]);
         }
-        out[(size_t)blockIdx.x * out_ld + blockIdx.y * vdim + c] = from_f<T>(acc);
+        store_v<V>(part[warp] + lane * V, acc);
+        __syncthreads();
+        if (threadIdx.x < 32 * V && c0 + (int)threadIdx.x < vdim) {
+            float t = 0.0f;
+#pragma unroll
+            for (int i = 0; i < 8; i++) t += part[i][threadIdx.x];
+            out[(size_t)blockIdx.x * out_ld + blockIdx.y * vdim + c0 + threadIdx.x] = from_f<T>(t);
+        }
+        __syncthreads();
     }
 }
 

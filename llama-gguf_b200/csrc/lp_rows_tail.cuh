@@ -12,6 +12,45 @@
 // expert e (0 when it is not chosen); sel[k] / selw[k] list the chosen experts in the order they were taken.
 __device__ __forceinline__ void route_row(const float* __restrict__ z, int E, int top, float* __restrict__ w, int* __restrict__ sel,
                                           float* __restrict__ selw, int lane, int mode, float scale, const float* __restrict__ corr = nullptr) {
+    if (E <= 32) {      // a lane per output: everything in registers
+        const float zl = lane < E ? z[lane] : -INFINITY;
+        float mx = -INFINITY, all = 0.0f;
+        if (mode == B200_ROUTE_SOFTMAX_TOP) {
+            mx = wmax(zl);
+            all = wsum(lane < E ? expf(zl - mx) : 0.0f);
+        }
+        float score = zl;
+        if (corr && lane < E) score = (mode == B200_ROUTE_SIGMOID_TOP ? sigmoid_f(zl) : expf(zl - mx) / all) + corr[lane];
+        if (!(score == score)) score = -INFINITY;
+        bool taken = lane >= E;
+        float wl = 0.0f, pk = 0.0f, zmax = mx, sum = 0.0f;
+        int ck = 0;                     // lane k: choice k and its weight
+        for (int k = 0; k < top; k++) {
+            float best = taken ? -INFINITY : score;
+            int bi = taken ? 0x7fffffff : lane;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+                if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
+            }
+            bi = min(bi, E - 1);
+            const float zb = __shfl_sync(0xffffffffu, zl, bi);
+            if (k == 0 && mode != B200_ROUTE_SOFTMAX_TOP) zmax = zb;
+            const float p = mode == B200_ROUTE_SIGMOID_TOP ? sigmoid_f(zb) : expf(zb - zmax);
+            sum += p;
+            if (lane == bi) { taken = true; wl = p; }
+            if (lane == k) { pk = p; ck = bi; }
+        }
+        const float inv = mode == B200_ROUTE_SIGMOID_TOP ? (scale != 0.0f ? scale : 1.0f) : mode == B200_ROUTE_SOFTMAX_TOP ? scale / all : 1.0f / sum;
+        if (lane < E) w[lane] = wl * inv;
+        if (lane < top) {
+            sel[lane] = ck;
+            selw[lane] = pk * inv;
+        }
+        __syncwarp();
+        return;
+    }
     for (int e = lane; e < E; e += 32) w[e] = 0.0f;
     __syncwarp();
     float zmax = 0.0f, sum = 0.0f;

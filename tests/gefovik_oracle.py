@@ -98,17 +98,21 @@ def silu_unit(h, W, pre):
     return W[pre + "down"] @ (z * sigmoid(z) * (W[pre + "up"] @ h))
 
 
-def expert_mixture(h, W, pre, mlp):
-    """Softmax over all outputs of the router; the correction decides who is chosen but not with what weight; the outputs behind the
-    experts' stand for the input itself."""
-    r = mlp["router"]
+def routing(h, W, pre):
+    """-> (softmax over all outputs of the router, the same plus the correction)"""
     z = W[pre + "router"] @ h
     s = np.exp(z - z.max())
     s /= s.sum()
-    choice = s + W[pre + "correction"]
-    order = sorted(range(len(z)), key=lambda e: (-choice[e], e))[:r["top"]]
+    return s, s + W[pre + "correction"]
+
+
+def expert_mixture(h, W, pre, mlp):
+    """The corrected scores decide who is chosen, the scores alone with what weight; the outputs behind the experts' stand for the input
+    itself."""
+    r = mlp["router"]
+    s, choice = routing(h, W, pre)
     out = np.zeros_like(h)
-    for e in order:
+    for e in sorted(range(len(s)), key=lambda e: (-choice[e], e))[:r["top"]]:
         out = out + s[e] * (silu_unit(h, W, pre + "e%d." % e) if e < r["experts"] else h)
     return out
 
@@ -123,6 +127,7 @@ class Sequence:
 
     def __init__(self, cfg, W):
         self.cfg, self.W, self.p = cfg, W, 0
+        self.margin = math.inf          # the closest call of any choice so far
         self.rows = [Rows(("k", "v")) for _ in cfg["layers"]]
 
     def token(self, tok):
@@ -135,6 +140,9 @@ class Sequence:
             mix = attention if L["type"] == "attention" else latent_attention
             x = sublayer_step(x, mix(x, self.p, W, pre + "mix.", L["mixer"], eps, self.rows[i]), W[pre + "norm1"], eps)
             mlp = L.get("mlp")
+            if mlp is not None and mlp["kind"] == "moe":
+                c = np.append(np.sort(routing(x, W, pre + "mlp.")[1])[::-1], -math.inf)
+                self.margin = min(self.margin, c[mlp["router"]["top"] - 1] - c[mlp["router"]["top"]])
             if mlp is not None:
                 ff = relu_unit(x, W, pre + "mlp.") if mlp["kind"] == "dense" else expert_mixture(x, W, pre + "mlp.", mlp)
                 x = sublayer_step(x, ff, W[pre + "norm2"], eps)

@@ -6,6 +6,7 @@ import math
 
 import numpy as np
 
+import gefovik_oracle as O
 import llama_gguf_b200 as B
 from llama_gguf_b200 import gefovik
 from llama_gguf_b200.safetensors_io import bf16_bits, bf16_to_f32
@@ -53,6 +54,25 @@ def random_weights(cfg, seed=0):
             a = rng.standard_normal(shape) * (1.0 / math.sqrt(shape[-1]))
         w[name] = bf16_to_f32(bf16_bits(np.asarray(a, dtype=np.float32))).reshape(shape)
     return w
+
+
+def clear_weights(cfg, sequences, seed, margin=0.012):
+    """Random weights with which no token of the sequences is a close call for a router, so that rounding turns no choice around"""
+    for s in range(seed, seed + 20000, 100):
+        w = random_weights(cfg, s)
+        w64, ok = f64(w), True
+        for toks in sequences:
+            q = O.Sequence(cfg, w64)
+            for t in toks:
+                q.token(t)
+                if q.margin < margin:
+                    ok = False
+                    break
+            if not ok:
+                break
+        if ok:
+            return w
+    raise AssertionError("no clear choices found")
 
 
 def gpu_model(cfg, weights, compute="float32", max_seq_len=256, max_batch=4, taps=False):
