@@ -149,6 +149,21 @@ constexpr bool epi_is_act(int epi) { return epi >= EPI_RELU2; }
 // act.x z^2 + z / 2 above zero, act.y (exp(z) - 1 - z) + z / 2 below
 __device__ __forceinline__ float xielu_f(float z, float2 act) { return fmaf(0.5f, z, z > 0.0f ? act.x * z * z : act.y * (expm1f(z) - z)); }
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+// 2^z and 1 / z by the special-function unit (relative error about 2^-22, tiny results flushed): where the result is rounded to bf16 next
+__device__ __forceinline__ float ex2_fast(float z) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z));
+    return r;
+}
+__device__ __forceinline__ float rcp_fast(float z) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z));
+    return r;
+}
+// the unit of a gated layer for a bf16 result
+template <int EPI> __device__ __forceinline__ float glu_fast(float v, float up) {
+    return EPI == EPI_SILU_GLU ? v * rcp_fast(1.0f + ex2_fast(-1.4426950408889634f * v)) * up : fmaxf(v, 0.0f) * up;
+}
 template <typename T, int EPI>
 __device__ __forceinline__ void epi_store(void* Y, size_t idx, float v, float2 act, float up = 0.0f) {
     if (EPI == EPI_STORE) reinterpret_cast<float*>(Y)[idx] = v;
@@ -395,6 +410,8 @@ __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict_
     const float bn = (bias && n < N) ? bias[n] : 0.0f;
     if constexpr (GLU) {
         float* ex = reinterpret_cast<float*>(base);        // [2 halves][16 tokens][64 units]
+        bf16* ob = reinterpret_cast<bf16*>(ex + 2 * 16 * 64);      // [2][32 tokens][64 units]: the units on their way out, 16 bytes per store
+        const bool v8 = N % 8 == 0 && ldy % 8 == 0 && ((uintptr_t)Y & 15) == 0;
         const bool up = tid >= TC_M / 2;
         __syncthreads();                                    // every thread's copies have landed, every MMA has read its stage
 #pragma unroll 1
@@ -413,10 +430,21 @@ __global__ void __launch_bounds__(128) lp_gemm_tc_kernel(const bf16* __restrict_
 #pragma unroll
             for (int c = 0; c < 16; c++) {
                 const float mine = alpha * __uint_as_float(v[up ? 16 + c : c]), other = alpha * ex[(up ? 16 * 64 : 0) + c * 64 + (tid & 63)];
-                const int t = t0 + c0 + (up ? 16 + c : c);
-                if (alive && n < N && t < R) epi_store<bf16, EPI>(Y, (size_t)t * ldy + n, up ? other : mine, act, up ? mine : other);
+                ob[(c0 & 32) * 64 + (up ? 16 + c : c) * 64 + (tid & 63)] = __float2bfloat16_rn(glu_fast<EPI>(up ? other : mine, up ? mine : other));
             }
             __syncthreads();
+            const bf16* o = ob + (c0 & 32) * 64;
+            bf16* y = reinterpret_cast<bf16*>(Y) + (size_t)(t0 + c0) * ldy + n0;
+            if (alive && v8) {
+#pragma unroll
+                for (int u = 0; u < 2; u++) {
+                    const int i = tid + u * 128, t = i >> 3, c = (i & 7) * 8;
+                    if (t0 + c0 + t < R && n0 + c < N) *reinterpret_cast<uint4*>(y + (size_t)t * ldy + c) = *reinterpret_cast<const uint4*>(o + t * 64 + c);
+                }
+            } else if (alive) {
+                for (int i = tid; i < 32 * 64; i += 128)
+                    if (t0 + c0 + (i >> 6) < R && n0 + (i & 63) < N) y[(size_t)(i >> 6) * ldy + (i & 63)] = o[i];
+            }
         }
     } else if (alive) {
 #pragma unroll 1
@@ -3021,7 +3049,7 @@ bool row_tile_launch(LpModel* m, const StepMeta& sm, const AttnGeom& ag, int n_r
         }
         if (dev >= 0 && dev < 64) once[dev] = true;
     }
-    launch(m, lp_row_tile_kernel<DK, DV>, dim3((unsigned)(((size_t)max_len * (ag.H / ag.G) + LT_ROWS - 1) / LT_ROWS), n_runs, ag.G), dim3(256), row_tile_smem<DK>(), sm, ag,
+    launch(m, lp_row_tile_kernel<DK, DV>, dim3((unsigned)(((size_t)max_len * (ag.H / ag.G) + LT_ROWS - 1) / LT_ROWS * ag.G), n_runs), dim3(256), row_tile_smem<DK>(), sm, ag,
            (const float*)m->qbuf, (bf16*)m->act_a);
     return true;
 }
@@ -3537,7 +3565,9 @@ void enqueue_step(LpModel* m, const StepMeta& sm, int R, int n_runs, int n_want,
             bool routed = par || moe_next != nullptr;
             if (p.in_conv > 0 || out_norm) {
                 StepRoute rt{};
-                if (R <= LS_ROWS && (out_norm ? m->use_fuse && (size_t)W * es <= 40 * 1024 : ring_step)) {       // few rows: the block that norms a row also routes it
+                // (a block per row reads the whole router: with many rows only one that stays in L1)
+                const bool own_route = out_norm ? m->use_fuse && (size_t)W * es <= 40 * 1024 && (R <= LS_ROWS || (size_t)rrows * W * es <= 64 * 1024) : ring_step && R <= LS_ROWS;
+                if (own_route) {       // few rows: the block that norms a row also routes it
                     rt.router = L.w_up; rt.bias = L.router_bias; rt.corr = L.router_corr; rt.rows = rrows; rt.E = outs; rt.top = e.top; rt.mode = e.route; rt.scale = e.route_scale;
                     rt.logits = m->P; rt.wts = m->moe_w; rt.sel = m->moe_sel; rt.selw = m->moe_selw; rt.shw = shw;
                     routed = true;

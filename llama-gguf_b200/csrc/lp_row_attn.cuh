@@ -228,7 +228,7 @@ __global__ void __launch_bounds__(256) lp_row_combine_kernel(int H, int vdim, co
 }
 
 // ------------------------------------------------------------------------------------------------ prompt rows (bf16)
-// The hpg = H / G heads of K/V head g (blockIdx.z) meet the same cached rows, so their (token, head) pairs are ONE list of query rows, pair f
+// The hpg = H / G heads of K/V head g = blockIdx.x % G meet the same cached rows, so their (token, head) pairs are ONE list of query rows, pair f
 // = (token f / hpg, head g hpg + f % hpg): a block of 8 warps takes LT_ROWS neighbours of the list (16 per warp) against tiles of LT_KEYS
 // cached rows.  A tile is
 // staged once, as bf16 [key][channel], and serves both products on the tensor pipe (mma.sync m16n8k16, f32 accumulators): ldmatrix gives
@@ -239,7 +239,7 @@ constexpr int LT_ROWS = 128, LT_KEYS = 64;
 template <int DK> constexpr size_t row_tile_smem() { return (size_t)(LT_ROWS + 2 * LT_KEYS) * (DK + 8) * 2 + 2 * LT_KEYS * 4; }
 // cap tanh(s / cap) through one exponential: 1 - 2 / (exp(2 s / cap) + 1), off by a few 1e-7 of cap
 __device__ __forceinline__ float soft_cap_exp(float s, float two_log2e_over_cap, float cap) {
-    return cap - __fdividef(2.0f * cap, exp2f(s * two_log2e_over_cap) + 1.0f);
+    return fmaf(-2.0f * cap, rcp_fast(ex2_fast(s * two_log2e_over_cap) + 1.0f), cap);
 }
 __device__ __forceinline__ void ldsm4(uint32_t* r, uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -255,11 +255,11 @@ __global__ void __launch_bounds__(256) lp_row_tile_kernel(StepMeta sm, AttnGeom 
     bf16* Qs = reinterpret_cast<bf16*>(lt_sm);          // [LT_ROWS][PITCH]
     bf16* Ks = Qs + LT_ROWS * PITCH;                    // [2][LT_KEYS][PITCH]
     float* Fs = reinterpret_cast<float*>(Ks + 2 * LT_KEYS * PITCH);     // [2][LT_KEYS] factors of the rows (k_inv)
-    const int run = blockIdx.y, g = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+    const int run = blockIdx.y, g = blockIdx.x % a.G, bx = blockIdx.x / a.G, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     const int r0 = sm.run_start[run], len = sm.run_start[run + 1] - r0, p0 = sm.run_pos0[run];
     const int hpg = a.H / a.G, rows = len * hpg, nb = (rows + LT_ROWS - 1) / LT_ROWS;
-    if ((int)blockIdx.x >= nb) return;
-    const int f0 = (nb - 1 - (int)blockIdx.x) * LT_ROWS, D = a.dim, ldk = a.G * D;
+    if (bx >= nb) return;
+    const int f0 = (nb - 1 - bx) * LT_ROWS, D = a.dim, ldk = a.G * D;
     const float* cache = reinterpret_cast<const float*>(sm.run_kv[run] + a.kv_off) + g * D;
     const float* kinv = a.k_inv ? reinterpret_cast<const float*>(sm.run_kv[run] + a.kv_off) + (size_t)a.cap * ldk + g : nullptr;
     // pair f of the list: its place among the step's (row, head) pairs
@@ -374,14 +374,14 @@ __global__ void __launch_bounds__(256) lp_row_tile_kernel(StepMeta sm, AttnGeom 
             x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
             const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
             const float b0 = n0 == -INFINITY ? 0.0f : n0, b1 = n1 == -INFINITY ? 0.0f : n1;      // (a row without a visible key yet: all weights 0)
-            const float c0 = exp2f(m0 - b0), c1 = exp2f(m1 - b1);
+            const float c0 = ex2_fast(m0 - b0), c1 = ex2_fast(m1 - b1);
             m0 = n0;
             m1 = n1;
             float s0 = 0.0f, s1 = 0.0f;
             uint32_t pa[LT_KEYS / 16][4];
 #pragma unroll
             for (int n = 0; n < LT_KEYS / 8; n++) {
-                const float e0 = exp2f(sc[n][0] - b0), e1 = exp2f(sc[n][1] - b0), e2 = exp2f(sc[n][2] - b1), e3 = exp2f(sc[n][3] - b1);
+                const float e0 = ex2_fast(sc[n][0] - b0), e1 = ex2_fast(sc[n][1] - b0), e2 = ex2_fast(sc[n][2] - b1), e3 = ex2_fast(sc[n][3] - b1);
                 s0 += e0 + e1;
                 s1 += e2 + e3;
                 pa[n >> 1][(n & 1) * 2] = pack_bf2(e0, e1);
