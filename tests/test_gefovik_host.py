@@ -116,11 +116,11 @@ def test_parse_config_reads_every_constant():
 def test_tensor_list_follows_the_config():
     from llama_gguf_b200 import gefovik
 
-    cfg = S.config([S.attn(heads=6, kv_heads=3, dim=8, mlp=S.dense(12)), S.latent(heads=3, dim=16, vdim=24, kv_rank=40, mlp=S.moe(experts=3, identity=2, top=2, ff=10)),
+    cfg = S.config([S.attn(heads=6, kv_heads=2, dim=12, mlp=S.dense(12)), S.latent(heads=3, dim=16, vdim=24, kv_rank=40, mlp=S.moe(experts=3, identity=2, top=2, ff=10)),
                     S.attn(mlp=None)], width=32, vocab=50)
     t = gefovik.tensor_shapes(cfg)
     assert t["embed"] == (50, 32) and "head" not in t and t["final.norm"] == (32,)
-    assert t["l0.mix.q"] == (48, 32) and t["l0.mix.k"] == (24, 32) and t["l0.mix.o"] == (32, 48) and "l0.mix.v" not in t and "l0.mix.sink" not in t
+    assert t["l0.mix.q"] == (72, 32) and t["l0.mix.k"] == (24, 32) and t["l0.mix.o"] == (32, 72) and "l0.mix.v" not in t and "l0.mix.sink" not in t
     assert t["l0.mlp.gate"] == (12, 32) and t["l0.mlp.up"] == (12, 32) and t["l0.mlp.down"] == (32, 12)
     assert t["l1.mix.q"] == (48, 32) and t["l1.mix.dkv"] == (40, 32) and t["l1.mix.dkv.norm"] == (40,) and t["l1.mix.uk"] == (48, 40)
     assert t["l1.mix.uv"] == (72, 40) and t["l1.mix.sink"] == (3,) and t["l1.mix.g"] == (3, 32) and t["l1.mix.o"] == (32, 72)

@@ -539,7 +539,7 @@ def test_bad_arguments(b200):
 
 
 # ---------------------------------------------------------------------------------------------------- kernels against their plain forms
-@pytest.mark.parametrize("layer", [S.attn(heads=6, kv_heads=3, dim=64), S.attn(heads=5, kv_heads=1, dim=16), S.attn(heads=4, kv_heads=4, dim=128, scale=0.1),
+@pytest.mark.parametrize("layer", [S.attn(heads=8, kv_heads=2, dim=64), S.attn(heads=5, kv_heads=1, dim=16), S.attn(heads=4, kv_heads=4, dim=128, scale=0.1),
                                    S.attn(heads=2, kv_heads=1, dim=24), S.attn(heads=14, kv_heads=2, dim=48), S.attn(heads=2, kv_heads=1, dim=176, scale=0.1),
                                    S.latent(heads=3, kv_rank=64), S.latent(heads=1, kv_rank=96), S.latent(heads=7, kv_rank=224)])
 def test_tile_attention_against_warp_attention(b200, monkeypatch, layer):
